@@ -126,14 +126,16 @@ class ScheduleEntry:
     writes nothing).
 
     What the model feeds into the stream right before the entry's layer (a repeated range of
-    layers starts each pass this way): ``add_embedding`` adds the tokens' input embedding once
-    more, ``add_pass_vector`` adds row ``i`` of the model's ``pass_vectors`` table to every token.
+    layers starts each pass this way): ``mix_embedding`` replaces the stream by a product of the stream and the
+    embedding output (the model's ``pass_input``), ``add_embedding`` adds the tokens' input embedding once
+    more, ``add_pass_vector`` adds row ``i`` of the model's ``pass_vectors`` table to every token; in this order.
     """
 
     layer: int
     cache_from: Optional[int] = None
     add_embedding: bool = False
     add_pass_vector: Optional[int] = None
+    mix_embedding: bool = False
 
 
 @dataclass(frozen=True)
@@ -153,6 +155,8 @@ class ModelSpec:
     head_name: str = "lm_head"
     pass_vectors: Optional[PartSpec] = None  # an embedding part with ``vector(i)`` (kind "pass_vectors")
     pass_vectors_name: str = "pass_vectors"
+    pass_input: Optional[PartSpec] = None  # an embedding part with ``keep`` and ``mix`` (kind "stream_mix")
+    pass_input_name: str = "pass_input"
     source: Any = None  # the architecture's own typed config, kept for reporting
 
     def validate(self) -> None:
@@ -171,6 +175,8 @@ class ModelSpec:
                     raise ConfigError(
                         f"schedule[{i}].cache_from={e.cache_from} names an entry that owns no cache"
                     )
+            if e.mix_embedding and self.pass_input is None:
+                raise ConfigError(f"schedule[{i}].mix_embedding: the model has no pass_input")
             if e.add_pass_vector is not None:
                 n_vec = int(self.pass_vectors["passes"]) if self.pass_vectors is not None else 0
                 if not 0 <= e.add_pass_vector < n_vec:

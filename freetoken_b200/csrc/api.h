@@ -78,7 +78,75 @@ typedef struct {
   float sink_logit;
   // with has_sink: one logit per query head [n_q_heads] (float32) instead of sink_logit; null = sink_logit for all
   const float* sink_heads;
+  // scores (scaled) become softcap * tanh(score / softcap); 0 = as they are.  Not with block selection, a bias by
+  // distance or the form with two 128-row tiles.
+  float softcap;
 } FtkAttnExtras;
+
+// What ftk_stream_step does to the rows of the 32-bit stream (see gated_stream.cu).  x, passed, shared, gate, raw_out,
+// out and conv_out are of `dtype`.
+typedef struct {
+  float* residual;           // [T, hidden]
+  const float* vec;          // [hidden] added to every row first, or null
+  const void* x;             // [*, hidden] the sub-layer's rows, or the experts' rows with route_pos; null: none
+  const int32_t* route_pos;  // [T, top_k] or null; negative: a route without a row
+  int top_k;
+  int n_routes;
+  const float* aux;          // [T, 2] (weight of `passed`, weight of `shared`), or null (0, 1)
+  const void* passed;        // [T, hidden] or null
+  const void* shared;        // [T, hidden] or null
+  const void* gate;          // [T, hidden] logits of the gate on the result, or null
+  const float* gate_bias;    // [hidden] or null
+  const float* post_w;       // [hidden] weight of the result's norm
+  float post_eps;
+  void* raw_out;             // the stream itself, row r at raw_out + r * raw_stride elements, or null
+  long long raw_stride;
+  const float* pre_w;        // [hidden] weight of the stream's norm, or null: no outputs below
+  float pre_eps;
+  void* out;                 // [n_rows, hidden] or null
+  float* norm_f32;           // [n_rows, hidden] the same, not rounded, or null (may be the stream)
+  const float* conv_w;       // [hidden, taps] or null; rows are then one token per segment
+  int taps;
+  float* state;              // [n_slots, taps - 1, hidden]
+  int n_slots;
+  const int32_t* state_slots;  // [n_rows]
+  const int32_t* seg_info;     // [n_rows, 4]
+  void* conv_out;            // [n_rows, hidden]
+  float* conv_out_f32;       // [n_rows, hidden] float32(conv_out), or null
+  const int32_t* rows;       // null, or the rows to take
+  int n_rows;
+  int hidden;
+  int groups;
+  int dtype;
+} FtkStreamStep;
+
+// What ftk_conv_rope_store reads and writes (see conv_rope.cu).
+typedef struct {
+  const void* x;             // [n_tokens, *] rows of q | k | v, row stride x_stride elements
+  long long x_stride;
+  int dtype;
+  const float* conv_w;       // [channels, taps]
+  int taps;
+  float* state;              // [n_slots, taps - 1, channels] or null (taps == 1)
+  int n_slots;
+  const int32_t* state_slots;
+  const int32_t* seg_info;
+  int n_segs;
+  int n_tokens;
+  int n_heads, n_kv_heads, maps, dim, vdim;
+  int n_rot;                 // leading dimensions of a map's head that turn
+  int interleaved;
+  const int32_t* positions;
+  const float* table;        // [max_pos, n_rot] cos || sin, or null
+  int max_pos;
+  void* q_out;               // [n_tokens, n_heads * maps, pad_dim]
+  void* k_slab;              // [num_pages, n_kv_heads, page_size, pad_dim]
+  void* v_slab;
+  const int32_t* slot_map;   // [n_tokens]
+  int page_size;
+  int num_pages;
+  int pad_dim;
+} FtkConvRope;
 
 const char* ftk_last_error(void);
 
@@ -94,6 +162,12 @@ int ftk_add_rmsnorm_routes(const void* y, int y_dtype, const int32_t* route_pos,
                            float* out_f32, const int32_t* rows, int n_rows, int hidden, float eps, int gemma,
                            void* stream);
 int ftk_stream_add_norm(const FtkStreamNorm* args, void* stream);
+int ftk_stream_step(const FtkStreamStep* args, void* stream);
+int ftk_conv_rope_store(const FtkConvRope* args, void* stream);
+// out[t, h, :] = unit(o[t, maps h, :vdim] - lambda o[t, maps h + 1, :vdim]) * scale for two maps a head; o rows of
+// o_stride elements, out [n_tokens, n_heads, vdim]; `lambda` is one float on the device
+int ftk_diff_heads(const void* o, int o_stride, int dtype, const float* lambda, float eps, float scale, void* out,
+                   int n_tokens, int n_heads, int vdim, void* stream);
 // o[t, h, :] *= sigmoid(gates[t * gate_stride + h]) in place; o [T, n_heads, head_dim]
 int ftk_head_gate(void* o, int dtype, const void* gates, long long gate_stride, int n_tokens, int n_heads,
                   int head_dim, void* stream);
@@ -265,15 +339,19 @@ int ftk_sparse_select(const void* iq, const void* ik_slab, int dtype, const int3
 // Whether bfloat16 block scores of these sizes can be taken on the tensor cores (`scores [T, n_heads, max_blocks]`
 // float32 scratch must then be given to ftk_sparse_select).
 int ftk_sparse_score_fits(int n_heads, int dim, int block_size);
+// A token's row of logits may hold n_extra values behind the experts' (0 or 1).  aux [n_tokens, 2] or null: the sum of
+// the weights of the chosen ids >= n_real (experts without tensors), and the sigmoid of the extra logit (1 without).
 int ftk_router_topk(const float* logits, int n_parts, const float* bias, int n_tokens, int n_experts, int top_k,
-                    int scoring, float scale, int32_t* ids, float* weights, void* stream);
+                    int scoring, float scale, int32_t* ids, float* weights, int n_extra, int n_real, float* aux,
+                    void* stream);
 // Router logits (float32 x [T, hidden] times gate_w [E, hidden]), choice and sort of the routes in one
 // launch, for steps of at most 32 tokens (beyond that the
 // separate kernels are faster); ftk_moe_route_fits says whether the sizes are taken.
 int ftk_moe_route_fits(int n_tokens, int hidden, int n_experts, int top_k);
 int ftk_moe_route(const float* x, const float* gate_w, const float* bias, int n_tokens, int hidden, int n_experts,
                   int top_k, int scoring, float scale, float* logits, int32_t* ids, float* weights,
-                  int32_t* counts, int32_t* offsets, int32_t* routes, int32_t* pos, int do_sort, void* stream);
+                  int32_t* counts, int32_t* offsets, int32_t* routes, int32_t* pos, int do_sort, int n_extra,
+                  int n_real, float* aux, void* stream);
 // Products of very few tokens (bfloat16): the weights are streamed once by warps of every SM (gemv.cu).
 int ftk_small_linear_fits(int n_tokens, int n_out, int k);
 int ftk_small_linear(const void* x, const void* w, void* out, int n_tokens, int n_out, int k, void* stream);
@@ -301,7 +379,7 @@ int ftk_moe_gemm2(const void* a, const void* w2, int dtype, const int32_t* exper
                   const int32_t* sorted_routes, const float* topk_weights, int n_experts, int n_routes,
                   int hidden, int inter, void* out, void* stream);
 int ftk_moe_combine(const void* y, int dtype, const int32_t* route_pos, int n_tokens, int top_k,
-                    int hidden, const void* shared, void* out, void* stream);
+                    int hidden, const void* shared, const float* aux, const void* passed, void* out, void* stream);
 // Status words of the kernels' bounded waits: out[0] = first code since the last call (0 = none),
 // out[1] = block that recorded it.  Synchronises with the device and clears the words.
 // Kernel forms launched so far, as "name<TAB>count" lines (see ftk::note_variant); returns the bytes needed.

@@ -63,7 +63,18 @@ struct AttnParams {
   float sink;
   // one sink logit per query head instead of `sink` (learned sinks); nullptr: `sink` for every head
   const float* sink_heads;
+  // scaled scores s become softcap * tanh(s / softcap); 0: as they are
+  float softcap;
 };
+
+// softcap * tanh(x * to_arg) for results in `out_scale` units: out_scale * (1 - 2 / (e^(2 x to_arg) + 1)), with the
+// exponential's argument in base 2.  About 1e-7 of out_scale away from the exact value; saturates cleanly at both ends.
+__device__ __forceinline__ float capped_score(float x, float to_exp2, float out_scale) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * to_exp2));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.f));
+  return fmaf(-2.f * out_scale, r, out_scale);
+}
 
 // What the sink adds to a row's sum of exponentials taken relative to the maximum `m` (natural logarithm domain).
 // `head` is the row's query head.
@@ -201,6 +212,7 @@ __global__ void __launch_bounds__(kF32Rows * 32) attention_f32_kernel(AttnParams
       float dot = 0.f;
       for (int d = 0; d < D; ++d) dot = fmaf(qr[d], kr[d], dot);
       s = dot * p.scale + dist_bias_at(brow, p.dist_len, q_pos - key);
+      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
     }
     const float cm = warp_max(s);
     if (cm == -INFINITY) continue;  // nothing visible in this chunk
@@ -469,7 +481,10 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(AttnParams p) {
   const int qp1 = r1 < R ? pos_base + r1 / G : -1;
   const int lo0 = p.window > 0 ? qp0 - p.window + 1 : 0;
   const int lo1 = p.window > 0 ? qp1 - p.window + 1 : 0;
-  const float sl2 = p.scale * 1.4426950408889634f;
+  // with a soft cap the scores are scaled while they are capped
+  const float cap_arg = p.softcap > 0.f ? 2.f * p.scale / p.softcap * 1.4426950408889634f : 0.f;
+  const float cap_out = p.softcap * 1.4426950408889634f;
+  const float sl2 = p.softcap > 0.f ? 1.f : p.scale * 1.4426950408889634f;
   const bool tied = p.k == p.v;
   const float kLog2e = 1.4426950408889634f;
   const float* brow0 = (p.dist_bias && r0 < R) ? p.dist_bias + (size_t)(kvh * G + r0 % G) * p.dist_len : nullptr;
@@ -509,6 +524,12 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(AttnParams p) {
           mma_bf16(s[2 * n2 + 1], a, b[2], b[3]);
         }
       }
+    }
+    if (p.softcap > 0.f) {
+#pragma unroll
+      for (int n = 0; n < kBN / 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[n][e] = capped_score(s[n][e], cap_arg, cap_out);
     }
     // mask, running max
     const int c0 = it.kb + iter * kBN;
@@ -737,7 +758,10 @@ __global__ void __launch_bounds__(128) attention_decode_bf16_kernel(AttnParams p
   const int qp1 = r1 < R ? pos_base + r1 / G : -1;
   const int lo0 = p.window > 0 ? qp0 - p.window + 1 : 0;
   const int lo1 = p.window > 0 ? qp1 - p.window + 1 : 0;
-  const float sl2 = p.scale * 1.4426950408889634f;
+  // with a soft cap the scores are scaled while they are capped
+  const float cap_arg = p.softcap > 0.f ? 2.f * p.scale / p.softcap * 1.4426950408889634f : 0.f;
+  const float cap_out = p.softcap * 1.4426950408889634f;
+  const float sl2 = p.softcap > 0.f ? 1.f : p.scale * 1.4426950408889634f;
   const bool tied = p.k == p.v;
   const float kLog2e = 1.4426950408889634f;
   const float* brow0 = (p.dist_bias && r0 < R) ? p.dist_bias + (size_t)(kvh * G + r0 % G) * p.dist_len : nullptr;
@@ -772,6 +796,12 @@ __global__ void __launch_bounds__(128) attention_decode_bf16_kernel(AttnParams p
         mma_bf16(s[0], a, b[0], b[1]);
         mma_bf16(s[1], a, b[2], b[3]);
       }
+    }
+    if (p.softcap > 0.f) {
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[n][e] = capped_score(s[n][e], cap_arg, cap_out);
     }
     const int c0 = it.kb + iter * kBN + warp * 16;
     float mx0 = -INFINITY, mx1 = -INFINITY;
@@ -1024,10 +1054,15 @@ static int paged_attention_tc_impl(const void* q, const void* k_slab, const void
   p.has_sink = extras ? extras->has_sink : 0;
   p.sink = extras ? extras->sink_logit : 0.f;
   p.sink_heads = extras ? extras->sink_heads : nullptr;
+  p.softcap = extras ? extras->softcap : 0.f;
+  FTK_REQUIRE(!(p.softcap > 0.f) || (!pair && !p.dist_bias && scale > 0.f),
+              "paged_attention_tc: a soft cap goes with one query tile a piece, a positive scale and no distance bias");
   FTK_REQUIRE(!p.has_sink || form == kTcSingle,
               "paged_attention_tc: of the tcgen05 kernels the one with 128-row tiles takes a softmax sink");
   cudaStream_t s = (cudaStream_t)stream;
-  if (p.dist_bias) note_variant(few ? "attention: tcgen05, tiles of at most 16 rows, bias by distance"
+  if (p.softcap > 0.f) note_variant(few ? "attention: tcgen05, tiles of at most 16 rows, soft cap"
+                                        : "attention: tcgen05, 128-row query tiles, soft cap");
+  else if (p.dist_bias) note_variant(few ? "attention: tcgen05, tiles of at most 16 rows, bias by distance"
                                     : "attention: tcgen05, 128-row query tiles, bias by distance");
   else if (window > 0 || p.has_sink) note_variant("attention: tcgen05, 128-row query tiles, window or sink");
   else
@@ -1125,6 +1160,9 @@ static int paged_attention_impl(const void* q, const void* k_slab, const void* v
   p.has_sink = extras ? extras->has_sink : 0;
   p.sink = extras ? extras->sink_logit : 0.f;
   p.sink_heads = extras ? extras->sink_heads : nullptr;
+  p.softcap = extras ? extras->softcap : 0.f;
+  FTK_REQUIRE(!(p.softcap > 0.f) || (!sel && !p.dist_bias),
+              "paged_attention: a soft cap cannot be combined with block selection or a distance bias");
   FTK_REQUIRE(!p.has_sink || !sel, "paged_attention: a sink cannot be combined with block selection");
   if (extras && extras->kv_split > 1) {
     FTK_REQUIRE(!sel && p.G % extras->kv_split == 0 && (long long)n_kv_heads * extras->kv_split <= 65535,

@@ -155,13 +155,16 @@ __device__ __forceinline__ uint32_t tc_pack(float lo, float hi) {
 
 // Softmax and epilogue of a tile's rows 0..15 by one warp (the warp of TMEM lanes 0..31), for tiles
 // that have no more rows: thread t has rows t / 4 and t / 4 + 8 and a quarter of their columns.
-template <bool BIASED>
+template <bool BIASED, bool CAPPED>
 __device__ __forceinline__ void attention_tc_few_rows(const AttnParams& p, uint32_t tmem, int lane, int n_work, int n_rounds,
                                                       uint64_t* s_full, uint64_t* s_empty, uint64_t* p_full,
                                                       uint64_t* pv_done, uint64_t* o_free, volatile int* abortp,
                                                       int* abort_flag) {
   const int G = p.G;
-  const float sl2 = p.scale * 1.4426950408889634f;
+  // with a soft cap the scores are scaled while they are capped
+  const float sl2 = CAPPED ? 1.f : p.scale * 1.4426950408889634f;
+  const float cap_arg = CAPPED ? 2.f * p.scale / p.softcap * 1.4426950408889634f : 0.f;
+  const float cap_out = p.softcap * 1.4426950408889634f;
   const int ra = lane >> 2, rb = ra + 8, cq = lane & 3;
   auto fail = [&](int code) {
     atomicCAS(&g_attn_status[0], 0, code);
@@ -201,6 +204,10 @@ __device__ __forceinline__ void attention_tc_few_rows(const AttnParams& p, uint3
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty[sb]);  // the next product may overwrite this buffer
+      if constexpr (CAPPED) {
+#pragma unroll
+        for (int i = 0; i < 64; ++i) v[i] = capped_score(v[i], cap_arg, cap_out);
+      }
       const int key0 = it.kb + j * kTcKeys;
       const bool interior = __all_sync(0xffffffffu, key0 + kTcKeys - 1 <= min(hi_a, hi_b));
       if (!interior) {
@@ -378,7 +385,7 @@ __device__ __forceinline__ void attention_tc_few_rows(const AttnParams& p, uint3
   }
 }
 
-template <bool FEW, bool BIASED = false>
+template <bool FEW, bool BIASED = false, bool CAPPED = false>
 __global__ void __launch_bounds__(kTcThreads)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, AttnParams p) {
@@ -629,13 +636,15 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
   } else if (FEW) {
     // ------------------------------------------------------------ softmax and epilogue of rows 0..15 by one warp
     if ((warp & 3) == 0) {
-      attention_tc_few_rows<BIASED>(p, tmem, lane, n_work, n_rounds, s_full, s_empty, p_full, pv_done, &o_free, abortp, &abort_flag);
+      attention_tc_few_rows<BIASED, CAPPED>(p, tmem, lane, n_work, n_rounds, s_full, s_empty, p_full, pv_done, &o_free, abortp, &abort_flag);
     }
   } else {
     // ------------------------------------------------------------ softmax and epilogue (warps 2..5), one row per thread
     const int quad = warp & 3;
     const int r = quad * 32 + lane;           // row of the tile = TMEM lane
-    const float sl2 = p.scale * 1.4426950408889634f;
+    const float sl2 = CAPPED ? 1.f : p.scale * 1.4426950408889634f;  // (capped scores are scaled while they are capped)
+    const float cap_arg = CAPPED ? 2.f * p.scale / p.softcap * 1.4426950408889634f : 0.f;
+    const float cap_out = p.softcap * 1.4426950408889634f;
     const uint32_t lane_addr = tmem + ((uint32_t)(quad * 32) << 16);
     bool ok = true;
     int g0 = 0;  // tiles of the pieces before this one
@@ -677,6 +686,15 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty[sb]);  // the next product may overwrite this buffer
+      if constexpr (CAPPED) {
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          v0[i] = capped_score(v0[i], cap_arg, cap_out);
+          v1[i] = capped_score(v1[i], cap_arg, cap_out);
+          v2[i] = capped_score(v2[i], cap_arg, cap_out);
+          v3[i] = capped_score(v3[i], cap_arg, cap_out);
+        }
+      }
       // a tile that every row of the warp reads in full needs no mask (most tiles of a long prompt)
       const bool interior = __all_sync(0xffffffffu, key0 + kTcKeys - 1 <= hi && key0 >= lo);
       if (!interior) {
@@ -860,7 +878,9 @@ inline int launch_attention_tc(const AttnParams& p, int n_tokens, cudaStream_t s
     if (cudaFuncSetAttribute(attention_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess ||
         cudaFuncSetAttribute(attention_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess ||
         cudaFuncSetAttribute(attention_tc_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess ||
-        cudaFuncSetAttribute(attention_tc_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess)
+        cudaFuncSetAttribute(attention_tc_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess ||
+        cudaFuncSetAttribute(attention_tc_kernel<false, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess ||
+        cudaFuncSetAttribute(attention_tc_kernel<true, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess)
       return 2;
     configured = true;
   }
@@ -888,7 +908,11 @@ inline int launch_attention_tc(const AttnParams& p, int n_tokens, cudaStream_t s
   }
   const long long n_work = (long long)p.n_items * p.Hkv;  // one CTA per SM, each takes every sms-th piece of work
   const int grid = (int)(n_work < sms ? n_work : sms);
-  if (p.tile_rows == kTcFewRows && p.dist_bias) {
+  if (p.tile_rows == kTcFewRows && p.softcap > 0.f) {
+    FTK_LAUNCH((attention_tc_kernel<true, false, true>), grid, kTcThreads, kTcSmem, s, mq, mk, mv, p);
+  } else if (p.softcap > 0.f) {
+    FTK_LAUNCH((attention_tc_kernel<false, false, true>), grid, kTcThreads, kTcSmem, s, mq, mk, mv, p);
+  } else if (p.tile_rows == kTcFewRows && p.dist_bias) {
     FTK_LAUNCH((attention_tc_kernel<true, true>), grid, kTcThreads, kTcSmem, s, mq, mk, mv, p);
   } else if (p.tile_rows == kTcFewRows) {
     FTK_LAUNCH(attention_tc_kernel<true>, grid, kTcThreads, kTcSmem, s, mq, mk, mv, p);

@@ -214,7 +214,8 @@ __global__ void moe_gather_kernel(const T* __restrict__ h, const int32_t* __rest
 // (python/freetoken/kernel/triton/fused_moe.py:111-153).
 template <typename T>
 __global__ void moe_combine_kernel(const T* __restrict__ y, const int32_t* __restrict__ route_pos, int top_k,
-                                   int hidden, int n_routes, const T* __restrict__ shared, T* __restrict__ out) {
+                                   int hidden, int n_routes, const T* __restrict__ shared, const float* __restrict__ aux,
+                                   const T* __restrict__ passed, T* __restrict__ out) {
   pdl_wait();
   pdl_trigger();
   const int t = blockIdx.y;
@@ -225,7 +226,8 @@ __global__ void moe_combine_kernel(const T* __restrict__ y, const int32_t* __res
     const int p = route_pos[t * top_k + j];
     if (p >= 0 && p < n_routes) acc += to_float(y[(size_t)p * hidden + i]);
   }
-  if (shared) acc += to_float(shared[(size_t)t * hidden + i]);
+  if (passed) acc = fmaf(aux[2 * t], to_float(passed[(size_t)t * hidden + i]), acc);
+  if (shared) acc = fmaf(aux ? aux[2 * t + 1] : 1.f, to_float(shared[(size_t)t * hidden + i]), acc);
   out[(size_t)t * hidden + i] = from_float<T>(acc);
 }
 
@@ -402,7 +404,9 @@ extern "C" int ftk_moe_gather(const void* h, int dtype, const int32_t* sorted_ro
 }
 
 extern "C" int ftk_moe_combine(const void* y, int dtype, const int32_t* route_pos, int n_tokens, int top_k,
-                               int hidden, const void* shared, void* out, void* stream) {
+                               int hidden, const void* shared, const float* aux, const void* passed, void* out,
+                               void* stream) {
+  FTK_REQUIRE(!passed || aux, "moe_combine: passed rows need their weights");
   FTK_REQUIRE(dtype_ok(dtype), "moe_combine: bad dtype %d", dtype);
   FTK_REQUIRE(n_tokens >= 0 && top_k > 0 && hidden > 0, "moe_combine: bad sizes");
   if (n_tokens == 0) return 0;
@@ -414,10 +418,14 @@ extern "C" int ftk_moe_combine(const void* y, int dtype, const int32_t* route_po
     if (dtype == FTK_F32)
       FTK_LAUNCH(moe_combine_kernel<float>, grid, 256, 0, s, (const float*)y, route_pos + (size_t)t0 * top_k, top_k, hidden,
                                                      n_tokens * top_k, shared ? (const float*)shared + (size_t)t0 * hidden : nullptr,
+                                                     aux ? aux + (size_t)t0 * 2 : nullptr,
+                                                     passed ? (const float*)passed + (size_t)t0 * hidden : nullptr,
                                                      (float*)out + (size_t)t0 * hidden);
     else
       FTK_LAUNCH(moe_combine_kernel<__nv_bfloat16>, grid, 256, 0, s, (const __nv_bfloat16*)y, route_pos + (size_t)t0 * top_k, top_k, hidden,
                                                              n_tokens * top_k, shared ? (const __nv_bfloat16*)shared + (size_t)t0 * hidden : nullptr,
+                                                             aux ? aux + (size_t)t0 * 2 : nullptr,
+                                                             passed ? (const __nv_bfloat16*)passed + (size_t)t0 * hidden : nullptr,
                                                              (__nv_bfloat16*)out + (size_t)t0 * hidden);
   }
   FTK_LAUNCH_CHECK("moe_combine");

@@ -16,14 +16,29 @@ constexpr int kRouterWarps = 4;
 // A token's logit of expert e: the row holds n_parts blocks of n_experts values that are added in their
 // order (one block: the logits themselves; three: the products of the activations with the three
 // bfloat16 pieces of the float32 router weights, largest first).
-__device__ __forceinline__ float logit_of(const float* __restrict__ row, int e, int n_experts, int n_parts) {
+__device__ __forceinline__ float logit_of(const float* __restrict__ row, int e, int part_stride, int n_parts) {
   float v = __ldcg(row + e);
-  for (int q = 1; q < n_parts; ++q) v += __ldcg(row + (size_t)q * n_experts + e);
+  for (int q = 1; q < n_parts; ++q) v += __ldcg(row + (size_t)q * part_stride + e);
   return v;
 }
 
+// What a token's routing leaves beside ids and weights (one warp): the sum of the chosen experts' weights that belong
+// to ids from n_real on (experts without tensors), and the sigmoid of the logit behind the experts' (1 without one).
+__device__ __forceinline__ void token_aux(const float* __restrict__ row, int part_stride, int n_parts, int n_experts, int n_extra,
+                                          int n_real, const int32_t* ids, const float* weights, int top_k, float* __restrict__ aux) {
+  const int lane = threadIdx.x & 31;
+  __syncwarp();  // the warp's own stores of ids and weights
+  float sum = 0.f;
+  for (int j = lane; j < top_k; j += 32) sum += ids[j] >= n_real ? weights[j] : 0.f;
+  sum = warp_sum(sum);
+  if (lane == 0) {
+    aux[0] = sum;
+    aux[1] = n_extra ? 1.f / (1.f + expf(-logit_of(row, n_experts, part_stride, n_parts))) : 1.f;
+  }
+}
+
 // Scores, choice and weights of one token, by one warp.  `s` and `c` hold n_experts floats each.
-__device__ __forceinline__ void route_token(const float* __restrict__ row, int n_parts, const float* __restrict__ bias,
+__device__ __forceinline__ void route_token(const float* __restrict__ row, int part_stride, int n_parts, const float* __restrict__ bias,
                                             int n_experts, int top_k, int scoring, float scale, float* s, float* c,
                                             int32_t* __restrict__ ids, float* __restrict__ weights,
                                             int32_t* ids_copy) {
@@ -33,14 +48,14 @@ __device__ __forceinline__ void route_token(const float* __restrict__ row, int n
   const float* pre = scoring == FTK_SCORE_SOFTMAX_OF_CHOSEN ? bias : nullptr;
   if (pre) bias = nullptr;
   if (scoring == FTK_SCORE_SIGMOID || scoring == FTK_SCORE_SIGMOID_RAW) {
-    for (int e = lane; e < n_experts; e += 32) s[e] = 1.f / (1.f + expf(-logit_of(row, e, n_experts, n_parts)));
+    for (int e = lane; e < n_experts; e += 32) s[e] = 1.f / (1.f + expf(-logit_of(row, e, part_stride, n_parts)));
   } else {
     float mx = -INFINITY;
-    for (int e = lane; e < n_experts; e += 32) mx = fmaxf(mx, logit_of(row, e, n_experts, n_parts) + (pre ? pre[e] : 0.f));
+    for (int e = lane; e < n_experts; e += 32) mx = fmaxf(mx, logit_of(row, e, part_stride, n_parts) + (pre ? pre[e] : 0.f));
     mx = warp_max(mx);
     float sum = 0.f;
     for (int e = lane; e < n_experts; e += 32) {
-      const float v = expf(logit_of(row, e, n_experts, n_parts) + (pre ? pre[e] : 0.f) - mx);
+      const float v = expf(logit_of(row, e, part_stride, n_parts) + (pre ? pre[e] : 0.f) - mx);
       s[e] = v;
       sum += v;
     }
@@ -80,7 +95,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ row, int n
     }
     __syncwarp();
   }
-  const float denom = scoring == FTK_SCORE_SIGMOID_RAW ? 1.f : scoring == FTK_SCORE_SIGMOID ? wsum + 1e-20f : wsum;  // (raw: the scores as they are)
+  const float denom = scoring == FTK_SCORE_SIGMOID_RAW ? 1.f : scoring == FTK_SCORE_SOFTMAX_OF_CHOSEN ? wsum : wsum + 1e-20f;  // (raw: the scores as they are)
   for (int j = lane; j < top_k; j += 32) weights[j] = weights[j] / denom * scale;
 }
 
@@ -94,7 +109,7 @@ __device__ __forceinline__ unsigned int order_key(float v) {
 }
 
 template <int PER>
-__device__ __forceinline__ void route_token_regs(const float* __restrict__ row, int n_parts, const float* __restrict__ bias,
+__device__ __forceinline__ void route_token_regs(const float* __restrict__ row, int part_stride, int n_parts, const float* __restrict__ bias,
                                                  int n_experts, int top_k, int scoring, float scale, float* wbuf,
                                                  int32_t* __restrict__ ids, float* __restrict__ weights,
                                                  int32_t* ids_copy) {
@@ -104,7 +119,7 @@ __device__ __forceinline__ void route_token_regs(const float* __restrict__ row, 
 #pragma unroll
   for (int q = 0; q < PER; ++q) {
     const int e = q * 32 + lane;
-    sv[q] = e < n_experts ? logit_of(row, e, n_experts, n_parts) : -INFINITY;
+    sv[q] = e < n_experts ? logit_of(row, e, part_stride, n_parts) : -INFINITY;
   }
   if (scoring == FTK_SCORE_SOFTMAX_OF_CHOSEN) {  // the bias joins the logit (see route_token)
     if (bias) {
@@ -173,28 +188,29 @@ __device__ __forceinline__ void route_token_regs(const float* __restrict__ row, 
     }
   }
   __syncwarp();
-  const float denom = scoring == FTK_SCORE_SIGMOID_RAW ? 1.f : scoring == FTK_SCORE_SIGMOID ? wsum + 1e-20f : wsum;  // (raw: the scores as they are)
+  const float denom = scoring == FTK_SCORE_SIGMOID_RAW ? 1.f : scoring == FTK_SCORE_SOFTMAX_OF_CHOSEN ? wsum : wsum + 1e-20f;  // (raw: the scores as they are)
   for (int j = lane; j < top_k; j += 32) weights[j] = wbuf[j] / denom * scale;
   __syncwarp();
 }
 
 // One token by one warp, in registers where the experts fit; `s` holds 2 * n_experts floats.
-__device__ __forceinline__ void route_one(const float* __restrict__ row, int n_parts, const float* __restrict__ bias, int n_experts,
+__device__ __forceinline__ void route_one(const float* __restrict__ row, int part_stride, int n_parts, const float* __restrict__ bias, int n_experts,
                                           int top_k, int scoring, float scale, float* s, int32_t* __restrict__ ids,
                                           float* __restrict__ weights, int32_t* ids_copy) {
   if (n_experts <= 128)
-    route_token_regs<4>(row, n_parts, bias, n_experts, top_k, scoring, scale, s, ids, weights, ids_copy);
+    route_token_regs<4>(row, part_stride, n_parts, bias, n_experts, top_k, scoring, scale, s, ids, weights, ids_copy);
   else if (n_experts <= 256)
-    route_token_regs<8>(row, n_parts, bias, n_experts, top_k, scoring, scale, s, ids, weights, ids_copy);
+    route_token_regs<8>(row, part_stride, n_parts, bias, n_experts, top_k, scoring, scale, s, ids, weights, ids_copy);
   else if (n_experts <= 512)
-    route_token_regs<16>(row, n_parts, bias, n_experts, top_k, scoring, scale, s, ids, weights, ids_copy);
+    route_token_regs<16>(row, part_stride, n_parts, bias, n_experts, top_k, scoring, scale, s, ids, weights, ids_copy);
   else
-    route_token(row, n_parts, bias, n_experts, top_k, scoring, scale, s, s + n_experts, ids, weights, ids_copy);
+    route_token(row, part_stride, n_parts, bias, n_experts, top_k, scoring, scale, s, s + n_experts, ids, weights, ids_copy);
 }
 
 __global__ void router_topk_kernel(const float* __restrict__ logits, int n_parts, const float* __restrict__ bias,
                                    int n_tokens, int n_experts, int top_k, int scoring, float scale,
-                                   int32_t* __restrict__ ids, float* __restrict__ weights) {
+                                   int32_t* __restrict__ ids, float* __restrict__ weights, int n_extra, int n_real,
+                                   float* __restrict__ aux) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ float sm[];
@@ -202,8 +218,13 @@ __global__ void router_topk_kernel(const float* __restrict__ logits, int n_parts
   const int t = blockIdx.x * kRouterWarps + warp;
   if (t >= n_tokens) return;
   float* s = sm + (size_t)warp * 2 * n_experts;  // unbiased scores
-  route_one(logits + (size_t)t * n_parts * n_experts, n_parts, bias, n_experts, top_k, scoring, scale, s,
-            ids + (size_t)t * top_k, weights + (size_t)t * top_k, nullptr);
+  const int stride = n_experts + n_extra;
+  const float* row = logits + (size_t)t * n_parts * stride;
+  route_one(row, stride, n_parts, bias, n_experts, top_k, scoring, scale, s, ids + (size_t)t * top_k,
+            weights + (size_t)t * top_k, nullptr);
+  if (aux)
+    token_aux(row, stride, n_parts, n_experts, n_extra, n_real, ids + (size_t)t * top_k, weights + (size_t)t * top_k, top_k,
+              aux + (size_t)t * 2);
 }
 
 // The whole routing of a small step in one launch: router logits (a float32 matrix-vector product
@@ -251,7 +272,8 @@ moe_route_kernel(const float* __restrict__ x, const float* __restrict__ w, const
                  int n_tokens, int hidden, int n_experts, int top_k, int scoring, float scale,
                  float* __restrict__ logits, int32_t* __restrict__ ids, float* __restrict__ weights,
                  int32_t* __restrict__ counts, int32_t* __restrict__ offsets, int32_t* __restrict__ routes,
-                 int32_t* __restrict__ pos, int do_sort) {
+                 int32_t* __restrict__ pos, int do_sort, int n_extra, int n_real, float* __restrict__ aux) {
+  const int n_rows = n_experts + n_extra;  // rows of the weight, logits of a token
   extern __shared__ float sm[];
   __shared__ float part[kRouteVals][kRouteWarps + 1];
   __shared__ bool last;
@@ -265,7 +287,7 @@ moe_route_kernel(const float* __restrict__ x, const float* __restrict__ w, const
   float4 w_first[kRouteExperts];
 #pragma unroll
   for (int j = 0; j < kRouteExperts; ++j)
-    w_first[j] = tid < h4 ? __ldg(w4 + (size_t)min(e0 + j, n_experts - 1) * h4 + tid) : make_float4(0.f, 0.f, 0.f, 0.f);
+    w_first[j] = tid < h4 ? __ldg(w4 + (size_t)min(e0 + j, n_rows - 1) * h4 + tid) : make_float4(0.f, 0.f, 0.f, 0.f);
   pdl_wait();
   // every block fetches the bias now, under the matrix product, so that the one that turns out to
   // be last does not wait for it
@@ -282,7 +304,7 @@ moe_route_kernel(const float* __restrict__ x, const float* __restrict__ w, const
       float4 wv[kRouteExperts], xv[kRouteTokens];
 #pragma unroll
       for (int j = 0; j < kRouteExperts; ++j)
-        wv[j] = i == tid ? w_first[j] : __ldg(w4 + (size_t)min(e0 + j, n_experts - 1) * h4 + i);
+        wv[j] = i == tid ? w_first[j] : __ldg(w4 + (size_t)min(e0 + j, n_rows - 1) * h4 + i);
 #pragma unroll
       for (int u = 0; u < kRouteTokens; ++u)  // (rows past the step's tokens are never stored: no load for them)
         xv[u] = u < nt ? __ldg(x4 + (size_t)(t0 + u) * h4 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -303,11 +325,11 @@ moe_route_kernel(const float* __restrict__ x, const float* __restrict__ w, const
     __syncthreads();
     if (tid < kRouteVals) {
       const int j = tid / kRouteTokens, u = tid % kRouteTokens;
-      if (u < nt && e0 + j < n_experts) {
+      if (u < nt && e0 + j < n_rows) {
         float v = part[tid][0];
 #pragma unroll
         for (int q = 1; q < kRouteWarps; ++q) v += part[tid][q];
-        logits[(size_t)(t0 + u) * n_experts + e0 + j] = v;
+        logits[(size_t)(t0 + u) * n_rows + e0 + j] = v;
       }
     }
     __syncthreads();
@@ -322,9 +344,14 @@ moe_route_kernel(const float* __restrict__ x, const float* __restrict__ w, const
   const int n_routes = n_tokens * top_k;
   int* sid = reinterpret_cast<int*>(sbias + n_experts);  // n_routes: the routes' experts
   float* s = sm + (size_t)warp * 2 * n_experts;
-  for (int t = warp; t < n_tokens; t += kRouteWarps)
-    route_one(logits + (size_t)t * n_experts, 1, bias ? sbias : nullptr, n_experts, top_k, scoring, scale, s,
-              ids + (size_t)t * top_k, weights + (size_t)t * top_k, do_sort ? sid + (size_t)t * top_k : nullptr);
+  for (int t = warp; t < n_tokens; t += kRouteWarps) {
+    const float* row = logits + (size_t)t * n_rows;
+    route_one(row, n_rows, 1, bias ? sbias : nullptr, n_experts, top_k, scoring, scale, s, ids + (size_t)t * top_k,
+              weights + (size_t)t * top_k, do_sort ? sid + (size_t)t * top_k : nullptr);
+    if (aux)
+      token_aux(row, n_rows, 1, n_experts, n_extra, n_real, ids + (size_t)t * top_k, weights + (size_t)t * top_k, top_k,
+                aux + (size_t)t * 2);
+  }
   if (!do_sort) {  // the caller's kernels take the routes in token order
     if (tid == 0) g_route_arrivals = 0;
     return;
@@ -341,9 +368,9 @@ moe_route_kernel(const float* __restrict__ x, const float* __restrict__ w, const
       before += (eq < e || (eq == e && q < r)) ? 1 : 0;
     }
     routes[before] = r;
-    pos[r] = before;
+    pos[r] = e < n_real ? before : -1;  // (an expert without tensors has no rows)
   }
-  for (int i = tid; i <= n_experts; i += blockDim.x) {
+  for (int i = tid; i <= n_real; i += blockDim.x) {
     int below = 0, same = 0;
     for (int q = 0; q < n_routes; ++q) {
       const int eq = sid[q];
@@ -351,7 +378,7 @@ moe_route_kernel(const float* __restrict__ x, const float* __restrict__ w, const
       same += eq == i ? 1 : 0;
     }
     offsets[i] = below;
-    if (i < n_experts) counts[i] = same;
+    if (i < n_real) counts[i] = same;
   }
   if (tid == 0) g_route_arrivals = 0;  // every block has arrived: ready for the next launch
 }
@@ -361,7 +388,9 @@ moe_route_kernel(const float* __restrict__ x, const float* __restrict__ w, const
 using namespace ftk;
 
 extern "C" int ftk_router_topk(const float* logits, int n_parts, const float* bias, int n_tokens, int n_experts, int top_k,
-                               int scoring, float scale, int32_t* ids, float* weights, void* stream) {
+                               int scoring, float scale, int32_t* ids, float* weights, int n_extra, int n_real, float* aux,
+                               void* stream) {
+  FTK_REQUIRE((n_extra == 0 || n_extra == 1) && n_real >= 0 && n_real <= n_experts, "router_topk: bad extra logits or expert counts");
   FTK_REQUIRE(n_parts >= 1 && n_parts <= 4, "router_topk: %d blocks of logits per token (1 to 4)", n_parts);
   FTK_REQUIRE(scoring >= FTK_SCORE_SIGMOID && scoring <= FTK_SCORE_SIGMOID_RAW, "router_topk: unknown scoring %d", scoring);
   FTK_REQUIRE(n_experts >= 1 && top_k >= 1 && top_k <= n_experts, "router_topk: top_k=%d of %d experts", top_k, n_experts);
@@ -374,7 +403,7 @@ extern "C" int ftk_router_topk(const float* logits, int n_parts, const float* bi
   const int blocks = (n_tokens + kRouterWarps - 1) / kRouterWarps;
   note_variant(n_parts > 1 ? "routing: expert choice from logits given in pieces" : "routing: expert choice from given logits");
   FTK_LAUNCH(router_topk_kernel, blocks, kRouterWarps * 32, smem, (cudaStream_t)stream, logits, n_parts, bias, n_tokens, n_experts, top_k,
-                                                                               scoring, scale, ids, weights);
+                                                                               scoring, scale, ids, weights, n_extra, n_real, aux);
   FTK_LAUNCH_CHECK("router_topk");
   return 0;
 }
@@ -391,7 +420,8 @@ extern "C" int ftk_moe_route_fits(int n_tokens, int hidden, int n_experts, int t
 extern "C" int ftk_moe_route(const float* x, const float* gate_w, const float* bias, int n_tokens, int hidden,
                              int n_experts, int top_k, int scoring, float scale, float* logits, int32_t* ids,
                              float* weights, int32_t* counts, int32_t* offsets, int32_t* routes, int32_t* pos,
-                             int do_sort, void* stream) {
+                             int do_sort, int n_extra, int n_real, float* aux, void* stream) {
+  FTK_REQUIRE((n_extra == 0 || n_extra == 1) && n_real >= 0 && n_real <= n_experts, "moe_route: bad extra logits or expert counts");
   FTK_REQUIRE(scoring >= FTK_SCORE_SIGMOID && scoring <= FTK_SCORE_SIGMOID_RAW, "moe_route: unknown scoring %d", scoring);
   FTK_REQUIRE(ftk_moe_route_fits(n_tokens, hidden, n_experts, top_k),
               "moe_route: %d tokens, width %d, %d experts, top %d do not fit the one-launch routing (at most 32 tokens, "
@@ -402,11 +432,11 @@ extern "C" int ftk_moe_route(const float* x, const float* gate_w, const float* b
   FTK_REQUIRE(((uintptr_t)x | (uintptr_t)gate_w) % 16 == 0, "moe_route: x and the gate weight must be 16-byte aligned");
   const size_t smem = route_smem(n_tokens, n_experts, top_k);
   if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  const int blocks = (n_experts + kRouteExperts - 1) / kRouteExperts;
+  const int blocks = (n_experts + n_extra + kRouteExperts - 1) / kRouteExperts;
   note_variant(do_sort ? "routing: product, choice and sort in one launch" : "routing: product and choice in one launch");
   FTK_LAUNCH(moe_route_kernel, blocks, kRouteWarps * 32, smem, (cudaStream_t)stream, 
       x, gate_w, bias, n_tokens, hidden, n_experts, top_k, scoring, scale, logits, ids, weights, counts, offsets, routes, pos,
-      do_sort);
+      do_sort, n_extra, n_real, aux);
   FTK_LAUNCH_CHECK("moe_route");
   return 0;
 }

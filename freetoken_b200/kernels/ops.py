@@ -31,6 +31,10 @@ head_gate, table_route, scale  no counterpart: per-head output gate, experts by 
                        token ids, logit scale
 hyper_step, norm_mean  no counterpart: several residual streams (write, read, norm in one pass), the
                        mean of normed branch outputs
+stream_step            no counterpart: gate, group norm, sum into the 32-bit stream, its group norm and (one
+                       token per request) the short convolution behind it, in one pass
+conv_rope_store,       no counterpart: convolution, rotation and cache write of several softmax maps a head;
+diff_heads             the difference of two maps' outputs, normed
 conv_act, ssm_gates,   no counterpart: convolution of projected rows with a per-request state, step sizes
 ssm_output, delta_scan and decays, gated group norm of a state-space layer; the gated delta rule
 =====================  ==========================================================
@@ -80,7 +84,28 @@ class _StreamNorm(ctypes.Structure):
 
 class _AttnExtras(ctypes.Structure):
     _fields_ = [("dist_bias", _vp), ("dist_len", _i), ("kv_split", _i), ("has_sink", _i), ("sink_logit", _f),
-                ("sink_heads", _vp)]
+                ("sink_heads", _vp), ("softcap", _f)]
+
+
+class _StreamStep(ctypes.Structure):
+    _fields_ = [
+        ("residual", _vp), ("vec", _vp), ("x", _vp), ("route_pos", _vp), ("top_k", _i), ("n_routes", _i), ("aux", _vp),
+        ("passed", _vp), ("shared", _vp), ("gate", _vp), ("gate_bias", _vp), ("post_w", _vp), ("post_eps", _f),
+        ("raw_out", _vp), ("raw_stride", ctypes.c_longlong), ("pre_w", _vp), ("pre_eps", _f), ("out", _vp),
+        ("norm_f32", _vp), ("conv_w", _vp), ("taps", _i), ("state", _vp), ("n_slots", _i), ("state_slots", _vp),
+        ("seg_info", _vp), ("conv_out", _vp), ("conv_out_f32", _vp), ("rows", _vp), ("n_rows", _i), ("hidden", _i),
+        ("groups", _i), ("dtype", _i),
+    ]
+
+
+class _ConvRope(ctypes.Structure):
+    _fields_ = [
+        ("x", _vp), ("x_stride", ctypes.c_longlong), ("dtype", _i), ("conv_w", _vp), ("taps", _i), ("state", _vp),
+        ("n_slots", _i), ("state_slots", _vp), ("seg_info", _vp), ("n_segs", _i), ("n_tokens", _i), ("n_heads", _i),
+        ("n_kv_heads", _i), ("maps", _i), ("dim", _i), ("vdim", _i), ("n_rot", _i), ("interleaved", _i),
+        ("positions", _vp), ("table", _vp), ("max_pos", _i), ("q_out", _vp), ("k_slab", _vp), ("v_slab", _vp),
+        ("slot_map", _vp), ("page_size", _i), ("num_pages", _i), ("pad_dim", _i),
+    ]
 
 
 _SIGNATURES = {
@@ -111,10 +136,10 @@ _SIGNATURES = {
                                    _i, _i, _i, _i, _i, _i, _f, _vp, _i, _i, _vp],
     "ftk_sparse_select": [_vp, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp],
     "ftk_sparse_score_fits": [_i, _i, _i],
-    "ftk_router_topk": [_vp, _i, _vp, _i, _i, _i, _i, _f, _vp, _vp, _vp],
+    "ftk_router_topk": [_vp, _i, _vp, _i, _i, _i, _i, _f, _vp, _vp, _i, _i, _vp, _vp],
     "ftk_moe_permute": [_vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp],
     "ftk_moe_route_fits": [_i, _i, _i, _i],
-    "ftk_moe_route": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp],
+    "ftk_moe_route": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _vp],
     "ftk_small_linear_fits": [_i, _i, _i],
     "ftk_small_linear": [_vp, _vp, _vp, _i, _i, _i, _vp],
     "ftk_moe_small_fits": [_i, _i, _i, _i],
@@ -125,7 +150,10 @@ _SIGNATURES = {
     "ftk_moe_gemm1_gather_fits": [_i, _i, _i, _i],
     "ftk_moe_gemm1_act_gather": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _f, _vp, _vp],
     "ftk_moe_gemm2": [_vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp],
-    "ftk_moe_combine": [_vp, _i, _vp, _i, _i, _i, _vp, _vp, _vp],
+    "ftk_moe_combine": [_vp, _i, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp],
+    "ftk_stream_step": [ctypes.POINTER(_StreamStep), _vp],
+    "ftk_conv_rope_store": [ctypes.POINTER(_ConvRope), _vp],
+    "ftk_diff_heads": [_vp, _i, _i, _vp, _f, _f, _vp, _i, _i, _i, _vp],
     "ftk_act_and_mul": [_vp, _i, _i, _i, _i, _f, _f, _vp, _vp],
     "ftk_sample": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp],
     "ftk_cast": [_vp, _i, _vp, _i, ctypes.c_longlong, _vp],
@@ -438,7 +466,7 @@ def paged_attention(q: torch.Tensor, k_slab: torch.Tensor, v_slab: torch.Tensor,
                     part_ml: Optional[torch.Tensor], out: torch.Tensor, tile_rows: int, scale: float,
                     window: Optional[int], sel: Optional[torch.Tensor] = None, block_size: int = 0,
                     few_rows: bool = False, dist_bias: Optional[torch.Tensor] = None, kv_split: int = 1,
-                    sink: Any = None) -> None:
+                    sink: Any = None, softcap: Optional[float] = None) -> None:
     """Causal softmax attention of the step's queries over the paged keys and values.
 
     ``q, out [T, Hq, D]``; slabs ``[pages, Hkv, page_size, D]``; ``block_table [rows, width]``
@@ -471,7 +499,14 @@ def paged_attention(q: torch.Tensor, k_slab: torch.Tensor, v_slab: torch.Tensor,
     in the merge.  Not with block selection.  Of the tcgen05 kernels the one with 128-row tiles takes a window and a
     sink (its work list then starts every piece on a key tile: ``build_plan(..., window, key_tile=128)``), also with
     one slab for keys and values, and a sink together with a bias by distance.
+
+    ``softcap`` (positive, or None): scaled scores ``s`` become ``softcap * tanh(s / softcap)`` before the softmax.  Not with
+    block selection or a bias by distance; of the tcgen05 kernels the ones with one query tile a piece (128 rows, or at most
+    16) take it.
     """
+    softcap = 0.0 if softcap is None else float(softcap)
+    if softcap < 0 or (softcap and (sel is not None or dist_bias is not None)):
+        raise KernelError("paged_attention: a soft cap is positive, without block selection or a distance bias")
     T, Hq, D = q.shape
     pages, Hkv, P, D2 = k_slab.shape
     if D2 != D or v_slab.shape != k_slab.shape or Hq % Hkv:
@@ -497,7 +532,9 @@ def paged_attention(q: torch.Tensor, k_slab: torch.Tensor, v_slab: torch.Tensor,
         # bfloat16 steps on the tcgen05 kernels: one query tile per CTA, a pair of them, or tiles of a few rows
         if sel is not None or q.dtype != torch.bfloat16:
             raise KernelError("paged_attention: the tcgen05 kernels take bfloat16 without block selection")
-        if window or sink is not None or dist_bias is not None:
+        if window or sink is not None or dist_bias is not None or softcap:
+            if softcap and tile_rows == 256:
+                raise KernelError("paged_attention: of the tcgen05 kernels the ones with one query tile a piece take a soft cap")
             # the form with one 128-row query tile a piece takes a window, a sink and a bias by distance (a bias not
             # together with a window); the form for tiles of at most 16 rows takes the bias alone
             if (window or sink is not None) and (tile_rows != 128 or few_rows):
@@ -506,8 +543,8 @@ def paged_attention(q: torch.Tensor, k_slab: torch.Tensor, v_slab: torch.Tensor,
                 raise KernelError("paged_attention: of the tcgen05 kernels the ones with one query tile a piece take a "
                                   "distance bias [Hq, L] (no window)")
             ex = _AttnExtras(_dev(dist_bias, "dist_bias", torch.float32), dist_bias.shape[1] if dist_bias is not None else 0,
-                             1, 0 if sink is None else 1, 0.0 if sink is None else float(sink), sink_heads)
-            what = "distance bias" if dist_bias is not None else "window or sink"
+                             1, 0 if sink is None else 1, 0.0 if sink is None else float(sink), sink_heads, softcap)
+            what = "soft cap" if softcap else "distance bias" if dist_bias is not None else "window or sink"
             _check(_lib().ftk_paged_attention_tc_ex(
                 _dev(q, "q"), _dev(k_slab, "k_slab"), _dev(v_slab, "v_slab"),
                 _dev(block_table, "block_table", torch.int32), block_table.shape[1],
@@ -544,11 +581,11 @@ def paged_attention(q: torch.Tensor, k_slab: torch.Tensor, v_slab: torch.Tensor,
             _dev(sel, "sel", torch.int32), sel.shape[2], int(block_size), _stream()),
             "paged_attention (block-sparse)", 2 if n_slots else 1)
         return
-    if dist_bias is not None or kv_split > 1 or sink is not None:
+    if dist_bias is not None or kv_split > 1 or sink is not None or softcap:
         if dist_bias is not None and (dist_bias.dim() != 2 or dist_bias.shape[0] != Hq or dist_bias.shape[1] < 1):
             raise KernelError("paged_attention: dist_bias must be [Hq, L]")
         ex = _AttnExtras(_dev(dist_bias, "dist_bias", torch.float32), dist_bias.shape[1] if dist_bias is not None else 0,
-                         kv_split, 0 if sink is None else 1, 0.0 if sink is None else float(sink), sink_heads)
+                         kv_split, 0 if sink is None else 1, 0.0 if sink is None else float(sink), sink_heads, softcap)
         _check(_lib().ftk_paged_attention_ex(
             _dev(q, "q"), _dev(k_slab, "k_slab"), _dev(v_slab, "v_slab"), _code(q, "q"),
             _dev(block_table, "block_table", torch.int32), block_table.shape[1],
@@ -617,7 +654,8 @@ def sparse_select(iq: torch.Tensor, ik_slab: torch.Tensor, block_table: torch.Te
 
 # --------------------------------------------------------------------------- experts
 def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, scoring: str,
-                scale: float, ids: torch.Tensor, weights: torch.Tensor, n_parts: int = 1) -> None:
+                scale: float, ids: torch.Tensor, weights: torch.Tensor, n_parts: int = 1, n_extra: int = 0,
+                n_real: Optional[int] = None, aux: Optional[torch.Tensor] = None) -> None:
     """Expert choice from float32 router logits ``[T, E]``.
 
     sigmoid: ``s = sigmoid(l)``; choice by ``s + bias``; ``w = s[ids] / (sum + 1e-20) * scale``.
@@ -627,11 +665,18 @@ def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, 
 
     With ``n_parts > 1`` the logits come as ``[T, n_parts * E]``: a token's logit of expert ``e`` is the
     32-bit sum of ``logits[t, q * E + e]`` over the parts ``q`` in their order.
+
+    A token's logits (each part) may end in ``n_extra`` (0 or 1) values that belong to no expert.  ``aux [T, 2]`` receives
+    the sum of the token's weights that fell on ids from ``n_real`` on (experts without tensors; default: none) and the
+    sigmoid of the extra logit (1 without one).  A softmax router's weights are divided by their sum + 1e-20.
     """
     T, PE = logits.shape
     if n_parts < 1 or PE % n_parts or not logits.is_contiguous():
         raise KernelError("router_topk: logits must be contiguous [T, n_parts * E]")
-    E = PE // n_parts
+    E = PE // n_parts - n_extra
+    n_real = E if n_real is None else int(n_real)
+    if aux is not None and aux.shape != (T, 2):
+        raise KernelError("router_topk: aux must be [T, 2]")
     if ids.shape != (T, top_k) or weights.shape != (T, top_k):
         raise KernelError("router_topk: ids / weights must be [T, top_k]")
     if bias is not None and bias.shape != (E,):
@@ -639,7 +684,7 @@ def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, 
     _check(_lib().ftk_router_topk(_dev(logits, "logits", torch.float32), int(n_parts), _dev(bias, "bias", torch.float32),
                                   T, E, top_k, SCORE_CODES[scoring], float(scale),
                                   _dev(ids, "ids", torch.int32), _dev(weights, "weights", torch.float32),
-                                  _stream()), "router_topk")
+                                  int(n_extra), n_real, _dev(aux, "aux", torch.float32), _stream()), "router_topk")
 
 
 def moe_permute(topk_ids: torch.Tensor, n_experts: int, expert_counts: torch.Tensor,
@@ -744,18 +789,24 @@ def moe_route_fits(n_tokens: int, hidden: int, n_experts: int, top_k: int) -> bo
 def moe_route(x: torch.Tensor, gate_w: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, scoring: str,
               scale: float, logits: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
               expert_counts: Optional[torch.Tensor] = None, expert_offsets: Optional[torch.Tensor] = None,
-              sorted_routes: Optional[torch.Tensor] = None, route_pos: Optional[torch.Tensor] = None) -> None:
+              sorted_routes: Optional[torch.Tensor] = None, route_pos: Optional[torch.Tensor] = None, n_extra: int = 0,
+              n_real: Optional[int] = None, aux: Optional[torch.Tensor] = None) -> None:
     """``logits = x @ gate_w^T`` in float32, then :func:`router_topk` and :func:`moe_permute`, in one launch.
     Without the four outputs of the sort only ids and weights are made (the few-token expert kernels take
-    the routes in token order)."""
+    the routes in token order).  ``n_extra``, ``n_real`` and ``aux`` as in :func:`router_topk` (``gate_w`` and ``logits`` then
+    have ``n_extra`` more rows and columns); routes to ids from ``n_real`` on are sorted behind the others and get the
+    place -1, and the sort's outputs count ``n_real`` experts."""
     T, H = x.shape
-    E = gate_w.shape[0]
-    if gate_w.shape != (E, H) or logits.shape != (T, E) or ids.shape != (T, top_k) or weights.shape != (T, top_k):
+    E = gate_w.shape[0] - n_extra
+    n_real = E if n_real is None else int(n_real)
+    if aux is not None and aux.shape != (T, 2):
+        raise KernelError("moe_route: aux must be [T, 2]")
+    if gate_w.shape != (E + n_extra, H) or logits.shape != (T, E + n_extra) or ids.shape != (T, top_k) or weights.shape != (T, top_k):
         raise KernelError("moe_route: shapes do not agree")
     sort = expert_counts is not None
     if sort and (expert_offsets is None or sorted_routes is None or route_pos is None):
         raise KernelError("moe_route: give all four outputs of the sort, or none")
-    if sort and (expert_offsets.shape != (E + 1,) or expert_counts.shape != (E,) or sorted_routes.numel() != T * top_k
+    if sort and (expert_offsets.shape != (n_real + 1,) or expert_counts.shape != (n_real,) or sorted_routes.numel() != T * top_k
                  or route_pos.numel() != T * top_k):
         raise KernelError("moe_route: output shapes are wrong")
     if bias is not None and bias.shape != (E,):
@@ -767,7 +818,8 @@ def moe_route(x: torch.Tensor, gate_w: torch.Tensor, bias: Optional[torch.Tensor
                                 _dev(expert_counts, "expert_counts", torch.int32),
                                 _dev(expert_offsets, "expert_offsets", torch.int32),
                                 _dev(sorted_routes, "sorted_routes", torch.int32),
-                                _dev(route_pos, "route_pos", torch.int32), 1 if sort else 0, _stream()), "moe_route")
+                                _dev(route_pos, "route_pos", torch.int32), 1 if sort else 0, int(n_extra), n_real,
+                                _dev(aux, "aux", torch.float32), _stream()), "moe_route")
 
 
 def moe_small_fits(n_tokens: int, hidden: int, inter: int, top_k: int) -> bool:
@@ -870,16 +922,21 @@ def moe_gemm2(a: torch.Tensor, w2: torch.Tensor, expert_offsets: torch.Tensor,
 
 
 def moe_combine(y: torch.Tensor, route_pos: torch.Tensor, n_tokens: int, top_k: int,
-                shared: Optional[torch.Tensor], out: torch.Tensor) -> None:
-    """``out[t] = sum_j y[route_pos[t*k + j]]`` in route order, 32-bit sum, ``+ shared[t]``."""
+                shared: Optional[torch.Tensor], out: torch.Tensor, aux: Optional[torch.Tensor] = None,
+                passed: Optional[torch.Tensor] = None) -> None:
+    """``out[t] = sum_j y[route_pos[t*k + j]]`` in route order (negative places skipped), 32-bit sum, ``+ shared[t]``; with
+    ``aux [T, 2]`` (float32) ``+ aux[t, 0] passed[t] + aux[t, 1] shared[t]``."""
     R, H = y.shape
     if R != n_tokens * top_k or out.shape != (n_tokens, H) or out.dtype != y.dtype:
         raise KernelError("moe_combine: shapes or dtypes do not agree")
     if shared is not None and (shared.shape != out.shape or shared.dtype != y.dtype):
         raise KernelError("moe_combine: shared must match out")
+    if (aux is not None and aux.shape != (n_tokens, 2)) or (passed is not None and (
+            aux is None or passed.shape != out.shape or passed.dtype != y.dtype)):
+        raise KernelError("moe_combine: aux must be [tokens, 2], passed must match out")
     _check(_lib().ftk_moe_combine(_dev(y, "y"), _code(y, "y"), _dev(route_pos, "route_pos", torch.int32),
-                                  n_tokens, top_k, H, _dev(shared, "shared"), _dev(out, "out"),
-                                  _stream()), "moe_combine")
+                                  n_tokens, top_k, H, _dev(shared, "shared"), _dev(aux, "aux", torch.float32),
+                                  _dev(passed, "passed"), _dev(out, "out"), _stream()), "moe_combine")
 
 
 # --------------------------------------------------------------------------- sampling
@@ -1348,6 +1405,125 @@ def conv_act(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], act
         _dev(bias, "bias", torch.float32), taps, CONV_ACT_CODES[act], _dev(state, "state", torch.float32),
         state.shape[0] if state is not None else 0, _dev(state_slots, "state_slots", torch.int32),
         _dev(seg_info, "seg_info", torch.int32), n_segs, _dev(out, "out"), T, C, _stream()), "conv_act")
+
+
+# --------------------------------------------------------------------------- gated stream, softmax maps
+def stream_step(residual: torch.Tensor, groups: int = 1, vec: Optional[torch.Tensor] = None, x: Optional[torch.Tensor] = None,
+                routed: Optional[tuple] = None, gate: Optional[torch.Tensor] = None,
+                gate_bias: Optional[torch.Tensor] = None, post_weight: Optional[torch.Tensor] = None, post_eps: float = 0.0,
+                raw_out: Optional[torch.Tensor] = None, pre_weight: Optional[torch.Tensor] = None, pre_eps: float = 0.0,
+                out: Optional[torch.Tensor] = None, norm_f32: Optional[torch.Tensor] = None,
+                conv: Optional[tuple] = None, rows: Optional[torch.Tensor] = None, dtype: Optional[torch.dtype] = None) -> None:
+    """One pass over the rows of the 32-bit stream; every part is optional.
+
+    ``r += vec``; ``y`` = row ``t`` of ``x``, or, with ``routed = (route_pos, top_k, shared, aux, passed)``, the 32-bit sum
+    ``sum_j x[route_pos[t top_k + j]] + aux[t, 0] passed[t] + aux[t, 1] shared[t]`` (negative places skipped; ``shared``,
+    ``aux`` and ``passed`` may be None); ``y *= sigmoid(gate + gate_bias)``; ``r += groupnorm(y) post_weight``;
+    ``raw_out = r`` (rows of the engine's type, any row stride); ``out = groupnorm(r) pre_weight`` and the same unrounded
+    in ``norm_f32`` (float32, may be the stream itself).  ``groupnorm`` divides each of ``groups`` equal consecutive parts
+    of a row by its own ``sqrt(mean(part^2) + eps)``.
+
+    ``conv = (weight [H, taps], state, state_slots, seg_info, conv_out, conv_out_f32 or None)``, for steps of one token per
+    request: ``conv_out = h + sum_j weight[:, j] h(t - taps + 1 + j)`` of the normed values as ``out`` stores them, the
+    earlier ones from the request's slot of ``state [slots, taps - 1, H]`` (float32, oldest first), which moves on.
+
+    With ``rows`` only those rows are read and the stream stays as it is."""
+    T, H = residual.shape
+    n_rows = rows.shape[0] if rows is not None else T
+    like = next((t for t in (x, out, raw_out) if t is not None), None)
+    dtype = dtype if dtype is not None else like.dtype if like is not None else conv[4].dtype if conv else torch.float32
+    for name, t in (("vec", vec), ("post_weight", post_weight), ("pre_weight", pre_weight), ("gate_bias", gate_bias)):
+        if t is not None and t.shape != (H,):
+            raise KernelError(f"stream_step: {name} must be [{H}]")
+    for name, t in (("x", x), ("gate", gate), ("out", out), ("raw_out", raw_out)):
+        if t is not None and (t.dtype != dtype or t.shape[-1] != H):
+            raise KernelError(f"stream_step: {name} must hold rows of {H} elements of {dtype}")
+    for name, t in (("out", out), ("norm_f32", norm_f32)):
+        if t is not None and t.numel() != n_rows * H:
+            raise KernelError(f"stream_step: {name} must be [{n_rows}, {H}]")
+    if gate is not None and gate.numel() < T * H:
+        raise KernelError("stream_step: gate has fewer rows than the stream")
+    a = _StreamStep()
+    a.residual, a.vec = _dev(residual, "residual", torch.float32), _dev(vec, "vec", torch.float32)
+    a.x, a.gate, a.gate_bias = _dev(x, "x"), _dev(gate, "gate"), _dev(gate_bias, "gate_bias", torch.float32)
+    if routed is not None:
+        pos, top_k, shared, aux, passed = routed
+        if x is None or pos.numel() < T * top_k or (aux is not None and aux.shape != (T, 2)):
+            raise KernelError("stream_step: routes do not match the rows")
+        for t in (shared, passed):
+            if t is not None and (t.shape != (T, H) or t.dtype != dtype):
+                raise KernelError("stream_step: shared and passed rows must match the stream's")
+        a.route_pos, a.top_k, a.n_routes = _dev(pos, "route_pos", torch.int32), int(top_k), x.shape[0]
+        a.aux, a.passed, a.shared = _dev(aux, "aux", torch.float32), _dev(passed, "passed"), _dev(shared, "shared")
+    elif x is not None and x.numel() < T * H:
+        raise KernelError("stream_step: x has fewer rows than the stream")
+    a.post_w, a.post_eps = _dev(post_weight, "post_weight", torch.float32), float(post_eps)
+    a.pre_w, a.pre_eps = _dev(pre_weight, "pre_weight", torch.float32), float(pre_eps)
+    if raw_out is not None:
+        if raw_out.shape != (n_rows, H) or raw_out.stride(1) != 1 or not raw_out.is_cuda:
+            raise KernelError("stream_step: raw_out must be rows of adjacent elements on the device")
+        a.raw_out, a.raw_stride = raw_out.data_ptr(), raw_out.stride(0) if n_rows > 1 else H
+    a.out, a.norm_f32 = _dev(out, "out"), _dev(norm_f32, "norm_f32", torch.float32)
+    if conv is not None:
+        w, state, slots, seg_info, c_out, c_out_f32 = conv
+        taps = w.shape[1]
+        if rows is not None or w.shape[0] != H or c_out.shape != (T, H) or c_out.dtype != dtype or seg_info.numel() < 4 * T \
+                or (taps > 1 and (state is None or state.shape[1:] != (taps - 1, H) or slots.numel() < T)):
+            raise KernelError("stream_step: the convolution's tensors do not match the rows")
+        a.conv_w, a.taps = _dev(w, "conv weight", torch.float32), taps
+        a.state, a.n_slots = _dev(state, "state", torch.float32), state.shape[0] if state is not None else 0
+        a.state_slots, a.seg_info = _dev(slots, "state_slots", torch.int32), _dev(seg_info, "seg_info", torch.int32)
+        a.conv_out, a.conv_out_f32 = _dev(c_out, "conv_out"), _dev(c_out_f32, "conv_out_f32", torch.float32)
+    a.rows, a.n_rows, a.hidden, a.groups = _dev(rows, "rows", torch.int32), n_rows, H, int(groups)
+    a.dtype = F32 if dtype == torch.float32 else BF16
+    _check(_lib().ftk_stream_step(ctypes.byref(a), _stream()), "stream_step")
+
+
+def conv_rope_store(x: torch.Tensor, conv_w: torch.Tensor, state: Optional[torch.Tensor], state_slots: torch.Tensor,
+                    seg_info: torch.Tensor, n_segs: int, n_heads: int, n_kv_heads: int, maps: int, dim: int, vdim: int,
+                    n_rot: int, interleaved: bool, positions: torch.Tensor, rope_table: Optional[torch.Tensor],
+                    q_out: torch.Tensor, k_slab: torch.Tensor, v_slab: torch.Tensor, slot_map: torch.Tensor) -> None:
+    """Rows ``q | k | v`` of a projection (``x [T, (n_heads + n_kv_heads) maps dim + n_kv_heads vdim]``, heads of q and k as
+    their maps one after the other) through a causal convolution over time per channel (``conv_w [channels, taps]``, state
+    as in :func:`conv_act`), the rotation of the first ``n_rot`` dimensions of every map of q and k, and to their places:
+    ``q_out [T, n_heads maps, P]`` holds map ``m`` of a head in columns ``m dim`` and on of its row (zeros elsewhere),
+    ``k_slab [pages, n_kv_heads, page_size, P]`` the maps side by side, ``v_slab`` the values (zeros behind them)."""
+    T = x.shape[0]
+    C = (n_heads + n_kv_heads) * maps * dim + n_kv_heads * vdim
+    P = q_out.shape[2]
+    taps = conv_w.shape[1]
+    if x.shape != (T, C) or x.stride(1) != 1 or not x.is_cuda or conv_w.shape != (C, taps):
+        raise KernelError("conv_rope_store: x and conv_w must hold the q, k and v channels")
+    if q_out.shape != (T, n_heads * maps, P) or k_slab.shape != v_slab.shape or k_slab.shape[1] != n_kv_heads \
+            or k_slab.shape[3] != P or q_out.dtype != x.dtype or k_slab.dtype != x.dtype or v_slab.dtype != x.dtype:
+        raise KernelError("conv_rope_store: q_out / slab shapes or dtypes do not agree")
+    if taps > 1 and (state is None or state.shape[1:] != (taps - 1, C)):
+        raise KernelError("conv_rope_store: state must be [slots, taps - 1, channels]")
+    if n_rot and (rope_table is None or rope_table.shape[1] != n_rot):
+        raise KernelError("conv_rope_store: rope_table must be [max_pos, n_rot]")
+    if slot_map.shape[0] < T or positions.shape[0] < T:
+        raise KernelError("conv_rope_store: slot_map or positions shorter than the tokens")
+    a = _ConvRope()
+    a.x, a.x_stride, a.dtype = x.data_ptr(), x.stride(0) if T > 1 else C, _code(x, "x")
+    a.conv_w, a.taps = _dev(conv_w, "conv_w", torch.float32), taps
+    a.state, a.n_slots = _dev(state, "state", torch.float32), state.shape[0] if state is not None else 0
+    a.state_slots, a.seg_info = _dev(state_slots, "state_slots", torch.int32), _dev(seg_info, "seg_info", torch.int32)
+    a.n_segs, a.n_tokens, a.n_heads, a.n_kv_heads, a.maps, a.dim, a.vdim = n_segs, T, n_heads, n_kv_heads, maps, dim, vdim
+    a.n_rot, a.interleaved, a.positions = n_rot, 1 if interleaved else 0, _dev(positions, "positions", torch.int32)
+    a.table, a.max_pos = _dev(rope_table, "rope_table", torch.float32), rope_table.shape[0] if rope_table is not None else 0
+    a.q_out, a.k_slab, a.v_slab = _dev(q_out, "q_out"), _dev(k_slab, "k_slab"), _dev(v_slab, "v_slab")
+    a.slot_map, a.page_size, a.num_pages, a.pad_dim = _dev(slot_map, "slot_map", torch.int32), k_slab.shape[2], k_slab.shape[0], P
+    _check(_lib().ftk_conv_rope_store(ctypes.byref(a), _stream()), "conv_rope_store")
+
+
+def diff_heads(o: torch.Tensor, lam: torch.Tensor, eps: float, scale: float, out: torch.Tensor) -> None:
+    """``out[t, h] = unit(o[t, 2 h, :vdim] - lam o[t, 2 h + 1, :vdim]) scale``: the second softmax map's output taken off the
+    first one's, divided by its root mean square over the head.  ``o [T, 2 H, P]``, ``lam`` one float32, ``out [T, H, vdim]``."""
+    T, H, Dv = out.shape
+    if o.shape[:2] != (T, 2 * H) or o.shape[2] < Dv or o.dtype != out.dtype or lam.numel() != 1:
+        raise KernelError("diff_heads: shapes or dtypes do not agree")
+    _check(_lib().ftk_diff_heads(_dev(o, "o"), o.shape[2], _code(o, "o"), _dev(lam, "lam", torch.float32), float(eps),
+                                 float(scale), _dev(out, "out"), T, H, Dv, _stream()), "diff_heads")
 
 
 # --------------------------------------------------------------------------- state space, delta rule

@@ -23,7 +23,7 @@ import torch
 from ..config.spec import ModelSpec, ParamSpec, PartSpec
 from ..errors import ConfigError
 from ..parts import BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, BuildEnv, Part, StepState
-from ..parts.base import NormedSum, StreamSum, as_rows, nvtx_range
+from ..parts.base import GatedSum, NormedSum, StreamSum, as_rows, nvtx_range
 
 
 def _walk(prefix: str, part: Part, out: Dict[str, Tuple[Part, str, ParamSpec]]) -> None:
@@ -55,6 +55,10 @@ class Model:
         if spec.pass_vectors is not None:
             self.pass_vectors = EMBEDDINGS.build(PartSpec(spec.pass_vectors.kind,
                                                           {"hidden": self.hidden, **spec.pass_vectors.params}), env)
+        self.pass_input = None
+        if spec.pass_input is not None:
+            self.pass_input = EMBEDDINGS.build(PartSpec(spec.pass_input.kind,
+                                                        {"hidden": self.hidden, **spec.pass_input.params}), env)
         self._index: Dict[str, Tuple[Part, str, ParamSpec]] = {}
         _walk(spec.embedding_name, self.embedding, self._index)
         _walk(spec.head_name, self.head, self._index)
@@ -63,6 +67,8 @@ class Model:
         _walk(spec.final_norm_name, self.final_norm, self._index)
         if self.pass_vectors is not None:
             _walk(spec.pass_vectors_name, self.pass_vectors, self._index)
+        if self.pass_input is not None:
+            _walk(spec.pass_input_name, self.pass_input, self._index)
 
     # ------------------------------------------------------------------ tensors
     def param_specs(self) -> Dict[str, ParamSpec]:
@@ -133,7 +139,7 @@ class Model:
             for c in p.children().values():
                 visit(c)
 
-        for p in (self.embedding, *self.blocks, self.final_norm, self.head, self.pass_vectors):
+        for p in (self.embedding, *self.blocks, self.final_norm, self.head, self.pass_vectors, self.pass_input):
             if p is not None:
                 visit(p)
         for p in self.env.shared.values():
@@ -164,12 +170,17 @@ class Model:
         ws, dt, cap = env.workspace, env.dtype, env.max_step_tokens
         residual = ws.get("model.residual", (T, self.hidden), torch.float32, (cap, self.hidden))
         self.embedding.forward(step.token_ids, residual)
+        if self.pass_input is not None:
+            self.pass_input.keep(residual)
         x = None
         for i, e in enumerate(self.spec.schedule):
+            if e.mix_embedding:
+                self.pass_input.mix(x, residual)
+                x = None
             if e.add_embedding or e.add_pass_vector is not None:
                 # fed into the stream with whatever the layer before left to be added: the entry's first norm
                 # (or, for a norm that cannot, one launch of its own) takes all of it in one 32-bit sum
-                if isinstance(x, NormedSum):  # it joins the stream through a norm of its own: add it now
+                if isinstance(x, (NormedSum, GatedSum)):  # it joins the stream through a norm of its own: add it now
                     x.fold(residual)
                     x = None
                 x = StreamSum.of(x) if x is not None else StreamSum()

@@ -178,17 +178,30 @@ class Part:
 class RouteSum:
     """A feed-forward output that is still a sum to be taken: row ``t`` is
     ``sum_j y[pos[t * top_k + j]] (+ shared[t])``.  A norm with ``takes_route_sum`` adds it to the
-    residual without the sum's trip through memory; for any other consumer :func:`as_rows` takes it."""
+    residual without the sum's trip through memory; for any other consumer :func:`as_rows` takes it.
+
+    With ``aux [T, 2]`` the row also has ``aux[t, 0] passed[t]`` (experts that hand the token's input back) and the shared
+    part counts ``aux[t, 1]`` times; negative places have no row.  Only a :class:`GatedSum` keeps those terms to itself;
+    for every other consumer :meth:`plain` takes the whole sum first."""
 
     def __init__(self, y: torch.Tensor, pos: torch.Tensor, top_k: int, shared: Optional[torch.Tensor],
-                 n_tokens: int, out: torch.Tensor):
+                 n_tokens: int, out: torch.Tensor, aux: Optional[torch.Tensor] = None,
+                 passed: Optional[torch.Tensor] = None):
         self.y, self.pos, self.top_k, self.shared, self.n_tokens, self.out = y, pos, top_k, shared, n_tokens, out
+        self.aux, self.passed = aux, passed
 
     def rows(self) -> torch.Tensor:
         from ..kernels import ops
 
-        ops.moe_combine(self.y, self.pos, self.n_tokens, self.top_k, self.shared, self.out)
+        if self.aux is None:
+            ops.moe_combine(self.y, self.pos, self.n_tokens, self.top_k, self.shared, self.out)
+        else:
+            ops.moe_combine(self.y, self.pos, self.n_tokens, self.top_k, self.shared, self.out, aux=self.aux, passed=self.passed)
         return self.out
+
+    def plain(self) -> Any:
+        """Itself, or its rows where it has terms beside the routes' and the plain shared part."""
+        return self if self.aux is None else self.rows()
 
 
 class StreamSum:
@@ -218,6 +231,8 @@ class StreamSum:
     def add(self, x: Any) -> "StreamSum":
         if x is None:
             return self
+        if isinstance(x, RouteSum):
+            x = x.plain()
         if isinstance(x, RouteSum):
             if self.routes is not None:
                 self.dense.append(self.routes.rows())
@@ -281,15 +296,41 @@ class NormedSum:
 
     def kernel_args(self):
         """``(rows, routed)`` as ``ops.postnorm_add_norm`` takes them."""
-        if isinstance(self.x, RouteSum):
-            return self.x.y, (self.x.pos, self.x.top_k, self.x.shared)
-        return self.x, None
+        x = self.x.plain() if isinstance(self.x, RouteSum) else self.x
+        if isinstance(x, RouteSum):
+            return x.y, (x.pos, x.top_k, x.shared)
+        return x, None
 
     def fold(self, residual: torch.Tensor) -> None:
         from ..kernels import ops
 
         rows, routed = self.kernel_args()
         ops.postnorm_add_norm(rows, routed, self.norm.params["weight"], self.norm.eps, self.norm.gemma, residual)
+
+
+class GatedSum:
+    """A sub-layer output that joins the stream through an element-wise gate and a norm over groups of channels:
+    ``groupnorm(x * sigmoid(gate + gate_bias)) * weight`` is still to be added.  ``x`` is a tensor or a :class:`RouteSum`
+    (its further terms included), ``weight`` holds whatever factor the result has.  A norm with ``takes_gated_sum`` adds
+    it in the pass that norms the stream; for any other consumer :meth:`fold` adds it first."""
+
+    def __init__(self, x: Any, weight: torch.Tensor, eps: float, groups: int, gate: Optional[torch.Tensor] = None,
+                 gate_bias: Optional[torch.Tensor] = None):
+        self.x, self.weight, self.eps, self.groups, self.gate, self.gate_bias = x, weight, eps, groups, gate, gate_bias
+
+    def kernel_args(self) -> Dict[str, Any]:
+        """Keyword arguments of ``ops.stream_step``."""
+        x, routed = self.x, None
+        if isinstance(x, RouteSum):
+            x, routed = self.x.y, (self.x.pos, self.x.top_k, self.x.shared, self.x.aux, self.x.passed)
+        return dict(x=x, routed=routed, gate=self.gate, gate_bias=self.gate_bias, post_weight=self.weight,
+                    post_eps=self.eps, groups=self.groups)
+
+    def fold(self, residual: torch.Tensor, raw_out: Optional[torch.Tensor] = None) -> None:
+        """Add it to ``residual`` now; ``raw_out`` also receives the stream, rounded to the engine's type."""
+        from ..kernels import ops
+
+        ops.stream_step(residual, raw_out=raw_out, **self.kernel_args())
 
 
 class HyperSum:
@@ -317,6 +358,11 @@ def as_rows(x: Any, consumer: Any = None, residual: Optional[torch.Tensor] = Non
             raise ConfigError("a HyperSum needs the stream that takes the sum of its streams")
         x.fold(residual)
         return None
+    if isinstance(x, GatedSum) and not getattr(consumer, "takes_gated_sum", False):
+        if residual is None:
+            raise ConfigError("a GatedSum needs the stream to be added to")
+        x.fold(residual)
+        return None
     if isinstance(x, NormedSum) and not getattr(consumer, "takes_normed_sum", False):
         if residual is None:
             raise ConfigError("a NormedSum needs the stream to be added to")
@@ -329,6 +375,8 @@ def as_rows(x: Any, consumer: Any = None, residual: Optional[torch.Tensor] = Non
         return None
     if isinstance(x, RouteSum) and not getattr(consumer, "takes_route_sum", False):
         return x.rows()
+    if isinstance(x, RouteSum):
+        return x.plain()
     return x
 
 
@@ -336,6 +384,7 @@ class Norm(Part):
     takes_route_sum: bool = False  # add_forward accepts a RouteSum as x
     takes_stream_sum: bool = False  # add_forward accepts a StreamSum as x
     takes_normed_sum: bool = False  # add_forward accepts a NormedSum as x
+    takes_gated_sum: bool = False  # add_forward accepts a GatedSum as x
 
     def forward(self, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
         """``out = norm(x)`` row by row."""

@@ -14,6 +14,12 @@ feed-forward kind ``none``.
 ``r += N_2b(ffn(N_2(r)))``.  The norm behind a sub-layer, the sum into the 32-bit stream and the norm in
 front of the next sub-layer are one kernel: a sub-layer's output travels on as a :class:`NormedSum`.
 
+``gated_sandwich_residual``: ``sandwich_residual`` with norms over groups of channels, in which a sub-layer reads its normed
+input ``h`` through a short causal convolution, ``h + conv(h)``, and its result passes an element-wise gate made from ``h``
+before its own norm: ``r += m N_1b(sigmoid(W h + b) * mixer(h + conv1(h)))`` with ``h = N_1(r)`` (``m`` one number), and the
+feed-forward alike.  Gate, norm, sum, the next norm and (one token per request) the next convolution are one kernel: a
+sub-layer's output travels on as a :class:`GatedSum`.  The convolutions' last inputs are per-request state of the block.
+
 ``conv_postnorm_residual``: the sub-layers read the stream itself through a short causal convolution over time
 and are normed on their way out only, ``r += ls1 * g1 * unit(mixer(r + conv1(r)))``, then
 ``r += ls2 * g2 * unit(ffn(r + conv2(r)))`` (``unit`` divides a row by its root mean square, ``g`` is one number,
@@ -39,7 +45,7 @@ import torch
 from ..config.spec import ParamSpec, PartSpec, StateNeed
 from ..errors import ConfigError
 from ..kernels import ops
-from .base import (BLOCKS, FEED_FORWARDS, NORMS, Block, BuildEnv, FeedForward, HyperSum, Mixer, NormedSum, Part, RouteSum, StepState,
+from .base import (BLOCKS, FEED_FORWARDS, NORMS, Block, BuildEnv, FeedForward, GatedSum, HyperSum, Mixer, NormedSum, Part, RouteSum, StepState,
                    StreamSum, as_rows, nvtx_range)
 
 
@@ -174,6 +180,122 @@ class SandwichResidualBlock(Block):
         with nvtx_range(f"feed-forward {self.ffn.kind}"):
             f = lazy(h2, step, h_f32=h32) if lazy is not None else self.ffn.forward(h2, step, h_f32=h32)
         return NormedSum(f, self.ffn_out)
+
+
+@BLOCKS.register("gated_sandwich_residual")
+class GatedSandwichResidualBlock(Block):
+    """params: ``hidden``, ``groups`` (of the norms), ``eps``, ``taps`` (of the input convolutions, 1 to 16), ``mult`` (the factor
+    on a sub-layer's normed result), ``init_std``.
+
+    Tensors: ``norm1``, ``norm1b``, ``norm2``, ``norm2b`` ``[hidden]``, ``canon1``, ``canon2`` ``[hidden, taps]``, ``rg1``, ``rg2``
+    ``[hidden, hidden]`` and their biases ``rg1.b``, ``rg2.b``; a layer without feed-forward has none of the second ones."""
+
+    graph_safe = False  # the convolutions' state moves on with every run of a step
+    graph_recordable = True
+
+    def __init__(self, spec: PartSpec, env: BuildEnv, mixer: Mixer, ffn: FeedForward,
+                 mixer_name: str, ffn_name: str):
+        super().__init__(spec, env, mixer, ffn, mixer_name, ffn_name)
+        self.hidden = int(spec["hidden"])
+        self.groups = int(spec.get("groups", 1))
+        self.eps = float(spec["eps"])
+        self.taps = int(spec.get("taps", 1))
+        self.mult = float(spec.get("mult", 1.0))
+        self.has_ffn = not isinstance(ffn, NoFeedForward)
+        if self.groups < 1 or self.hidden % self.groups:
+            raise ConfigError(f"gated_sandwich_residual: {self.hidden} channels do not divide into {self.groups} groups")
+        if not 1 <= self.taps <= 16:
+            raise ConfigError(f"gated_sandwich_residual: {self.taps} taps (1 to 16 taken)")
+        self._post: Dict[str, torch.Tensor] = {}
+        self._taps_and_input: Dict[str, torch.Tensor] = {}
+
+    def children(self) -> Dict[str, Part]:
+        out = {self.mixer_name: self.mixer}
+        if self.has_ffn:
+            out[self.ffn_name] = self.ffn
+        return out
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        std = self.spec.get("init_std")
+        f32 = dict(dtype="float32", store="bfloat16")
+        out: Dict[str, ParamSpec] = {}
+        for n in ("1", "2") if self.has_ffn else ("1",):
+            for b in ("", "b"):
+                out[f"norm{n}{b}"] = ParamSpec((self.hidden,), init=("normal", 1.0, 0.2 if std else 0.02), **f32)
+            out["canon" + n] = ParamSpec((self.hidden, self.taps), init=("normal", 0.0, 0.3 if std else 0.02), **f32)
+            out["rg" + n] = ParamSpec((self.hidden, self.hidden), init=("normal", 0.0, float(std) if std else 0.02))
+            out[f"rg{n}.b"] = ParamSpec((self.hidden,), init=("normal", 0.0, 0.5 if std else 0.02), **f32)
+        return out
+
+    def bind(self, tensors) -> None:
+        super().bind(tensors)
+        for n in ("1", "2") if self.has_ffn else ("1",):
+            self._post[n] = (self.params[f"norm{n}b"] * self.mult).contiguous()  # the result's factor joins its norm's weight
+            # h + conv(h) as one convolution: the last tap belongs to the row itself
+            w = self.params["canon" + n].clone()
+            w[:, -1] += 1.0
+            self._taps_and_input[n] = w.contiguous()
+
+    def state_need(self):
+        """The block's own per-request state: each convolution's last ``taps - 1`` inputs, 32-bit."""
+        if self.taps == 1:
+            return None
+        names = ("conv1", "conv2") if self.has_ffn else ("conv1",)
+        return StateNeed(tuple((n, (self.taps - 1, self.hidden), "float32") for n in names))
+
+    def workspace_bytes(self, n_tokens: int) -> int:
+        item = 4 if self.env.dtype == torch.float32 else 2
+        return n_tokens * self.hidden * (6 * item + 4)
+
+    def _enter(self, n: str, x, residual: torch.Tensor, step: StepState, wants_f32: bool):
+        """Add what is pending to the stream, norm it, convolve; the gate's logits from the normed rows.
+        Returns ``(sub-layer input, its 32-bit copy or None, gate logits)``."""
+        T = residual.shape[0]
+        ws, dt, cap = self.env.workspace, self.env.dtype, self.env.max_step_tokens
+        rows = lambda name, dtype=dt: ws.get(name, (T, self.hidden), dtype, (cap, self.hidden))  # noqa: E731
+        args: Dict[str, Any] = dict(groups=self.groups)
+        if isinstance(x, GatedSum) and x.groups == self.groups:
+            args = x.kernel_args()
+        elif isinstance(x, StreamSum) and not x.dense and x.routes is None and x.table is None:
+            args["vec"] = x.vec  # (a vector for every token: what a pass of a repeated range of layers adds)
+        elif x is not None:
+            x = as_rows(x, None, residual)
+            if x is not None:
+                StreamSum.of(x).fold(residual)
+        state = step.block_states.get(step.entry) if self.taps > 1 else None
+        if self.taps > 1 and state is None:
+            raise ConfigError("gated_sandwich_residual: the engine gave the block no state")
+        slots = state.tensors["conv" + n] if state is not None else None
+        h, u = rows("block.h"), rows(f"block.u{n}")
+        u32 = None
+        norm = dict(pre_weight=self.params["norm" + n], pre_eps=self.eps, out=h)
+        if step.decode_only:
+            u32 = rows("block.u_f32", torch.float32) if wants_f32 and dt != torch.float32 else None
+            ops.stream_step(residual, conv=(self.params["canon" + n], slots, step.state_slots, step.seg_info, u, u32),
+                            **norm, **args)
+        else:
+            ops.stream_step(residual, **norm, **args)
+            ops.conv_act(h, self._taps_and_input[n], None, None, slots, step.state_slots, step.seg_info,
+                         len(step.segments), u)
+        g = rows(f"block.gate{n}")
+        ops.linear(h, self.params["rg" + n], g)
+        return u, u32, g
+
+    def _leave(self, n: str, y, g: torch.Tensor) -> GatedSum:
+        return GatedSum(y, self._post[n], self.eps, self.groups, g, self.params[f"rg{n}.b"])
+
+    def forward(self, x, residual: torch.Tensor, step: StepState, cache: Any, writes_cache: bool):
+        T = residual.shape[0]
+        u, _, g = self._enter("1", x, residual, step, False)
+        with nvtx_range(f"mixer {self.mixer.kind}"):
+            a = self._leave("1", self.mixer.forward(u, step, cache, writes_cache), g)
+        if not self.has_ffn:
+            return a
+        u, u32, g = self._enter("2", a, residual, step, self.ffn.f32_input_needed(T))
+        lazy = getattr(self.ffn, "forward_lazy", None)
+        with nvtx_range(f"feed-forward {self.ffn.kind}"):
+            f = lazy(u, step, h_f32=u32) if lazy is not None else self.ffn.forward(u, step, h_f32=u32)
+        return self._leave("2", f, g)
 
 
 @BLOCKS.register("conv_postnorm_residual")

@@ -17,20 +17,21 @@ are other kinds in the same registries; the model asks for them by ``spec.embedd
 
 from __future__ import annotations
 
-from typing import Dict, Optional
+from typing import Any, Dict, Optional
 
 import torch
 
 from ..config.spec import ParamSpec, PartSpec
 from ..errors import ConfigError
 from ..kernels import ops
-from .base import EMBEDDINGS, HEADS, BuildEnv, Embedding, Head
+from .base import EMBEDDINGS, HEADS, NORMS, BuildEnv, Embedding, GatedSum, Head, Part, as_rows
 
 
 @EMBEDDINGS.register("token_embedding")
 class TokenEmbedding(Embedding):
     """params: ``vocab``, ``hidden``, ``init_std`` (spread of random weights, 0.02), ``scale`` (1.0: the rows
-    are multiplied by it in 32 bits as they enter the stream)."""
+    are multiplied by it in 32 bits as they enter the stream), ``norm`` (None, or the PartSpec of an RMS norm that the
+    rows pass in 32 bits, with a weight under ``norm``)."""
 
     def __init__(self, spec: PartSpec, env: BuildEnv):
         super().__init__(spec, env)
@@ -38,14 +39,20 @@ class TokenEmbedding(Embedding):
         self.hidden = int(spec["hidden"])
         self.init_std = float(spec.get("init_std", 0.02))
         self.scale = float(spec.get("scale", 1.0))
+        self.norm = NORMS.build(spec["norm"], env) if spec.get("norm") is not None else None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
         return {"weight": ParamSpec((self.vocab, self.hidden), init=("normal", 0.0, self.init_std))}
+
+    def children(self) -> Dict[str, Part]:
+        return {"norm": self.norm} if self.norm is not None else {}
 
     def forward(self, token_ids: torch.Tensor, residual: torch.Tensor) -> None:
         ops.embedding_gather(self.params["weight"], token_ids, residual)
         if self.scale != 1.0:
             ops.scale_(residual, self.scale)
+        if self.norm is not None:
+            self.norm.norm_stream(residual)
 
     def table(self) -> torch.Tensor:
         return self.params["weight"]
@@ -112,3 +119,42 @@ class PassVectors(Embedding):
 
     def table(self) -> torch.Tensor:
         return self.params[self.local_name]
+
+
+@EMBEDDINGS.register("stream_mix")
+class StreamMix(Embedding):
+    """What a repeated range of layers reads at the start of a pass: ``r <- W [r ; x0]`` with the stream ``r`` and the
+    embedding output ``x0`` (``weight [hidden, 2 hidden]``, the stream's columns first).  The product's operands are of the
+    engine's type, its 32-bit sums are the new stream."""
+
+    def __init__(self, spec: PartSpec, env: BuildEnv):
+        super().__init__(spec, env)
+        self.hidden = int(spec["hidden"])
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        std = self.spec.get("init_std")
+        return {"weight": ParamSpec((self.hidden, 2 * self.hidden),
+                                    init=("normal", 0.0, float(std) if std else 0.02))}
+
+    def workspace_bytes(self, n_tokens: int) -> int:
+        return n_tokens * 2 * self.hidden * (4 if self.env.dtype == torch.float32 else 2)
+
+    def _pair(self, n_tokens: int) -> torch.Tensor:
+        cap = self.env.max_step_tokens
+        return self.env.workspace.get("stream_mix.pair", (n_tokens, 2 * self.hidden), self.env.dtype, (cap, 2 * self.hidden))
+
+    def keep(self, residual: torch.Tensor) -> None:
+        """The stream as the embedding leaves it, for the passes of this step."""
+        ops.stream_step(residual, raw_out=self._pair(residual.shape[0])[:, self.hidden:])
+
+    def mix(self, x: Any, residual: torch.Tensor) -> None:
+        """Add what the layer before left (``x``) to the stream and replace the stream by the mix."""
+        pair = self._pair(residual.shape[0])
+        if isinstance(x, GatedSum):
+            x.fold(residual, raw_out=pair[:, : self.hidden])
+        else:
+            x = as_rows(x, None, residual)
+            if x is not None:
+                ops.stream_add_norm(residual, None, x1=x)
+            ops.stream_step(residual, raw_out=pair[:, : self.hidden])
+        ops.linear_f32(pair, self.params["weight"], residual)

@@ -18,6 +18,11 @@ and is added (moe.py:87-88).
 order, and the second product's weights are 1.  ``scoring="sigmoid_raw"`` leaves the chosen experts' sigmoid
 scores as they are (no division by their sum).  The reference has neither.
 
+``identity=n``: the router's last ``n`` outputs are experts without tensors that hand the layer's input back (times their
+weight).  Their routes get no rows; a token's weights on them are one number (``aux[t, 0]``), which the consumer of the
+:class:`RouteSum` applies to the input row.  ``shared_gate``: the shared expert's output is multiplied by
+``sigmoid(w_sg . h)``, whose logit is one more row of the router product (``aux[t, 1]``).  The reference has neither.
+
 ``router="token_table"`` has no router matrix: a table ``[vocab, top_k]`` of expert ids (the ids of a
 row differ) names each token id's experts, each with weight ``1 / top_k``; the expert products are
 the same kernels.  The reference has no such router.
@@ -65,7 +70,8 @@ class MoE(FeedForward):
     """params: ``hidden``, ``inter``, ``n_experts``, ``top_k``, ``scoring`` ("sigmoid" |
     "softmax"), ``bias`` (bool), ``scale``, ``act``, ``alpha``, ``limit``,
     ``shared_inter`` (0 = no shared expert), ``shared_limit`` (the shared expert's clamp; ``limit`` when absent), ``router`` ("learned" | "token_table"; the table also needs
-    ``vocab``), ``weight_on`` ("output" | "input").  ``h_f32`` given to the forward calls of a bfloat16 model
+    ``vocab``), ``weight_on`` ("output" | "input"), ``identity`` (experts behind the ``n_experts`` real ones that hand the
+    input back, 0), ``shared_gate`` (bool), ``router_store`` (dtype of router and bias in written files), ``bias_std``.  ``h_f32`` given to the forward calls of a bfloat16 model
     is ``float32(h)``, as a norm's ``out_f32`` is."""
 
     wants_f32_input = True
@@ -76,8 +82,10 @@ class MoE(FeedForward):
         self.inter = int(spec["inter"])
         self.n_experts = int(spec["n_experts"])
         self.top_k = int(spec["top_k"])
-        if not 1 <= self.top_k <= self.n_experts:
-            raise ConfigError("moe: top_k must be in [1, n_experts]")
+        self.identity = int(spec.get("identity", 0) or 0)
+        self.n_choices = self.n_experts + self.identity
+        if self.identity < 0 or not 1 <= self.top_k <= self.n_choices:
+            raise ConfigError("moe: top_k must be in [1, number of experts]")
         self.scoring = spec.get("scoring", "sigmoid")
         if self.scoring not in ops.SCORE_CODES:
             raise ConfigError(f"moe: unknown scoring '{self.scoring}'")
@@ -100,6 +108,11 @@ class MoE(FeedForward):
         if self.by_table and self.vocab < 1:
             raise ConfigError("moe: a token-table router needs the vocabulary size")
         self._gate_pieces: Optional[torch.Tensor] = None
+        self._gate: Optional[torch.Tensor] = None  # the router's rows, and the shared expert's gate behind them
+        self.shared_gate = bool(spec.get("shared_gate", False)) and self.shared_inter > 0
+        self.has_aux = self.identity > 0 or self.shared_gate
+        if self.has_aux and (self.by_table or self.on_input):
+            raise ConfigError("moe: identity experts and a gated shared expert go with a learned router and weighted outputs")
         self.shared: Optional[GatedMLP] = None
         if self.shared_inter:
             self.shared = GatedMLP(PartSpec("gated_mlp", dict(
@@ -116,11 +129,15 @@ class MoE(FeedForward):
         if self.by_table:
             out["table"] = ParamSpec((self.vocab, self.top_k), "int32", ("distinct_ids", self.n_experts))
         else:
-            out["gate.weight"] = ParamSpec((self.n_experts, self.hidden), "float32",
-                                           ("normal", 0.0, std_in if std else 0.02))
+            out["gate.weight"] = ParamSpec((self.n_choices, self.hidden), "float32",
+                                           ("normal", 0.0, std_in if std else 0.02), store=self.spec.get("router_store"))
+        if self.shared_gate:
+            out["shared_gate.weight"] = ParamSpec((1, self.hidden), "float32", ("normal", 0.0, std_in if std else 0.02),
+                                                  store=self.spec.get("router_store"))
         if self.has_bias:
-            out["e_score_correction_bias"] = ParamSpec((self.n_experts,), "float32",
-                                                       ("normal", 0.0, 0.5 if std else 0.01))
+            out["e_score_correction_bias"] = ParamSpec((self.n_choices,), "float32",
+                                                       ("normal", 0.0, float(self.spec.get("bias_std", 0.5)) if std else 0.01),
+                                                       store=self.spec.get("router_store"))
         return out
 
     def children(self) -> Dict[str, Part]:
@@ -131,26 +148,29 @@ class MoE(FeedForward):
             return False
         # long bfloat16 steps take the router product from the bfloat16 rows themselves
         return not (self._gate_pieces is not None and self.env.dtype == torch.bfloat16
-                    and not ops.moe_route_fits(n_tokens, self.hidden, self.n_experts, self.top_k))
+                    and not ops.moe_route_fits(n_tokens, self.hidden, self.n_choices, self.top_k))
 
     def bind(self, tensors) -> None:
         super().bind(tensors)
         self._gate_pieces = None
+        self._gate = self.params.get("gate.weight")
+        if self.shared_gate:
+            self._gate = torch.cat([self._gate, self.params["shared_gate.weight"]]).contiguous()
         if self.on_input:
             self._ones = torch.ones(self.env.max_step_tokens * self.top_k, dtype=torch.float32, device=self.env.device)
         if self.env.dtype == torch.bfloat16 and SPLIT_ROUTER_PRODUCT and not self.by_table:
-            self._gate_pieces = split_in_three(self.params["gate.weight"])
+            self._gate_pieces = split_in_three(self._gate)
 
     def workspace_bytes(self, n_tokens: int) -> int:
         item = 4 if self.env.dtype == torch.float32 else 2
         T, k, H, I, E = n_tokens, self.top_k, self.hidden, self.inter, self.n_experts
         routed = T * k * ((2 * H + I) * item + 4 * 4)  # expert-ordered input, activation, output; ids, weights, sort
-        return routed + T * (H * (4 + item) + E * 4 * 4) + (2 * E + 1) * 4  # (logits, and their three pieces)
+        return routed + T * (H * (4 + item) + (E + self.identity + 1) * 4 * 4 + 8) + (2 * E + 1) * 4  # (logits, and their three pieces)
 
     def forward(self, h: torch.Tensor, step: StepState, h_f32: Optional[torch.Tensor] = None) -> torch.Tensor:
         return self.forward_lazy(h, step, h_f32).rows()
 
-    def _few_tokens(self, h, h_f32, step, logits, ids, wts, bias) -> RouteSum:
+    def _few_tokens(self, h, h_f32, step, logits, ids, wts, bias, aux) -> RouteSum:
         """Steps of up to four tokens: the routes stay in token order (no sort, no gathered copy of the
         activations) and each route's expert rows are streamed by the few-token kernels."""
         T = h.shape[0]
@@ -159,10 +179,10 @@ class MoE(FeedForward):
         if self.by_table:
             ops.table_route(step.token_ids, self.params["table"], self.n_experts, ids, wts)
         else:
-            ops.moe_route(h_f32, self.params["gate.weight"], bias, k, self.scoring, self.scale, logits, ids, wts)
+            ops.moe_route(h_f32, self._gate, bias, k, self.scoring, self.scale, logits, ids, wts, **self._aux_args(aux))
         record = self.env.shared.get("record_expert_counts")
         if record is not None:
-            record.append(torch.bincount(ids.view(-1).long(), minlength=self.n_experts).to(torch.int32))
+            record.append(torch.bincount(ids.view(-1).long(), minlength=self.n_experts)[: self.n_experts].to(torch.int32))
         if "moe.pos.identity" not in self.env.shared:
             self.env.shared["moe.pos.identity"] = torch.arange(64 * 64, dtype=torch.int32, device=self.env.device)
         pos = self.env.shared["moe.pos.identity"][:R]
@@ -172,7 +192,12 @@ class MoE(FeedForward):
         ops.moe_small_down(a, ids, wts, self.params["experts.down_proj"], y)
         shared = self.shared.forward(h, step) if self.shared is not None else None
         out = ws.get("moe.out", (T, self.hidden), dt, (cap, self.hidden))
-        return RouteSum(y, pos, k, shared, T, out)
+        # (the rows of routes to identity experts are zeros)
+        return RouteSum(y, pos, k, shared, T, out, aux, h if self.identity else None)
+
+    def _aux_args(self, aux: Optional[torch.Tensor]) -> dict:
+        """What the routing kernels are told about identity experts and the shared expert's gate."""
+        return {} if aux is None else dict(n_extra=int(self.shared_gate), n_real=self.n_experts, aux=aux)
 
     def forward_lazy(self, h: torch.Tensor, step: StepState, h_f32: Optional[torch.Tensor] = None) -> RouteSum:
         """The experts' rows and where each token's routes lie among them; the sum over a token's routes
@@ -188,7 +213,10 @@ class MoE(FeedForward):
             else:
                 h_f32 = ws.get("moe.h_f32", (T, self.hidden), torch.float32, (cap, self.hidden))
                 ops.cast(h, h_f32)
-        logits = ws.get("moe.logits", (T, E), torch.float32, (cap, E))
+        C = self.n_choices
+        L = C + int(self.shared_gate)  # logits of a token
+        logits = ws.get("moe.logits", (T, L), torch.float32, (cap, L))
+        aux = ws.get("moe.aux", (T, 2), torch.float32, (cap, 2)) if self.has_aux else None
         ids = ws.get("moe.ids", (T, k), torch.int32, (cap, k))
         wts = ws.get("moe.weights", (T, k), torch.float32, (cap, k))
         counts = ws.get("moe.counts", (E,), torch.int32)
@@ -197,23 +225,23 @@ class MoE(FeedForward):
         pos = ws.get("moe.pos", (R,), torch.int32, (cap * k,))
         bias = self.params.get("e_score_correction_bias")
         if (dt == torch.bfloat16 and not self.on_input and ops.moe_small_fits(T, self.hidden, self.inter, k)
-                and (self.by_table or ops.moe_route_fits(T, self.hidden, E, k))):
-            return self._few_tokens(h, h_f32, step, logits, ids, wts, bias)
+                and (self.by_table or ops.moe_route_fits(T, self.hidden, C, k))):
+            return self._few_tokens(h, h_f32, step, logits, ids, wts, bias, aux)
         if self.by_table:  # the table names the experts; the sort is the one every router's choice gets
             ops.table_route(step.token_ids, self.params["table"], E, ids, wts)
             ops.moe_permute(ids, E, counts, offsets, routes, pos)
-        elif ops.moe_route_fits(T, self.hidden, E, k):  # small steps: logits, choice and sort in one launch
-            ops.moe_route(h_f32, self.params["gate.weight"], bias, k, self.scoring, self.scale, logits, ids, wts,
-                          counts, offsets, routes, pos)
+        elif ops.moe_route_fits(T, self.hidden, C, k):  # small steps: logits, choice and sort in one launch
+            ops.moe_route(h_f32, self._gate, bias, k, self.scoring, self.scale, logits, ids, wts,
+                          counts, offsets, routes, pos, **self._aux_args(aux))
         elif self._gate_pieces is not None and h.dtype == torch.bfloat16:
             # the router reads float32(h): the three products below are exact, their 32-bit sums are the logits
-            pieces = ws.get("moe.logit_pieces", (T, 3 * E), torch.float32, (cap, 3 * E))
+            pieces = ws.get("moe.logit_pieces", (T, 3 * L), torch.float32, (cap, 3 * L))
             torch.mm(h, self._gate_pieces.t(), out_dtype=torch.float32, out=pieces)
-            ops.router_topk(pieces, bias, k, self.scoring, self.scale, ids, wts, n_parts=3)
+            ops.router_topk(pieces, bias, k, self.scoring, self.scale, ids, wts, n_parts=3, **self._aux_args(aux))
             ops.moe_permute(ids, E, counts, offsets, routes, pos)
         else:
-            torch.matmul(h_f32, self.params["gate.weight"].t(), out=logits)
-            ops.router_topk(logits, bias, k, self.scoring, self.scale, ids, wts)
+            torch.matmul(h_f32, self._gate.t(), out=logits)
+            ops.router_topk(logits, bias, k, self.scoring, self.scale, ids, wts, **self._aux_args(aux))
             ops.moe_permute(ids, E, counts, offsets, routes, pos)
         record = self.env.shared.get("record_expert_counts")
         if record is not None:  # measurement hook: which experts a step touched, layer by layer
@@ -238,4 +266,4 @@ class MoE(FeedForward):
                       self._ones[:R] if self.on_input else wts.view(-1), y)
         shared = self.shared.forward(h, step) if self.shared is not None else None
         out = ws.get("moe.out", (T, self.hidden), dt, (cap, self.hidden))
-        return RouteSum(y, pos, k, shared, T, out)
+        return RouteSum(y, pos, k, shared, T, out, aux, h if self.identity else None)

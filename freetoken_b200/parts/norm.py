@@ -17,16 +17,19 @@ import torch
 
 from ..config.spec import ParamSpec, PartSpec
 from ..kernels import ops
-from .base import NORMS, BuildEnv, Norm, NormedSum, RouteSum, StreamSum
+from ..errors import ConfigError
+from .base import NORMS, BuildEnv, GatedSum, Norm, NormedSum, RouteSum, StreamSum
 
 
 @NORMS.register("rmsnorm")
 class RMSNorm(Norm):
     """params: ``size``, ``eps``, ``gemma`` (bool: multiply by ``1 + w``), ``scalar`` (bool: the weight is one
-    number for all coordinates; the checkpoint tensor has no axis)."""
+    number for all coordinates; the checkpoint tensor has no axis), ``groups`` (1: the row is cut into that many equal
+    consecutive parts, each divided by its own root mean square)."""
 
     takes_route_sum = True
     takes_normed_sum = True
+    takes_gated_sum = True
 
     def __init__(self, spec: PartSpec, env: BuildEnv):
         super().__init__(spec, env)
@@ -34,6 +37,10 @@ class RMSNorm(Norm):
         self.eps = float(spec["eps"])
         self.gemma = bool(spec.get("gemma", True))
         self.scalar = bool(spec.get("scalar", False))
+        self.groups = int(spec.get("groups", 1))
+        if self.groups < 1 or self.size % self.groups:
+            raise ConfigError(f"rmsnorm: {self.size} channels do not divide into {self.groups} groups")
+        self._w: Optional[torch.Tensor] = None  # the weight as the kernels for groups take it (1 + w in the Gemma form)
 
     def param_specs(self) -> Dict[str, ParamSpec]:
         init = ("normal", 0.0, 0.02) if self.gemma else ("normal", 1.0, 0.02)
@@ -45,8 +52,18 @@ class RMSNorm(Norm):
         super().bind(tensors)
         if self.scalar:  # the kernels take one weight per coordinate
             self.params["weight"] = self.params["weight"].reshape(1).expand(self.size).contiguous()
+        self._w = self.params["weight"] + 1.0 if self.gemma else self.params["weight"]
+
+    def norm_stream(self, residual: torch.Tensor) -> None:
+        """The stream's rows become their norms, in 32 bits."""
+        ops.stream_step(residual, groups=self.groups, pre_weight=self._w, pre_eps=self.eps, norm_f32=residual)
 
     def forward(self, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+        if self.groups > 1:
+            if x.dtype != torch.float32:
+                raise ConfigError("rmsnorm: a norm over groups takes 32-bit rows")
+            ops.stream_step(x, groups=self.groups, pre_weight=self._w, pre_eps=self.eps, out=out)
+            return out
         ops.add_rmsnorm(x, None, self.params["weight"], self.eps, self.gemma, out)
         return out
 
@@ -56,6 +73,20 @@ class RMSNorm(Norm):
         if isinstance(x, StreamSum):
             x.fold(residual)
             x = None
+        if isinstance(x, GatedSum) and x.groups != self.groups:
+            x.fold(residual)
+            x = None
+        if isinstance(x, GatedSum) or self.groups > 1:  # gate, the sub-layer's own norm, the sum and this norm in one pass
+            if out_f32 is not None:
+                raise ConfigError("rmsnorm: no 32-bit copy of the output of a norm over groups")
+            if x is not None and not isinstance(x, GatedSum):
+                (x if isinstance(x, NormedSum) else StreamSum.of(x)).fold(residual)
+                x = None
+            args = x.kernel_args() if x is not None else dict(groups=self.groups)
+            ops.stream_step(residual, pre_weight=self._w, pre_eps=self.eps, out=out, rows=rows, **args)
+            return out
+        if isinstance(x, RouteSum):
+            x = x.plain()
         if isinstance(x, NormedSum):  # the sub-layer's own norm, the sum and this norm in one pass
             data, routed = x.kernel_args()
             ops.postnorm_add_norm(data, routed, x.norm.params["weight"], x.norm.eps, x.norm.gemma, residual,

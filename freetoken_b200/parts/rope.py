@@ -12,6 +12,12 @@ their own kernels (``norm_rope_store``); one table serves all layers with equal 
 ``rope_interleaved``: the same angles and table; the pairs that turn together are the neighbours ``(2i, 2i + 1)``
 instead of ``(i, i + rotary_dim / 2)``.  A mixer's kernel asks the part (``interleaved``) which pairing to use.
 
+``yarn`` (a parameter of both): frequencies stretched for contexts longer than the ``original`` one a model was trained on
+(YaRN).  With ``index(t) = rotary_dim ln(original / (2 pi t)) / (2 ln theta)``, the index whose pair turns ``t`` times over
+the original context, ``lo = max(floor(index(fast)), 0)`` and ``hi = min(ceil(index(slow)), rotary_dim - 1)``, pair ``i``
+turns at ``f_i / factor`` with the share ``ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1)`` and at ``f_i`` with the
+rest; cosines and sines are multiplied by ``0.1 ln(factor) + 1``.
+
 ``none``: no position encoding (a mixer that needs none asks for this kind).
 
 ``log_temperature``: no rotation; the table holds one factor per position,
@@ -22,6 +28,7 @@ float32.
 
 from __future__ import annotations
 
+import math
 from typing import Optional
 
 import torch
@@ -34,7 +41,8 @@ from .base import POSITIONS, BuildEnv, PositionEncoding
 @POSITIONS.register("rope_neox")
 class NeoxRope(PositionEncoding):
     """params: ``rotary_dim`` (even, <= head_dim; 0 disables), ``theta``, ``precise`` (False: the reference's
-    float32 operations; True: angles, cosines and sines in float64, rounded to float32 once)."""
+    float32 operations; True: angles, cosines and sines in float64, rounded to float32 once), ``yarn`` (None, or
+    ``(factor, original, fast, slow)``; needs ``precise``)."""
 
     interleaved = False
 
@@ -44,7 +52,29 @@ class NeoxRope(PositionEncoding):
         self.theta = float(spec["theta"])
         if self.rotary_dim % 2 or self.rotary_dim < 0:
             raise ConfigError(f"rope_neox: rotary_dim={self.rotary_dim} must be even and >= 0")
+        self.yarn = spec.get("yarn")
+        if self.yarn is not None and not spec.get("precise", False):
+            raise ConfigError("rope: stretched frequencies are computed in float64 (precise)")
         self._table: Optional[torch.Tensor] = None
+
+    def frequencies(self) -> torch.Tensor:
+        """One per pair, float64."""
+        rd = self.rotary_dim
+        f = self.theta ** (-torch.arange(0, rd, 2, dtype=torch.float64) / rd)
+        if self.yarn is None:
+            return f
+        factor, original, fast, slow = (float(x) for x in self.yarn)
+
+        def index(turns: float) -> float:
+            return rd * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.theta))
+
+        lo, hi = max(math.floor(index(fast)), 0), min(math.ceil(index(slow)), rd - 1)
+        ramp = ((torch.arange(rd // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        return f / factor * ramp + f * (1.0 - ramp)
+
+    def magnitude(self) -> float:
+        """The factor on cosines and sines."""
+        return 1.0 if self.yarn is None else 0.1 * math.log(float(self.yarn[0])) + 1.0
 
     def table(self) -> Optional[torch.Tensor]:
         """Built at the first call: by then the engine has settled its longest sequence
@@ -53,9 +83,9 @@ class NeoxRope(PositionEncoding):
         if self._table is None and self.rotary_dim:
             rd = self.rotary_dim
             if self.spec.get("precise", False):
-                inv = self.theta ** (-torch.arange(0, rd, 2, dtype=torch.float64) / rd)
-                ang = torch.arange(self.env.max_seq_len, dtype=torch.float64)[:, None] * inv[None, :]
-                self._table = torch.cat((ang.cos(), ang.sin()), dim=-1).float().contiguous().to(self.env.device)
+                ang = torch.arange(self.env.max_seq_len, dtype=torch.float64)[:, None] * self.frequencies()[None, :]
+                tab = torch.cat((ang.cos(), ang.sin()), dim=-1) * self.magnitude()
+                self._table = tab.float().contiguous().to(self.env.device)
                 return self._table
             inv_freq = 1.0 / (self.theta ** (torch.arange(0, rd, 2, dtype=torch.float) / rd))
             t = torch.arange(self.env.max_seq_len, dtype=torch.float)

@@ -40,6 +40,7 @@ _LAZY: Dict[str, str] = {
     "Pabavik": "freetoken_b200.models.pabavik",
     "Kekopel": "freetoken_b200.models.kekopel",
     "Nusudra": "freetoken_b200.models.nusudra",
+    "Vodatar": "freetoken_b200.models.vodatar",
 }
 
 

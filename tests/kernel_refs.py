@@ -112,7 +112,7 @@ def norm_rope_store(x, head_dim, rotary_dim, positions, rope_table, eps, gemma, 
 
 def paged_attention(q, k_slab, v_slab, block_table, seg_info, n_segs, items, n_items, part_o, part_ml,
                     out, tile_rows, scale, window, sel=None, block_size=0, few_rows=False, dist_bias=None, kv_split=1,
-                    sink=None):
+                    sink=None, softcap=None):
     """Per query token, softmax over the visible keys gathered through the block table; the
     work list and the scratch are ignored (they only steer how the kernel splits the work).
     With ``sel`` a query reads only the keys of its chosen blocks."""
@@ -133,6 +133,8 @@ def paged_attention(q, k_slab, v_slab, block_table, seg_info, n_segs, items, n_i
             if sel is None:
                 kk, vv = K[lo:p_q + 1], V[lo:p_q + 1]
                 s = torch.einsum("hgd,khd->hgk", qq, kk) * scale
+                if softcap:
+                    s = softcap * torch.tanh(s / softcap)
                 if dist_bias is not None:  # [Hq, L] by distance, the last entry for everything farther
                     dist = (p_q - torch.arange(lo, p_q + 1, device=q.device)).clamp(max=dist_bias.shape[1] - 1)
                     s = s + dist_bias.float()[:, dist].view(Hkv, G, -1)
@@ -187,13 +189,26 @@ def sparse_select(iq, ik_slab, block_table, seg_info, n_segs, block_size, local_
             sel[q_start + t, :, : chosen.shape[1]] = chosen.to(torch.int32)
 
 
-def router_topk(logits, bias, top_k, scoring, scale, ids, weights, n_parts=1):
+def router_topk(logits, bias, top_k, scoring, scale, ids, weights, n_parts=1, n_extra=0, n_real=None, aux=None):
     l = logits.float()
     if n_parts > 1:
         parts = l.view(l.shape[0], n_parts, -1)
         l = parts[:, 0]
         for q in range(1, n_parts):
             l = l + parts[:, q]
+    extra = None
+    if n_extra:
+        l, extra = l[:, :-n_extra], l[:, -1]
+    if aux is not None:
+        _choose(l, bias, top_k, scoring, scale, ids, weights)
+        real = l.shape[1] if n_real is None else n_real
+        aux[:, 0] = torch.where(ids >= real, weights, torch.zeros_like(weights)).sum(-1)
+        aux[:, 1] = torch.sigmoid(extra) if extra is not None else 1.0
+        return
+    _choose(l, bias, top_k, scoring, scale, ids, weights)
+
+
+def _choose(l, bias, top_k, scoring, scale, ids, weights):
     if scoring == "softmax_of_chosen":  # the bias belongs to the logit; the softmax runs over the chosen logits only
         l = l + bias.float() if bias is not None else l
         idx = torch.argsort(l, dim=-1, descending=True, stable=True)[:, :top_k]
@@ -210,20 +225,22 @@ def router_topk(logits, bias, top_k, scoring, scale, ids, weights, n_parts=1):
     c = s + bias.float() if bias is not None else s
     idx = torch.argsort(c, dim=-1, descending=True, stable=True)[:, :top_k]
     w = s.gather(-1, idx)
-    w = w / (w.sum(-1, keepdim=True) + (1e-20 if scoring == "sigmoid" else 0.0))
+    w = w / (w.sum(-1, keepdim=True) + 1e-20)
     ids.copy_(idx.to(torch.int32))
     weights.copy_(w * scale)
 
 
 def moe_permute(topk_ids, n_experts, expert_counts, expert_offsets, sorted_routes, route_pos):
-    flat = topk_ids.reshape(-1).long()
+    flat = topk_ids.reshape(-1).long()  # ids from n_experts on name experts without rows: behind the others, place -1
     order = torch.argsort(flat, stable=True)
-    counts = torch.bincount(flat, minlength=n_experts)
+    counts = torch.bincount(flat, minlength=n_experts)[:n_experts]
     expert_counts.copy_(counts.to(torch.int32))
     expert_offsets[0] = 0
     expert_offsets[1:] = torch.cumsum(counts, 0).to(torch.int32)
     sorted_routes.copy_(order.to(torch.int32))
     route_pos[order] = torch.arange(flat.numel(), dtype=torch.int32, device=flat.device)
+    route_pos[flat >= n_experts] = -1
+    sorted_routes[int(counts.sum()):] = -1
 
 
 def moe_gemm1_gather_fits(dtype, hidden, inter, n_experts, n_routes):
@@ -247,14 +264,16 @@ def moe_route_fits(n_tokens, hidden, n_experts, top_k):
 
 
 def moe_route(x, gate_w, bias, top_k, scoring, scale, logits, ids, weights, expert_counts, expert_offsets,
-              sorted_routes, route_pos):
+              sorted_routes, route_pos, n_extra=0, n_real=None, aux=None):
     logits.copy_(x.float() @ gate_w.float().T)
-    router_topk(logits, bias, top_k, scoring, scale, ids, weights)
-    moe_permute(ids, gate_w.shape[0], expert_counts, expert_offsets, sorted_routes, route_pos)
+    router_topk(logits, bias, top_k, scoring, scale, ids, weights, n_extra=n_extra, n_real=n_real, aux=aux)
+    moe_permute(ids, gate_w.shape[0] - n_extra if n_real is None else n_real, expert_counts, expert_offsets, sorted_routes,
+                route_pos)
 
 
 def moe_gather(h, sorted_routes, top_k, out):
-    out.copy_(h[(sorted_routes.long() // top_k)])
+    live = sorted_routes >= 0
+    out[live] = h[(sorted_routes[live].long() // top_k)]
 
 
 def moe_gemm1_act(x_sorted, w1, expert_offsets, act, alpha, limit, out):
@@ -277,14 +296,20 @@ def moe_gemm2(a, w2, expert_offsets, sorted_routes, topk_weights, out):
             out[lo:hi] = y.to(out.dtype)
 
 
-def moe_combine(y, route_pos, n_tokens, top_k, shared, out):
-    pos = route_pos.view(n_tokens, top_k).long()
+def _sum_of_routes(y, route_pos, n_tokens, top_k, shared, aux=None, passed=None):
+    pos = route_pos.view(-1)[: n_tokens * top_k].view(n_tokens, top_k).long()
     acc = torch.zeros(n_tokens, y.shape[1], dtype=torch.float32, device=y.device)
     for j in range(top_k):
-        acc = acc + y[pos[:, j]].float()
+        acc = acc + torch.where((pos[:, j] >= 0)[:, None], y[pos[:, j].clamp(min=0)].float(), torch.zeros_like(acc))
+    if passed is not None:
+        acc = acc + aux[:, :1] * passed.float()
     if shared is not None:
-        acc = acc + shared.float()
-    out.copy_(acc.to(out.dtype))
+        acc = acc + shared.float() * (aux[:, 1:] if aux is not None else 1.0)
+    return acc
+
+
+def moe_combine(y, route_pos, n_tokens, top_k, shared, out, aux=None, passed=None):
+    out.copy_(_sum_of_routes(y, route_pos, n_tokens, top_k, shared, aux, passed).to(out.dtype))
 
 
 def sample(logits, temperature, top_k, top_p, u, out):
@@ -597,6 +622,89 @@ def conv_act(x, w, bias, act, state, state_slots, seg_info, n_segs, out):
             state[slot] = line[-keep:]
 
 
+def _group_norm(z, groups, eps):
+    parts = z.view(z.shape[0], groups, -1)
+    return (parts * torch.rsqrt((parts * parts).mean(-1, keepdim=True) + eps)).view(z.shape)
+
+
+def stream_step(residual, groups=1, vec=None, x=None, routed=None, gate=None, gate_bias=None, post_weight=None, post_eps=0.0,
+                raw_out=None, pre_weight=None, pre_eps=0.0, out=None, norm_f32=None, conv=None, rows=None, dtype=None):
+    z = residual.float().clone()
+    T = z.shape[0]
+    if vec is not None:
+        z = z + vec.float()
+    if x is not None:
+        if routed is not None:
+            pos, top_k, shared, aux, passed = routed
+            y = _sum_of_routes(x, pos, T, top_k, shared, aux, passed)
+        else:
+            y = x.float()[:T]
+        if gate is not None:
+            g = gate.float()[:T]
+            y = y * torch.sigmoid(g if gate_bias is None else g + gate_bias.float())
+        z = z + _group_norm(y, groups, post_eps) * post_weight.float()
+    if rows is None:
+        residual.copy_(z)
+    else:
+        z = z[rows.long()]
+    if raw_out is not None:
+        raw_out.copy_(z.to(raw_out.dtype))
+    if pre_weight is None:
+        return
+    h = _group_norm(z, groups, pre_eps) * pre_weight.float()
+    if norm_f32 is not None:
+        norm_f32.copy_(h)
+    if out is not None:
+        out.view(h.shape).copy_(h.to(out.dtype))
+    if conv is not None:
+        w, state, slots, seg_info, c_out, c_out_f32 = conv
+        h = h.to(c_out.dtype).float()
+        info = seg_info.view(-1, 4)
+        for t in range(T):
+            _, n, kv_len, _ = info[t].tolist()
+            assert n == 1
+            keep = w.shape[1] - 1
+            line = h[t:t + 1]
+            if keep:
+                slot = int(slots[t])
+                old = torch.zeros_like(state[slot]) if kv_len == 1 else state[slot].clone()
+                line = torch.cat([old, line])
+                state[slot] = line[-keep:]
+            c_out[t] = (h[t] + (w.float().T * line).sum(0)).to(c_out.dtype)
+        if c_out_f32 is not None:
+            c_out_f32.copy_(c_out.float())
+
+
+def conv_rope_store(x, conv_w, state, state_slots, seg_info, n_segs, n_heads, n_kv_heads, maps, dim, vdim, n_rot, interleaved,
+                    positions, rope_table, q_out, k_slab, v_slab, slot_map):
+    T = x.shape[0]
+    y = torch.empty(T, x.shape[1], dtype=torch.float32)
+    conv_act(x, conv_w, None, None, state, state_slots, seg_info, n_segs, y)
+    nq, nk = n_heads * maps * dim, n_kv_heads * maps * dim
+    q = y[:, :nq].reshape(T, n_heads, maps, dim)
+    k = y[:, nq:nq + nk].reshape(T, n_kv_heads, maps, dim)
+    v = y[:, nq + nk:].reshape(T, n_kv_heads, vdim)
+    page = k_slab.shape[2]
+    q_out.zero_()
+    for t in range(T):
+        p = int(positions[t])
+        qt, kt = (_turn(a[t], p, rope_table, n_rot, interleaved) if n_rot else a[t] for a in (q, k))
+        for m in range(maps):
+            q_out[t, m::maps, m * dim:(m + 1) * dim] = qt[:, m].to(q_out.dtype)
+        slot = int(slot_map[t])
+        if slot < 0:
+            continue
+        for slab, row in ((k_slab, kt.reshape(n_kv_heads, maps * dim)), (v_slab, v[t])):
+            slab[slot // page, :, slot % page] = 0
+            slab[slot // page, :, slot % page, : row.shape[1]] = row.to(slab.dtype)
+
+
+def diff_heads(o, lam, eps, scale, out):
+    Dv = out.shape[2]
+    d = o[:, 0::2, :Dv].float() - lam * o[:, 1::2, :Dv].float()
+    out.copy_((d * torch.rsqrt((d * d).mean(-1, keepdim=True) + eps) * scale).to(out.dtype))
+
+
 def ssm_gates(dt_raw, dt_bias, a_log, dt_out, decay_out):
     dt = torch.nn.functional.softplus(dt_raw.float() + dt_bias.float(), threshold=1e9)
     dt_out.copy_(dt)
@@ -634,7 +742,7 @@ def delta_scan(q, k, v, b_raw, a_raw, a_log, dt_bias, q_scale, unit_eps, state, 
         state[slot] = S.transpose(1, 2)
 
 
-ALL = ["hyper_step", "norm_mean", "conv_act", "ssm_gates", "ssm_output", "delta_scan", "short_conv", "depth_mix", "moe_gather_scaled", "relu2_", "latent_store", "latent_query_rotate", "mlstm_gates", "mlstm_output", "linear_f32", "softcap_", "postnorm_add_norm", "gated_heads", "gla_scan", "stream_add_norm", "head_gate", "table_route", "scale_", "sparse_score_fits", "moe_small_fits", "copy_tokens", "sparse_select", "embedding_gather", "add_rmsnorm", "add_rmsnorm_routes", "act_and_mul", "cast", "table_update", "norm_rope_store",
+ALL = ["stream_step", "conv_rope_store", "diff_heads", "hyper_step", "norm_mean", "conv_act", "ssm_gates", "ssm_output", "delta_scan", "short_conv", "depth_mix", "moe_gather_scaled", "relu2_", "latent_store", "latent_query_rotate", "mlstm_gates", "mlstm_output", "linear_f32", "softcap_", "postnorm_add_norm", "gated_heads", "gla_scan", "stream_add_norm", "head_gate", "table_route", "scale_", "sparse_score_fits", "moe_small_fits", "copy_tokens", "sparse_select", "embedding_gather", "add_rmsnorm", "add_rmsnorm_routes", "act_and_mul", "cast", "table_update", "norm_rope_store",
        "paged_attention", "router_topk", "moe_permute", "moe_route", "moe_route_fits", "linear", "attention_tc_fits", "attention_tc_few_fits", "moe_gemm1_gather_fits", "moe_gather", "moe_gemm1_act", "moe_gemm2",
        "moe_combine", "sample"]
 
