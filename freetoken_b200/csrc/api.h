@@ -78,8 +78,8 @@ typedef struct {
   float sink_logit;
   // with has_sink: one logit per query head [n_q_heads] (float32) instead of sink_logit; null = sink_logit for all
   const float* sink_heads;
-  // scores (scaled) become softcap * tanh(score / softcap); 0 = as they are.  Not with block selection, a bias by
-  // distance or the form with two 128-row tiles.
+  // scores (scaled) become softcap * tanh(score / softcap); 0 = as they are.  Not with block selection or a bias by
+  // distance.
   float softcap;
 } FtkAttnExtras;
 
@@ -310,13 +310,13 @@ int ftk_paged_attention_tc(const void* q, const void* k_slab, const void* v_slab
                            float* part_o, float* part_ml, int n_slots, void* out, int n_tokens, int n_q_heads,
                            int n_kv_heads, int head_dim, int page_size, int num_pages, float scale, int window,
                            void* stream);
-// The 128-row form, or with few_rows the form for tiles of at most 16 rows, with options (a distance bias).  In both
-// forms k_slab == v_slab (values that are the keys) makes the key tile in shared memory serve both products.
+// With options: the 128-row form (form 0), the one for tiles of at most 16 rows (1) or the one with two 128-row tiles (2;
+// a soft cap alone).  In the first two forms k_slab == v_slab (values that are the keys) makes the key tile in shared memory serve both products.
 int ftk_paged_attention_tc_ex(const void* q, const void* k_slab, const void* v_slab, const int32_t* block_table,
                               int bt_stride, const int32_t* seg_info, int n_segs, const int32_t* items, int n_items,
                               float* part_o, float* part_ml, int n_slots, void* out, int n_tokens, int n_q_heads,
                               int n_kv_heads, int head_dim, int page_size, int num_pages, float scale, int window,
-                              const FtkAttnExtras* extras, int few_rows, void* stream);
+                              const FtkAttnExtras* extras, int form, void* stream);
 // Decode steps in bfloat16 on the same kernel with tiles of at most 16 query rows (plan the items with
 // tile_rows = 16 and key pieces that are multiples of 128; at most 16 query heads per KV head): one
 // warp takes the softmax of the tile's rows.  part_o [slots, Hkv, 16, 128], part_ml [slots, Hkv, 16, 2].

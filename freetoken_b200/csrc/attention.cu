@@ -67,13 +67,89 @@ struct AttnParams {
   float softcap;
 };
 
-// softcap * tanh(x * to_arg) for results in `out_scale` units: out_scale * (1 - 2 / (e^(2 x to_arg) + 1)), with the
-// exponential's argument in base 2.  About 1e-7 of out_scale away from the exact value; saturates cleanly at both ends.
-__device__ __forceinline__ float capped_score(float x, float to_exp2, float out_scale) {
+// Soft-capped scores of the bfloat16 kernels: raw products s become softcap * log2(e) * tanh(s * scale / softcap), scores
+// in the exp2 domain.  Two ways to the same value, each within 2e-7 of softcap: for |argument| <= kCapSmall (most scores
+// of a model whose cap is there for outliers) an odd polynomial, two scores at a time, which leaves the special-function
+// unit to the softmax; else 1 - 2 / (e^(2x) + 1), which saturates cleanly at both ends.  The polynomial is a minimax fit
+// of tanh(x) / x in x^2 on [0, 1/16] (Lawson iteration; largest error of tanh 6e-8).
+constexpr float kCapSmall = 0.25f;
+// whether 2^(-2 softcap log2(e)) is far from the end of the exponent range
+inline bool soft_cap_bounded(float softcap) { return softcap * 1.4426950408889634f <= 50.f; }
+struct SoftCap {
+  float arg;          // scale / softcap
+  float arg_exp2;     // 2 log2(e) scale / softcap
+  float out;          // softcap log2(e)
+  uint64_t c0, c1, c2;  // the polynomial's coefficients for raw scores, times `out`, each twice
+};
+__device__ __forceinline__ uint64_t pack_f32x2(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void unpack_f32x2(uint64_t p, float& a, float& b) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(p));
+}
+__device__ __forceinline__ uint64_t fma_f32x2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul_f32x2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t add_f32x2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ SoftCap soft_cap(float scale, float softcap) {
+  SoftCap c;
+  c.arg = scale / softcap;
+  c.arg_exp2 = 2.f * 1.4426950408889634f * c.arg;
+  c.out = softcap * 1.4426950408889634f;
+  const float a1 = c.out * c.arg, a3 = a1 * c.arg * c.arg, a5 = a3 * c.arg * c.arg;
+  c.c0 = pack_f32x2(9.999986291e-01f * a1, 9.999986291e-01f * a1);
+  c.c1 = pack_f32x2(-3.331570029e-01f * a3, -3.331570029e-01f * a3);
+  c.c2 = pack_f32x2(1.276223212e-01f * a5, 1.276223212e-01f * a5);
+  return c;
+}
+__device__ __forceinline__ float capped_any(float s, const SoftCap& c) {
   float e, r;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * to_exp2));
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(s * c.arg_exp2));
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.f));
-  return fmaf(-2.f * out_scale, r, out_scale);
+  return fmaf(-2.f * c.out, r, c.out);
+}
+// (small arguments only) two scores, plus `add`
+__device__ __forceinline__ void capped_small2(float& s0, float& s1, const SoftCap& c, uint64_t add) {
+  const uint64_t x = pack_f32x2(s0, s1), y = mul_f32x2(x, x);
+  unpack_f32x2(fma_f32x2(x, fma_f32x2(y, fma_f32x2(y, c.c2, c.c1), c.c0), add), s0, s1);
+}
+// Whether all of the warp's scores have small arguments (NaNs of keys that do not exist are looked past, and so is a thread
+// whose rows do not: `live`).
+__device__ __forceinline__ float max3_abs(float a, float b, float c) {
+  float r;
+  asm("max.abs.f32 %0, %1, %2, %3;" : "=f"(r) : "f"(a), "f"(b), "f"(c));
+  return r;
+}
+template <int N>
+__device__ __forceinline__ bool all_small(const float (&s)[N], const SoftCap& c, bool live = true) {
+  float m[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < N; i += 2) m[(i >> 1) & 3] = max3_abs(m[(i >> 1) & 3], s[i], s[i + 1]);
+  return __all_sync(0xffffffffu, fmaxf(fmaxf(m[0], m[1]), fmaxf(m[2], m[3])) * c.arg <= kCapSmall || !live);
+}
+// In place, for a warp's scores.
+template <int N>
+__device__ __forceinline__ void cap_scores(float (&s)[N], const SoftCap& c, bool live) {
+  if (all_small(s, c, live)) {
+#pragma unroll
+    for (int i = 0; i < N; i += 2) capped_small2(s[i], s[i + 1], c, 0ull);
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i) s[i] = capped_any(s[i], c);
+  }
 }
 
 // What the sink adds to a row's sum of exponentials taken relative to the maximum `m` (natural logarithm domain).
@@ -482,8 +558,7 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(AttnParams p) {
   const int lo0 = p.window > 0 ? qp0 - p.window + 1 : 0;
   const int lo1 = p.window > 0 ? qp1 - p.window + 1 : 0;
   // with a soft cap the scores are scaled while they are capped
-  const float cap_arg = p.softcap > 0.f ? 2.f * p.scale / p.softcap * 1.4426950408889634f : 0.f;
-  const float cap_out = p.softcap * 1.4426950408889634f;
+  const SoftCap cap = soft_cap(p.scale, p.softcap > 0.f ? p.softcap : 1.f);
   const float sl2 = p.softcap > 0.f ? 1.f : p.scale * 1.4426950408889634f;
   const bool tied = p.k == p.v;
   const float kLog2e = 1.4426950408889634f;
@@ -526,10 +601,7 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(AttnParams p) {
       }
     }
     if (p.softcap > 0.f) {
-#pragma unroll
-      for (int n = 0; n < kBN / 8; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) s[n][e] = capped_score(s[n][e], cap_arg, cap_out);
+      cap_scores(*reinterpret_cast<float (*)[kBN / 2]>(&s), cap, qp0 >= 0 || qp1 >= 0);
     }
     // mask, running max
     const int c0 = it.kb + iter * kBN;
@@ -759,8 +831,7 @@ __global__ void __launch_bounds__(128) attention_decode_bf16_kernel(AttnParams p
   const int lo0 = p.window > 0 ? qp0 - p.window + 1 : 0;
   const int lo1 = p.window > 0 ? qp1 - p.window + 1 : 0;
   // with a soft cap the scores are scaled while they are capped
-  const float cap_arg = p.softcap > 0.f ? 2.f * p.scale / p.softcap * 1.4426950408889634f : 0.f;
-  const float cap_out = p.softcap * 1.4426950408889634f;
+  const SoftCap cap = soft_cap(p.scale, p.softcap > 0.f ? p.softcap : 1.f);
   const float sl2 = p.softcap > 0.f ? 1.f : p.scale * 1.4426950408889634f;
   const bool tied = p.k == p.v;
   const float kLog2e = 1.4426950408889634f;
@@ -798,10 +869,7 @@ __global__ void __launch_bounds__(128) attention_decode_bf16_kernel(AttnParams p
       }
     }
     if (p.softcap > 0.f) {
-#pragma unroll
-      for (int n = 0; n < 2; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) s[n][e] = capped_score(s[n][e], cap_arg, cap_out);
+      cap_scores(*reinterpret_cast<float (*)[8]>(&s), cap, qp0 >= 0 || qp1 >= 0);
     }
     const int c0 = it.kb + iter * kBN + warp * 16;
     float mx0 = -INFINITY, mx1 = -INFINITY;
@@ -1055,13 +1123,14 @@ static int paged_attention_tc_impl(const void* q, const void* k_slab, const void
   p.sink = extras ? extras->sink_logit : 0.f;
   p.sink_heads = extras ? extras->sink_heads : nullptr;
   p.softcap = extras ? extras->softcap : 0.f;
-  FTK_REQUIRE(!(p.softcap > 0.f) || (!pair && !p.dist_bias && scale > 0.f),
-              "paged_attention_tc: a soft cap goes with one query tile a piece, a positive scale and no distance bias");
+  FTK_REQUIRE(!(p.softcap > 0.f) || (!p.dist_bias && scale > 0.f),
+              "paged_attention_tc: a soft cap goes with a positive scale and no distance bias");
   FTK_REQUIRE(!p.has_sink || form == kTcSingle,
               "paged_attention_tc: of the tcgen05 kernels the one with 128-row tiles takes a softmax sink");
   cudaStream_t s = (cudaStream_t)stream;
   if (p.softcap > 0.f) note_variant(few ? "attention: tcgen05, tiles of at most 16 rows, soft cap"
-                                        : "attention: tcgen05, 128-row query tiles, soft cap");
+                                    : pair ? "attention: tcgen05, two 128-row query tiles per CTA, soft cap"
+                                           : "attention: tcgen05, 128-row query tiles, soft cap");
   else if (p.dist_bias) note_variant(few ? "attention: tcgen05, tiles of at most 16 rows, bias by distance"
                                     : "attention: tcgen05, 128-row query tiles, bias by distance");
   else if (window > 0 || p.has_sink) note_variant("attention: tcgen05, 128-row query tiles, window or sink");
@@ -1099,10 +1168,11 @@ extern "C" int ftk_paged_attention_tc_ex(const void* q, const void* k_slab, cons
                                          int n_segs, const int32_t* items, int n_items, float* part_o, float* part_ml,
                                          int n_slots, void* out, int n_tokens, int n_q_heads, int n_kv_heads,
                                          int head_dim, int page_size, int num_pages, float scale, int window,
-                                         const FtkAttnExtras* extras, int few_rows, void* stream) {
+                                         const FtkAttnExtras* extras, int form, void* stream) {
+  FTK_REQUIRE(form >= 0 && form <= 2, "paged_attention_tc: unknown form %d", form);
   return paged_attention_tc_impl(q, k_slab, v_slab, block_table, bt_stride, seg_info, n_segs, items, n_items, part_o,
                                  part_ml, n_slots, out, n_tokens, n_q_heads, n_kv_heads, head_dim, page_size, num_pages,
-                                 scale, window, stream, few_rows ? kTcFew : kTcSingle, extras);
+                                 scale, window, stream, form == 1 ? kTcFew : form == 2 ? kTcPair : kTcSingle, extras);
 }
 
 extern "C" int ftk_paged_attention_tc_pair(const void* q, const void* k_slab, const void* v_slab,

@@ -153,9 +153,136 @@ __device__ __forceinline__ uint32_t tc_pack(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&t);
 }
 
+// Soft-capped rows of 128 scores, one thread's each.  A capped score never exceeds the cap, so where every 2^(s - cap) is a
+// normal number (soft_cap_bounded, kCapBounded) the cap itself serves as the row's maximum: no pass for the largest score, no
+// rescaling, and the row is read once into registers, where capped_row_small takes the polynomial for all of it; the
+// tiles that have larger scores are read again by capped_row_probs.  (Capping the registers in one of two ways in place
+// took twice as long: the registers of both ways have to meet before the exponentials can start.)  Larger caps (kCapAny)
+// take two passes over TMEM, 32 columns at a time: capped_row_max, then capped_row_probs.  `live` is false for a thread
+// whose row the tile does not have: its scores may be anything, and must not decide how the others' are taken.
+enum CapForm { kCapNone = 0, kCapBounded = 1, kCapAny = 2 };
+// completes a tmem_ld32_start into `v`: nothing that reads it can move in front of the wait
+__device__ __forceinline__ void tmem_ld32_finish(float (&v)[32]) {
+  asm volatile("tcgen05.wait::ld.sync.aligned;"
+               : "+f"(v[0]), "+f"(v[1]), "+f"(v[2]), "+f"(v[3]), "+f"(v[4]), "+f"(v[5]), "+f"(v[6]), "+f"(v[7]),
+                 "+f"(v[8]), "+f"(v[9]), "+f"(v[10]), "+f"(v[11]), "+f"(v[12]), "+f"(v[13]), "+f"(v[14]), "+f"(v[15]),
+                 "+f"(v[16]), "+f"(v[17]), "+f"(v[18]), "+f"(v[19]), "+f"(v[20]), "+f"(v[21]), "+f"(v[22]), "+f"(v[23]),
+                 "+f"(v[24]), "+f"(v[25]), "+f"(v[26]), "+f"(v[27]), "+f"(v[28]), "+f"(v[29]), "+f"(v[30]), "+f"(v[31])
+               :: "memory");
+}
+// The row's largest capped score (exp2 domain, -inf for a row without keys).  Keys outside [lo, hi] do not count;
+// `interior`: no row of the warp has any in this tile.
+__device__ __forceinline__ float capped_row_max(uint32_t s_addr, int key0, int lo, int hi, bool interior, const SoftCap& cap) {
+  float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll 1
+  for (int c = 0; c < 4; c += 2) {
+    float a[32], b[32];
+    tmem_ld32_start(s_addr + 32 * c, a);
+    tmem_ld32_start(s_addr + 32 * c + 32, b);
+    tmem_ld32_finish(a);
+    tmem_ld32_finish(b);
+    const int k0 = key0 + 32 * c;
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+      if (interior || (k0 + i <= hi && k0 + i >= lo)) mx[0] = fmaxf(mx[0], a[i]);
+      if (interior || (k0 + 32 + i <= hi && k0 + 32 + i >= lo)) mx[1] = fmaxf(mx[1], b[i]);
+    }
+  }
+  const float m = fmaxf(mx[0], mx[1]);
+  return m == -INFINITY ? m : capped_any(m, cap);
+}
+// Probabilities of 32 scores (keys k0 and on) relative to `mb` as bfloat16 pairs into 16 TMEM columns; returns their sum.
+__device__ __forceinline__ float capped_probs32(float (&v)[32], uint32_t p_addr, int k0, int lo, int hi, bool interior,
+                                                const SoftCap& cap, bool live, float mb) {
+  if (!interior) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i)
+      if (k0 + i > hi || k0 + i < lo) v[i] = 0.f;
+  }
+  if (all_small(v, cap, live)) {
+    const uint64_t add = pack_f32x2(-mb, -mb);
+#pragma unroll
+    for (int i = 0; i < 32; i += 2) capped_small2(v[i], v[i + 1], cap, add);
+  } else {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) v[i] = capped_any(v[i], cap) - mb;
+  }
+  if (!interior) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i)
+      if (k0 + i > hi || k0 + i < lo) v[i] = -INFINITY;
+  }
+  uint32_t pk[16];
+  uint64_t sum[2] = {0ull, 0ull};
+#pragma unroll
+  for (int i = 0; i < 32; i += 2) {
+    const float p0 = tc_exp2(v[i]), p1 = tc_exp2(v[i + 1]);  // exp2(-inf) = 0 for masked keys
+    sum[(i >> 1) & 1] = add_f32x2(sum[(i >> 1) & 1], pack_f32x2(p0, p1));
+    pk[i >> 1] = tc_pack(p0, p1);
+  }
+  tmem_st16u(p_addr, pk);
+  float s0, s1;
+  unpack_f32x2(add_f32x2(sum[0], sum[1]), s0, s1);
+  return s0 + s1;
+}
+// All 128 of the row, into TMEM columns p_addr .. p_addr + 63 (which may be the first ones of the scores: a run of scores is
+// in registers, and the next one on its way there, before its probabilities are written).
+__device__ __forceinline__ float capped_row_probs(uint32_t s_addr, uint32_t p_addr, int key0, int lo, int hi, bool interior,
+                                                  const SoftCap& cap, bool live, float mb) {
+  float sum = 0.f;
+  float a[32], b[32];
+  tmem_ld32_start(s_addr, a);
+  tmem_ld32_finish(a);
+#pragma unroll 1
+  for (int c = 0; c < 4; c += 2) {
+    tmem_ld32_start(s_addr + 32 * c + 32, b);
+    sum += capped_probs32(a, p_addr + (uint32_t)(16 * c), key0 + 32 * c, lo, hi, interior, cap, live, mb);
+    tmem_ld32_finish(b);
+    if (c == 0) tmem_ld32_start(s_addr + 64, a);
+    sum += capped_probs32(b, p_addr + (uint32_t)(16 * c + 16), key0 + 32 * c + 32, lo, hi, interior, cap, live, mb);
+    if (c == 0) tmem_ld32_finish(a);
+  }
+  return sum;
+}
+
+// kCapBounded, all scores small: the row's 128 scores `v` (keys key0 and on) to probabilities relative to the cap as bfloat16
+// pairs into TMEM columns p_addr .. p_addr + 63; returns their sum.
+__device__ __forceinline__ float capped_row_small(float (&v)[128], uint32_t p_addr, int key0, int lo, int hi, bool interior,
+                                                  const SoftCap& cap) {
+  const uint64_t add = pack_f32x2(-cap.out, -cap.out);
+#pragma unroll
+  for (int i = 0; i < 128; i += 2) capped_small2(v[i], v[i + 1], cap, add);
+  if (!interior) {  // (one branch for all: inside the loop below it would be taken for every pair)
+#pragma unroll
+    for (int i = 0; i < 128; ++i)
+      if (key0 + i > hi || key0 + i < lo) v[i] = -INFINITY;
+  }
+  uint64_t sum[4] = {0ull, 0ull, 0ull, 0ull};
+#pragma unroll
+  for (int c = 0; c < 4; ++c) {
+    uint32_t pk[16];
+#pragma unroll
+    for (int i = 0; i < 32; i += 2) {
+      const float p0 = tc_exp2(v[32 * c + i]), p1 = tc_exp2(v[32 * c + i + 1]);  // exp2(-inf) = 0 for masked keys
+      sum[(i >> 1) & 3] = add_f32x2(sum[(i >> 1) & 3], pack_f32x2(p0, p1));
+      pk[i >> 1] = tc_pack(p0, p1);
+    }
+    tmem_st16u(p_addr + (uint32_t)(16 * c), pk);
+  }
+  float s0, s1;
+  unpack_f32x2(add_f32x2(add_f32x2(sum[0], sum[1]), add_f32x2(sum[2], sum[3])), s0, s1);
+  return s0 + s1;
+}
+// Keys that the row may not read: zero, so that they do not decide anything either.
+__device__ __forceinline__ void clear_outside(float (&v)[128], int key0, int lo, int hi) {
+#pragma unroll
+  for (int i = 0; i < 128; ++i)
+    if (key0 + i > hi || key0 + i < lo) v[i] = 0.f;
+}
+
 // Softmax and epilogue of a tile's rows 0..15 by one warp (the warp of TMEM lanes 0..31), for tiles
 // that have no more rows: thread t has rows t / 4 and t / 4 + 8 and a quarter of their columns.
-template <bool BIASED, bool CAPPED>
+template <bool BIASED, int CAPPED>
 __device__ __forceinline__ void attention_tc_few_rows(const AttnParams& p, uint32_t tmem, int lane, int n_work, int n_rounds,
                                                       uint64_t* s_full, uint64_t* s_empty, uint64_t* p_full,
                                                       uint64_t* pv_done, uint64_t* o_free, volatile int* abortp,
@@ -163,8 +290,7 @@ __device__ __forceinline__ void attention_tc_few_rows(const AttnParams& p, uint3
   const int G = p.G;
   // with a soft cap the scores are scaled while they are capped
   const float sl2 = CAPPED ? 1.f : p.scale * 1.4426950408889634f;
-  const float cap_arg = CAPPED ? 2.f * p.scale / p.softcap * 1.4426950408889634f : 0.f;
-  const float cap_out = p.softcap * 1.4426950408889634f;
+  const SoftCap cap = soft_cap(p.scale, CAPPED ? p.softcap : 1.f);
   const int ra = lane >> 2, rb = ra + 8, cq = lane & 3;
   auto fail = [&](int code) {
     atomicCAS(&g_attn_status[0], 0, code);
@@ -205,8 +331,7 @@ __device__ __forceinline__ void attention_tc_few_rows(const AttnParams& p, uint3
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty[sb]);  // the next product may overwrite this buffer
       if constexpr (CAPPED) {
-#pragma unroll
-        for (int i = 0; i < 64; ++i) v[i] = capped_score(v[i], cap_arg, cap_out);
+        cap_scores(v, cap, ra < R || rb < R);
       }
       const int key0 = it.kb + j * kTcKeys;
       const bool interior = __all_sync(0xffffffffu, key0 + kTcKeys - 1 <= min(hi_a, hi_b));
@@ -385,7 +510,7 @@ __device__ __forceinline__ void attention_tc_few_rows(const AttnParams& p, uint3
   }
 }
 
-template <bool FEW, bool BIASED = false, bool CAPPED = false>
+template <bool FEW, bool BIASED = false, int CAPPED = kCapNone>
 __global__ void __launch_bounds__(kTcThreads)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, AttnParams p) {
@@ -642,9 +767,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     // ------------------------------------------------------------ softmax and epilogue (warps 2..5), one row per thread
     const int quad = warp & 3;
     const int r = quad * 32 + lane;           // row of the tile = TMEM lane
-    const float sl2 = CAPPED ? 1.f : p.scale * 1.4426950408889634f;  // (capped scores are scaled while they are capped)
-    const float cap_arg = CAPPED ? 2.f * p.scale / p.softcap * 1.4426950408889634f : 0.f;
-    const float cap_out = p.softcap * 1.4426950408889634f;
+    const float sl2 = p.scale * 1.4426950408889634f;
+    const SoftCap cap = soft_cap(p.scale, CAPPED ? p.softcap : 1.f);
     const uint32_t lane_addr = tmem + ((uint32_t)(quad * 32) << 16);
     bool ok = true;
     int g0 = 0;  // tiles of the pieces before this one
@@ -665,7 +789,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     // turns a bias into raw-score units (the scores are scaled after the maximum is taken)
     const float* brow = (BIASED && r < R) ? p.dist_bias + (size_t)(kvh * G + r % G) * p.dist_len : nullptr;
     const float unscale = BIASED ? 1.f / p.scale : 0.f;
-    float m_used = -INFINITY, l = 0.f;
+    float m_used = CAPPED == kCapBounded ? cap.out : -INFINITY, l = 0.f;
     for (int j = 0; j < n_tiles && ok; ++j) {
       const int g = g0 + j, sb = g & 1;
       if (!__all_sync(0xffffffffu, mbar_wait(&s_full[sb], (uint32_t)((g >> 1) & 1), abortp))) {
@@ -676,8 +800,23 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       tc_fence_after();
       const uint32_t s_addr = lane_addr + (uint32_t)(sb * kTcKeys);
       const int key0 = it.kb + j * kTcKeys;
-      // the row's 128 scores, in registers for both passes
+      // the row's 128 scores, in registers for both passes (with a soft cap they are read once per pass instead)
       float v0[32], v1[32], v2[32], v3[32];
+      // a tile that every row of the warp reads in full needs no mask (most tiles of a long prompt)
+      const bool interior = __all_sync(0xffffffffu, key0 + kTcKeys - 1 <= hi && key0 >= lo);
+      float tile_bias = 0.f;  // what every score of this tile and row gets added, in the exp2 domain
+      float mx = -INFINITY;
+      float vb[CAPPED == kCapBounded ? 128 : 1];
+      if constexpr (CAPPED == kCapBounded) {
+        tmem_ld32_start(s_addr, vb);
+        tmem_ld32_start(s_addr + 32, vb + 32);
+        tmem_ld32_start(s_addr + 64, vb + 64);
+        tmem_ld32_start(s_addr + 96, vb + 96);
+        tmem_ld_wait();
+        mx = m_used;
+      } else if constexpr (CAPPED == kCapAny) {
+        mx = capped_row_max(s_addr, key0, lo, hi, interior, cap);
+      } else {
       tmem_ld32_start(s_addr, v0);
       tmem_ld32_start(s_addr + 32, v1);
       tmem_ld32_start(s_addr + 64, v2);
@@ -686,17 +825,6 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty[sb]);  // the next product may overwrite this buffer
-      if constexpr (CAPPED) {
-#pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          v0[i] = capped_score(v0[i], cap_arg, cap_out);
-          v1[i] = capped_score(v1[i], cap_arg, cap_out);
-          v2[i] = capped_score(v2[i], cap_arg, cap_out);
-          v3[i] = capped_score(v3[i], cap_arg, cap_out);
-        }
-      }
-      // a tile that every row of the warp reads in full needs no mask (most tiles of a long prompt)
-      const bool interior = __all_sync(0xffffffffu, key0 + kTcKeys - 1 <= hi && key0 >= lo);
       if (!interior) {
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
@@ -706,7 +834,6 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           if (key0 + 96 + i > hi || key0 + 96 + i < lo) v3[i] = -INFINITY;
         }
       }
-      float tile_bias = 0.f;  // what every score of this tile and row gets added, in the exp2 domain
       if constexpr (BIASED) {
         // a tile whose nearest key is as far from every row of the warp as the table's last entry reaches has
         // one bias per row (most tiles of a long prompt); the others look every key's distance up
@@ -724,10 +851,10 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           }
         }
       }
-      float mx = -INFINITY;
 #pragma unroll
       for (int i = 0; i < 32; ++i) mx = fmaxf(fmaxf(mx, v0[i]), fmaxf(v1[i], fmaxf(v2[i], v3[i])));
       mx = fmaf(mx, sl2, tile_bias);  // the scale is positive: the largest score stays the largest
+      }
       // move the running maximum only when it grew by more than 8 (or is not set yet)
       float alpha = 1.f;
       if (mx > m_used + 8.f || (m_used == -INFINITY && mx > -INFINITY)) {
@@ -764,6 +891,19 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       // probabilities as bfloat16 into this row of the A operand in tensor memory: two keys per 32-bit
       // column, 64 columns per buffer behind the output accumulator
       const uint32_t p_addr = lane_addr + (uint32_t)(kTcPCol + sb * (kTcKeys / 2));
+      if constexpr (CAPPED == kCapBounded) {
+        if (!interior) clear_outside(vb, key0, lo, hi);
+        if (all_small(vb, cap, r < R)) sum = capped_row_small(vb, p_addr, key0, lo, hi, interior, cap);
+        else sum = capped_row_probs(s_addr, p_addr, key0, lo, hi, interior, cap, r < R, mb);
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&s_empty[sb]);  // the next product may overwrite this buffer
+      } else if constexpr (CAPPED == kCapAny) {
+        sum = capped_row_probs(s_addr, p_addr, key0, lo, hi, interior, cap, r < R, mb);
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&s_empty[sb]);  // the next product may overwrite this buffer
+      } else {
       auto emit = [&](float (&v)[32], int c) {
         uint32_t pk[16];
 #pragma unroll
@@ -779,6 +919,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       emit(v1, 1);
       emit(v2, 2);
       emit(v3, 3);
+      }
       l += sum;
       tmem_st_wait();
       tc_fence_before();
@@ -879,8 +1020,9 @@ inline int launch_attention_tc(const AttnParams& p, int n_tokens, cudaStream_t s
         cudaFuncSetAttribute(attention_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess ||
         cudaFuncSetAttribute(attention_tc_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess ||
         cudaFuncSetAttribute(attention_tc_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess ||
-        cudaFuncSetAttribute(attention_tc_kernel<false, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess ||
-        cudaFuncSetAttribute(attention_tc_kernel<true, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess)
+        cudaFuncSetAttribute(attention_tc_kernel<false, false, kCapBounded>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess ||
+        cudaFuncSetAttribute(attention_tc_kernel<false, false, kCapAny>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess ||
+        cudaFuncSetAttribute(attention_tc_kernel<true, false, kCapAny>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess)
       return 2;
     configured = true;
   }
@@ -909,9 +1051,11 @@ inline int launch_attention_tc(const AttnParams& p, int n_tokens, cudaStream_t s
   const long long n_work = (long long)p.n_items * p.Hkv;  // one CTA per SM, each takes every sms-th piece of work
   const int grid = (int)(n_work < sms ? n_work : sms);
   if (p.tile_rows == kTcFewRows && p.softcap > 0.f) {
-    FTK_LAUNCH((attention_tc_kernel<true, false, true>), grid, kTcThreads, kTcSmem, s, mq, mk, mv, p);
+    FTK_LAUNCH((attention_tc_kernel<true, false, kCapAny>), grid, kTcThreads, kTcSmem, s, mq, mk, mv, p);
+  } else if (p.softcap > 0.f && soft_cap_bounded(p.softcap)) {
+    FTK_LAUNCH((attention_tc_kernel<false, false, kCapBounded>), grid, kTcThreads, kTcSmem, s, mq, mk, mv, p);
   } else if (p.softcap > 0.f) {
-    FTK_LAUNCH((attention_tc_kernel<false, false, true>), grid, kTcThreads, kTcSmem, s, mq, mk, mv, p);
+    FTK_LAUNCH((attention_tc_kernel<false, false, kCapAny>), grid, kTcThreads, kTcSmem, s, mq, mk, mv, p);
   } else if (p.tile_rows == kTcFewRows && p.dist_bias) {
     FTK_LAUNCH((attention_tc_kernel<true, true>), grid, kTcThreads, kTcSmem, s, mq, mk, mv, p);
   } else if (p.tile_rows == kTcFewRows) {

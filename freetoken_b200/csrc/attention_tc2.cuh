@@ -30,6 +30,7 @@ constexpr int kTc2Threads = 384;                                  // a warpgroup
 constexpr int kTc2RegsFew = 72, kTc2RegsMany = 216;                // of 384 x 168: what 128 threads give, 256 take
 constexpr int kTc2Smem = (2 + 2 * kTc2Stages) * kTcTile + 1024;    // Q_A, Q_B, K and V stages
 
+template <int CAPPED>
 __global__ void __launch_bounds__(kTc2Threads, 1)
 attention_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                      const __grid_constant__ CUtensorMap map_v, AttnParams p) {
@@ -244,6 +245,7 @@ attention_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
     const int quad = warp & 3;
     const int r = quad * 32 + lane;           // row of the tile = TMEM lane
     const float sl2 = p.scale * 1.4426950408889634f;
+    const SoftCap cap = soft_cap(p.scale, CAPPED ? p.softcap : 1.f);
     const uint32_t lane_addr = tmem + ((uint32_t)(quad * 32) << 16);
     const uint32_t s_addr = lane_addr + (uint32_t)(X * kTcKeys);        // scores, then probabilities over their first half
     const uint32_t o_addr = lane_addr + (uint32_t)((2 + X) * kTcKeys);  // output
@@ -262,7 +264,7 @@ attention_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
       const int qpos = r < R ? pos_base + r / G : -1;
       // last key this row may read; rows past the tile's last are never stored and must not hold the others up
       const int hi = r < R ? min(it.ke - 1, qpos) : 0x7fffffff;
-      float m_used = -INFINITY, l = 0.f;
+      float m_used = CAPPED == kCapBounded ? cap.out : -INFINITY, l = 0.f;
       for (int j = 0; j < n_tiles && ok; ++j) {
         const int g = gx + j;
         if (!__all_sync(0xffffffffu, mbar_wait(&s_full[X], (uint32_t)(g & 1), abortp))) {
@@ -272,15 +274,23 @@ attention_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
         }
         tc_fence_after();
         const int key0 = it.kb + j * kTcKeys;
-        // the row's 128 scores, in registers for both passes (the largest, then the probabilities)
+        // a tile that every row of the warp reads in full needs no mask (most tiles of a long prompt)
+        const bool interior = __all_sync(0xffffffffu, key0 + kTcKeys - 1 <= hi);
+        // the row's 128 scores, in registers for both passes (the largest, then the probabilities; with a soft cap they are
+        // read once per pass instead)
         float v[128];
+        float mx;
+        if constexpr (CAPPED == kCapAny) {
+          mx = capped_row_max(s_addr, key0, 0, hi, interior, cap);
+        } else {
         tmem_ld32_start(s_addr, v);
         tmem_ld32_start(s_addr + 32, v + 32);
         tmem_ld32_start(s_addr + 64, v + 64);
         tmem_ld32_start(s_addr + 96, v + 96);
         tmem_ld_wait();
-        // a tile that every row of the warp reads in full needs no mask (most tiles of a long prompt)
-        const bool interior = __all_sync(0xffffffffu, key0 + kTcKeys - 1 <= hi);
+        if constexpr (CAPPED == kCapBounded) {
+          mx = m_used;
+        } else {
         if (!interior) {
 #pragma unroll
           for (int i = 0; i < 128; ++i)
@@ -294,8 +304,10 @@ attention_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
           mx4[2] = fmaxf(mx4[2], v[i + 2]);
           mx4[3] = fmaxf(mx4[3], v[i + 3]);
         }
-        float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+        mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
         mx *= sl2;  // the scale is positive: the largest score stays the largest
+        }
+        }
         // move the running maximum only when it grew by more than 8 (or is not set yet)
         float alpha = 1.f;
         if (mx > m_used + 8.f || (m_used == -INFINITY && mx > -INFINITY)) {
@@ -322,6 +334,13 @@ attention_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
         const float mb = m_used == -INFINITY ? 0.f : m_used;
         float sum = 0.f;
         // probabilities as bfloat16 over the first 64 columns of the scores (which are all in registers by now)
+        if constexpr (CAPPED == kCapBounded) {
+          if (!interior) clear_outside(v, key0, 0, hi);
+          if (all_small(v, cap, r < R)) sum = capped_row_small(v, s_addr, key0, 0, hi, interior, cap);
+          else sum = capped_row_probs(s_addr, s_addr, key0, 0, hi, interior, cap, r < R, mb);
+        } else if constexpr (CAPPED == kCapAny) {
+          sum = capped_row_probs(s_addr, s_addr, key0, 0, hi, interior, cap, r < R, mb);
+        } else {
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
           uint32_t pk[16];
@@ -333,6 +352,7 @@ attention_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
             pk[i >> 1] = tc_pack(p0, p1);
           }
           tmem_st16u(s_addr + (uint32_t)(c * 16), pk);
+        }
         }
         l += sum;
         tmem_st_wait();
@@ -415,7 +435,9 @@ attention_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
 inline int launch_attention_tc2(const AttnParams& p, int n_tokens, cudaStream_t s) {
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(attention_tc2_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kTc2Smem) != cudaSuccess)
+    if (cudaFuncSetAttribute(attention_tc2_kernel<kCapNone>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTc2Smem) != cudaSuccess ||
+        cudaFuncSetAttribute(attention_tc2_kernel<kCapBounded>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTc2Smem) != cudaSuccess ||
+        cudaFuncSetAttribute(attention_tc2_kernel<kCapAny>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTc2Smem) != cudaSuccess)
       return 2;
     configured = true;
   }
@@ -442,7 +464,9 @@ inline int launch_attention_tc2(const AttnParams& p, int n_tokens, cudaStream_t 
   }
   const long long n_work = (long long)p.n_items * p.Hkv;
   const int grid = (int)(n_work < sms ? n_work : sms);
-  FTK_LAUNCH(attention_tc2_kernel, grid, kTc2Threads, kTc2Smem, s, mq, mk, mv, p);
+  if (p.softcap > 0.f && soft_cap_bounded(p.softcap)) FTK_LAUNCH(attention_tc2_kernel<kCapBounded>, grid, kTc2Threads, kTc2Smem, s, mq, mk, mv, p);
+  else if (p.softcap > 0.f) FTK_LAUNCH(attention_tc2_kernel<kCapAny>, grid, kTc2Threads, kTc2Smem, s, mq, mk, mv, p);
+  else FTK_LAUNCH(attention_tc2_kernel<kCapNone>, grid, kTc2Threads, kTc2Smem, s, mq, mk, mv, p);
   return 0;
 }
 

@@ -22,10 +22,14 @@ struct StepArgs {
   int warps_per_group;  // of the register form
 };
 
-constexpr int kStepMaxThreads = 512;
 constexpr int kStepMaxTaps = 16;
 
-__device__ __forceinline__ float gate_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+// (results that are rounded to bfloat16 after the norm take the fast exponential and division, about 2^-21 relative each)
+template <typename T>
+__device__ __forceinline__ float gate_sigmoid(float z) {
+  if constexpr (sizeof(T) == 4) return 1.f / (1.f + expf(-z));
+  else return __fdividef(1.f, 1.f + __expf(-z));
+}
 
 // One element (or four adjacent ones) of the sub-layer's gated result.
 template <typename T, int W>
@@ -80,7 +84,7 @@ __device__ __forceinline__ void gated_result(const FtkStreamStep& p, int src_row
       for (int u = 0; u < W; ++u) b[u] = 0.f;
     }
 #pragma unroll
-    for (int u = 0; u < W; ++u) v[u] *= gate_sigmoid(g[u] + b[u]);
+    for (int u = 0; u < W; ++u) v[u] *= gate_sigmoid<T>(g[u] + b[u]);
   }
 }
 
@@ -140,46 +144,145 @@ __device__ __forceinline__ bool step_state(const FtkStreamStep& p, int row, floa
   return true;
 }
 
-// A row in registers: the block has `groups` teams of whole warps, a team takes one group, a thread at most PER runs
-// of four elements.  Everything the row needs from memory is asked for in the first pass.
-template <typename T, int PER>
-__global__ void __launch_bounds__(kStepMaxThreads) stream_step_regs_kernel(const __grid_constant__ StepArgs a) {
-  pdl_wait();
-  pdl_trigger();
+// A row in registers: the block has `groups` teams of whole warps, a team takes one group, a thread PER runs of four
+// elements.  What a row needs from memory is asked for at once, weights (and with CONV, one token per request, the taps
+// and the request's earlier inputs, which a kernel of an earlier step wrote) before the wait on the kernel before.
+// ROUTED: the result is a sum over expert routes.  TAPS: the tap count where it is four, else 0.
+template <typename T, int PER, bool ROUTED, bool CONV, int TAPS, int MAX_THREADS>
+__global__ void __launch_bounds__(MAX_THREADS) stream_step_regs_kernel(const __grid_constant__ StepArgs a) {
   const FtkStreamStep& p = a.p;
-  __shared__ float red[2][kStepMaxThreads / 32];
-  const int r = blockIdx.x;
-  const int src_row = p.rows ? p.rows[r] : r;
-  const size_t src = (size_t)src_row * p.hidden, dst = (size_t)r * p.hidden;
+  __shared__ float red[2][32];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int team = warp / a.warps_per_group, team_threads = a.warps_per_group * 32;
   const int tl = threadIdx.x - team * team_threads;
   const int quads = a.group_size >> 2;
-  const bool has_y = p.x != nullptr;
-  float2 aux = make_float2(0.f, 1.f);
-  if (has_y && p.aux) aux = *reinterpret_cast<const float2*>(p.aux + (size_t)src_row * 2);
-  float yv[PER][4], zv[PER][4], wp[PER][4], wr[PER][4];
-  float ss = 0.f;
+  const int r = blockIdx.x;
+  int at[PER];   // first element of each run
+  bool in[PER];
 #pragma unroll
   for (int q = 0; q < PER; ++q) {
     const int quad = q * team_threads + tl;
+    in[q] = quad < quads;
+    at[q] = team * a.group_size + (in[q] ? quad * 4 : 0);
+  }
+  float yv[PER][4], zv[PER][4], wp[PER][4], wr[PER][4], gb[PER][4];
+  float cw[CONV && TAPS == 4 ? PER : 1][4][4], old[CONV && TAPS == 4 ? PER : 1][3][4];
+  if (p.post_w) {
 #pragma unroll
-    for (int u = 0; u < 4; ++u) yv[q][u] = zv[q][u] = wp[q][u] = wr[q][u] = 0.f;
-    if (quad >= quads) continue;
-    const int i = team * a.group_size + quad * 4;
-    Vec4<float>::load(p.residual + src + i, zv[q]);
-    if (p.pre_w) Vec4<float>::load(p.pre_w + i, wr[q]);
-    if (p.vec) {
+    for (int q = 0; q < PER; ++q) Vec4<float>::load(p.post_w + at[q], wp[q]);
+  }
+  if (p.pre_w) {
+#pragma unroll
+    for (int q = 0; q < PER; ++q) Vec4<float>::load(p.pre_w + at[q], wr[q]);
+  }
+#pragma unroll
+  for (int q = 0; q < PER; ++q) gb[q][0] = gb[q][1] = gb[q][2] = gb[q][3] = 0.f;
+  if (p.gate_bias) {
+#pragma unroll
+    for (int q = 0; q < PER; ++q) Vec4<float>::load(p.gate_bias + at[q], gb[q]);
+  }
+  float* st = nullptr;
+  int before = 0;
+  bool live = false;
+  if constexpr (CONV) live = step_state(p, r, st, before);
+  if constexpr (CONV && TAPS == 4) {
+#pragma unroll
+    for (int q = 0; q < PER; ++q)
+#pragma unroll
+      for (int u = 0; u < 4; ++u) Vec4<float>::load(p.conv_w + (size_t)(at[q] + u) * 4, cw[q][u]);
+#pragma unroll
+    for (int q = 0; q < PER; ++q)
+#pragma unroll
+      for (int j = 0; j < 3; ++j) {
+        if (live && 3 - j <= before) Vec4<float>::load(st + (size_t)j * p.hidden + at[q], old[q][j]);
+        else old[q][j][0] = old[q][j][1] = old[q][j][2] = old[q][j][3] = 0.f;
+      }
+  }
+  pdl_wait();
+  pdl_trigger();
+  const int src_row = p.rows ? p.rows[r] : r;
+  const size_t src = (size_t)src_row * p.hidden, dst = (size_t)r * p.hidden;
+  const bool has_y = p.x != nullptr;
+  float2 aux = make_float2(0.f, 1.f);
+  if (ROUTED && p.aux) aux = *reinterpret_cast<const float2*>(p.aux + (size_t)src_row * 2);
+#pragma unroll
+  for (int q = 0; q < PER; ++q) Vec4<float>::load(p.residual + src + at[q], zv[q]);
+  float ss = 0.f;
+  if (has_y) {
+    const T* x = (const T*)p.x;
+    float gv[PER][4];
+    if (p.gate) {
+#pragma unroll
+      for (int q = 0; q < PER; ++q) Vec4<T>::load((const T*)p.gate + src + at[q], gv[q]);
+    }
+    if constexpr (ROUTED) {
+#pragma unroll
+      for (int q = 0; q < PER; ++q) yv[q][0] = yv[q][1] = yv[q][2] = yv[q][3] = 0.f;
+      constexpr int J = PER <= 1 ? 8 : PER <= 2 ? 4 : 2;  // routes whose rows are asked for before the first is added
+      for (int j0 = 0; j0 < p.top_k; j0 += J) {            // route order
+        float y[J][PER][4];
+        int pos[J];
+#pragma unroll
+        for (int j = 0; j < J; ++j) {
+          pos[j] = j0 + j < p.top_k ? __ldg(p.route_pos + (size_t)src_row * p.top_k + j0 + j) : -1;
+          if (pos[j] >= p.n_routes) pos[j] = -1;
+        }
+#pragma unroll
+        for (int j = 0; j < J; ++j)
+#pragma unroll
+          for (int q = 0; q < PER; ++q) {
+            if (pos[j] >= 0) Vec4<T>::load(x + (size_t)pos[j] * p.hidden + at[q], y[j][q]);
+            else y[j][q][0] = y[j][q][1] = y[j][q][2] = y[j][q][3] = 0.f;
+          }
+#pragma unroll
+        for (int j = 0; j < J; ++j)
+#pragma unroll
+          for (int q = 0; q < PER; ++q)
+#pragma unroll
+            for (int u = 0; u < 4; ++u) yv[q][u] += y[j][q][u];
+      }
+      if (p.passed && aux.x != 0.f) {
+#pragma unroll
+        for (int q = 0; q < PER; ++q) {
+          float y[4];
+          Vec4<T>::load((const T*)p.passed + src + at[q], y);
+#pragma unroll
+          for (int u = 0; u < 4; ++u) yv[q][u] = fmaf(aux.x, y[u], yv[q][u]);
+        }
+      }
+      if (p.shared) {
+#pragma unroll
+        for (int q = 0; q < PER; ++q) {
+          float y[4];
+          Vec4<T>::load((const T*)p.shared + src + at[q], y);
+#pragma unroll
+          for (int u = 0; u < 4; ++u) yv[q][u] = fmaf(aux.y, y[u], yv[q][u]);
+        }
+      }
+    } else {
+#pragma unroll
+      for (int q = 0; q < PER; ++q) Vec4<T>::load(x + src + at[q], yv[q]);
+    }
+    if (p.gate) {
+#pragma unroll
+      for (int q = 0; q < PER; ++q)
+#pragma unroll
+        for (int u = 0; u < 4; ++u) yv[q][u] *= gate_sigmoid<T>(gv[q][u] + gb[q][u]);
+    }
+#pragma unroll
+    for (int q = 0; q < PER; ++q)
+      if (in[q]) {
+#pragma unroll
+        for (int u = 0; u < 4; ++u) ss = fmaf(yv[q][u], yv[q][u], ss);
+      }
+  }
+  if (p.vec) {
+#pragma unroll
+    for (int q = 0; q < PER; ++q) {
       float v[4];
-      Vec4<float>::load(p.vec + i, v);
+      Vec4<float>::load(p.vec + at[q], v);
 #pragma unroll
       for (int u = 0; u < 4; ++u) zv[q][u] += v[u];
-    }
-    if (has_y) {
-      Vec4<float>::load(p.post_w + i, wp[q]);
-      gated_result<T, 4>(p, src_row, src, i, aux, yv[q]);
-#pragma unroll
-      for (int u = 0; u < 4; ++u) ss = fmaf(yv[q][u], yv[q][u], ss);
     }
   }
   auto team_sum = [&](float v, float* scratch) {
@@ -201,24 +304,18 @@ __global__ void __launch_bounds__(kStepMaxThreads) stream_step_regs_kernel(const
   const bool changed = (has_y || p.vec) && !p.rows;
 #pragma unroll
   for (int q = 0; q < PER; ++q) {
-    const int quad = q * team_threads + tl;
-    if (quad >= quads) continue;
-    const int i = team * a.group_size + quad * 4;
+    if (!in[q]) continue;
 #pragma unroll
     for (int u = 0; u < 4; ++u) ss2 = fmaf(zv[q][u], zv[q][u], ss2);
-    if (changed) Vec4<float>::store(p.residual + src + i, zv[q]);
-    if (p.raw_out) Vec4<T>::store((T*)p.raw_out + (size_t)r * p.raw_stride + i, zv[q]);
+    if (changed) Vec4<float>::store(p.residual + src + at[q], zv[q]);
+    if (p.raw_out) Vec4<T>::store((T*)p.raw_out + (size_t)r * p.raw_stride + at[q], zv[q]);
   }
   if (!p.pre_w) return;
   const float inv = rsqrtf(team_sum(ss2, red[1]) / (float)a.group_size + p.pre_eps);
-  float* st;
-  int before;
-  const bool live = step_state(p, r, st, before);
 #pragma unroll
   for (int q = 0; q < PER; ++q) {
-    const int quad = q * team_threads + tl;
-    if (quad >= quads) continue;
-    const int i = team * a.group_size + quad * 4;
+    if (!in[q]) continue;
+    const int i = at[q];
     float y[4];
 #pragma unroll
     for (int u = 0; u < 4; ++u) y[u] = zv[q][u] * inv * wr[q][u];
@@ -226,7 +323,25 @@ __global__ void __launch_bounds__(kStepMaxThreads) stream_step_regs_kernel(const
 #pragma unroll
     for (int u = 0; u < 4; ++u) y[u] = to_float(from_float<T>(y[u]));
     if (p.out) Vec4<T>::store((T*)p.out + dst + i, y);
-    if (p.conv_w) step_conv<T, 4>(p, r, dst, i, y, live, st, before);
+    if constexpr (CONV && TAPS == 4) {
+      float acc[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        acc[u] = fmaf(cw[q][u][3], y[u], y[u]);
+#pragma unroll
+        for (int j = 0; j < 3; ++j) acc[u] = fmaf(cw[q][u][j], old[q][j][u], acc[u]);
+        acc[u] = to_float(from_float<T>(acc[u]));
+      }
+      if (live) {
+        Vec4<float>::store(st + i, old[q][1]);
+        Vec4<float>::store(st + p.hidden + i, old[q][2]);
+        Vec4<float>::store(st + 2 * (size_t)p.hidden + i, y);
+      }
+      Vec4<T>::store((T*)p.conv_out + dst + i, acc);
+      if (p.conv_out_f32) Vec4<float>::store(p.conv_out_f32 + dst + i, acc);
+    } else if constexpr (CONV) {
+      step_conv<T, 4>(p, r, dst, i, y, live, st, before);
+    }
   }
 }
 
@@ -316,32 +431,53 @@ extern "C" int ftk_stream_step(const FtkStreamStep* args, void* stream) {
   auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
   const bool vec = a.group_size % 4 == 0 && al16(p.residual) && al16(p.x) && al16(p.passed) && al16(p.shared) && al16(p.gate) &&
                    al16(p.gate_bias) && al16(p.post_w) && al16(p.pre_w) && al16(p.vec) && al16(p.out) && al16(p.norm_f32) &&
-                   al16(p.conv_out) && al16(p.conv_out_f32) && al16(p.state) && (p.raw_stride * item) % (4 * item) == 0 &&
+                   al16(p.conv_out) && al16(p.conv_out_f32) && al16(p.state) && al16(p.conv_w) && (p.raw_stride * item) % (4 * item) == 0 &&
                    (reinterpret_cast<uintptr_t>(p.raw_out) % (4 * item)) == 0;
   cudaStream_t s = (cudaStream_t)stream;
-  if (vec && p.groups <= kStepMaxThreads / 32) {
-    const int quads = a.group_size / 4, most = kStepMaxThreads / 32 / p.groups;
-    int w = (quads + 63) / 64;                  // about two runs of four a thread
+  // teams of warps: steps of single tokens spread a row over up to 768 threads (few rows, each as soon as possible), others
+  // over up to 256 (many rows side by side)
+  const bool conv = p.conv_w != nullptr, routed = p.route_pos != nullptr;
+  const int quads = a.group_size / 4;
+  auto shape = [&](int max_threads) {  // (warps a group, runs a thread)
+    const int most = max_threads / 32 / p.groups;
+    int w = conv ? (quads + 31) / 32 : (quads + 95) / 96;
     w = w < 1 ? 1 : (w > most ? most : w);
     a.warps_per_group = w;
-    const int per = (quads + w * 32 - 1) / (w * 32);
-    const int threads = w * 32 * p.groups;
-    if (per <= 4) {
-      note_variant("stream step: rows in registers");
-#define FTK_STEP(TY, N) FTK_LAUNCH((stream_step_regs_kernel<TY, N>), p.n_rows, threads, 0, s, a)
-#define FTK_STEP_PER(TY)                                   \
-      do {                                                 \
-        if (per <= 1) FTK_STEP(TY, 1);                     \
-        else if (per <= 2) FTK_STEP(TY, 2);                \
-        else FTK_STEP(TY, 4);                              \
-      } while (0)
-      if (p.dtype == FTK_F32) FTK_STEP_PER(float);
-      else FTK_STEP_PER(__nv_bfloat16);
-#undef FTK_STEP_PER
+    return w < 1 ? 1 << 20 : (quads + w * 32 - 1) / (w * 32);
+  };
+  int per = vec && p.groups <= 24 ? shape(conv ? 768 : 256) : 1 << 20;
+  bool wide = conv;
+  if (!conv && per > 4 && vec && p.groups <= 24) {
+    per = shape(768);
+    wide = true;
+  }
+  if (per <= 4 && !(wide && per > 2)) {
+    const int threads = a.warps_per_group * 32 * p.groups;
+    note_variant(conv ? "stream step: rows in registers, convolution" : "stream step: rows in registers");
+#define FTK_STEP(TY, N, RT, CV, TP, MT) FTK_LAUNCH((stream_step_regs_kernel<TY, N, RT, CV, TP, MT>), p.n_rows, threads, 0, s, a)
+#define FTK_STEP_R(TY, N, CV, TP, MT)            \
+    do {                                         \
+      if (routed) FTK_STEP(TY, N, true, CV, TP, MT); \
+      else FTK_STEP(TY, N, false, CV, TP, MT);   \
+    } while (0)
+#define FTK_STEP_ALL(TY)                                                   \
+    do {                                                                   \
+      if (conv && p.taps == 4 && per <= 1) FTK_STEP_R(TY, 1, true, 4, 768); \
+      else if (conv && per <= 1) FTK_STEP_R(TY, 1, true, 0, 768);          \
+      else if (conv) FTK_STEP_R(TY, 2, true, 0, 768);                      \
+      else if (wide) FTK_STEP_R(TY, 2, false, 0, 768);                     \
+      else if (per <= 1) FTK_STEP_R(TY, 1, false, 0, 256);                 \
+      else if (per <= 2) FTK_STEP_R(TY, 2, false, 0, 256);                 \
+      else if (per <= 3) FTK_STEP_R(TY, 3, false, 0, 256);                 \
+      else FTK_STEP_R(TY, 4, false, 0, 256);                               \
+    } while (0)
+    if (p.dtype == FTK_F32) FTK_STEP_ALL(float);
+    else FTK_STEP_ALL(__nv_bfloat16);
+#undef FTK_STEP_ALL
+#undef FTK_STEP_R
 #undef FTK_STEP
-      FTK_LAUNCH_CHECK("stream_step");
-      return 0;
-    }
+    FTK_LAUNCH_CHECK("stream_step");
+    return 0;
   }
   a.warps_per_group = 1;
   const size_t smem = ((size_t)2 * p.hidden + p.groups) * sizeof(float);

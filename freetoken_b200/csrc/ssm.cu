@@ -13,7 +13,7 @@
 
 namespace ftk {
 
-constexpr int kCaTile = 32;      // tokens per tile (at least taps - 1)
+constexpr int kCaTile = 16;      // tokens per tile (at least taps - 1)
 constexpr int kCaMaxTaps = 16;
 constexpr int kCaThreads = 128;  // four channels a thread
 

@@ -16,6 +16,8 @@
     python -m freetoken_b200.kernels.microbench attention --prefill 2048 --tied --kv-heads 1 --window 1024 --head-sinks
     python -m freetoken_b200.kernels.microbench nusudra --tokens 2048 [--batch 8]
     python -m freetoken_b200.kernels.microbench attention --prefill 2048 --dist-bias 2048 --head-sinks
+    python -m freetoken_b200.kernels.microbench vodatar --tokens 2048 [--batch 8]
+    python -m freetoken_b200.kernels.microbench attention --prefill 2048 --q-heads 96 --softcap 30 --maps 2
 
 Each case allocates its inputs once (larger than L2 where the real workload is), warms up, then
 times ``--iters`` launches with CUDA events and prints one JSON line: time, the bytes the kernel has
@@ -148,6 +150,10 @@ def bench_attention(a) -> dict:
     if getattr(a, "head_sinks", False):  # a logit per query head
         sink = torch.randn(Hq, device=dev, generator=g)
     special = window is not None or sink is not None  # of the tcgen05 kernels the one with 128-row tiles takes these
+    cap = float(getattr(a, "softcap", 0) or 0) or None  # scores become cap * tanh(score / cap)
+    maps = max(1, int(getattr(a, "maps", 1) or 1))  # query rows are zero outside a map's place: a part of Q K^T does no work
+    if maps > 1:
+        q.view(q0, Hq // maps, maps, maps, D // maps).mul_(torch.eye(maps, device=dev, dtype=q.dtype)[None, None, :, :, None])
     no_tc = a.no_tc
     tile = 128 if (a.prefill >= 128 and not no_tc and ops.attention_tc_fits(D, P, G)) else 64
     if tile == 128 and a.pair and bias is None and not special:
@@ -171,13 +177,13 @@ def bench_attention(a) -> dict:
         pm = torch.empty(plan.n_slots, Hkv, tile, 2, dtype=torch.float32, device=dev)
     out = torch.empty_like(q)
     us = _time(lambda: ops.paged_attention(q, ks, vs, bt, seg, len(segs), items, plan.n_items, po, pm, out, tile,
-                                           D ** -0.5, window, few_rows=few_rows, dist_bias=bias, sink=sink), a.iters,
+                                           D ** -0.5, window, few_rows=few_rows, dist_bias=bias, sink=sink, softcap=cap), a.iters,
                a.warmup, a.profile)
     seen = [(ql, kv if window is None else min(kv, window - 1 + ql)) for ql, kv in segs]  # keys a segment's queries can see
     kv_bytes = sum(kv for _, kv in seen) * Hkv * D * 2 * (1 if tied else 2)
     pairs = lambda ql, kv: sum(min(kv - ql + t + 1, window or (1 << 60)) for t in range(ql))  # noqa: E731  (query, key) pairs
-    flops = sum(4 * pairs(ql, kv) * Hq * D for ql, kv in segs)
-    return {"us": round(us, 2), "tile_rows": tile, "tied": tied, "dist_bias": n_bias, "window": window, "sink": sink is not None,
+    flops = sum((2 + 2 / maps) * pairs(ql, kv) * Hq * D for ql, kv in segs)
+    return {"us": round(us, 2), "tile_rows": tile, "tied": tied, "dist_bias": n_bias, "window": window, "sink": sink is not None, "softcap": cap,
             "items": plan.n_items,
             "est_us": None if plan.est_us is None else round(plan.est_us, 1), "kv_bytes": kv_bytes, "gbs": round(kv_bytes / us / 1e3, 1),
             "hbm_frac": round(kv_bytes / us / 1e3 / HBM_GBS, 3), "tflops": round(flops / us / 1e6, 1),
@@ -492,6 +498,96 @@ def bench_nusudra(a) -> dict:
     return results
 
 
+def bench_vodatar(a) -> dict:
+    """The kernels that the Vodatar layers add around the library products: the pass over the stream (gate, group norm,
+    sum, group norm, and with one token per request the short convolution), the short convolution of a portion, the
+    convolution, rotation and cache write of two-map heads, the difference of the maps, and the routing with identity
+    experts and a gated shared expert.  Attention is ``attention --q-heads 2H --softcap C --maps 2``."""
+    dev = "cuda"
+    T, C, H, G, D, Dv, k, taps = a.tokens, a.hidden, a.heads, a.kv_heads, a.dim, a.vdim, a.top_k, a.taps
+    decode = a.batch > 0
+    segs = [(1, a.context)] * a.batch if decode else [(T, T)]
+    T = sum(q for q, _ in segs)
+    g = torch.Generator(device=dev).manual_seed(0)
+    bf = torch.bfloat16
+    info, q0 = [], 0
+    for ql, kv in segs:
+        info.append([q0, ql, kv, 0])
+        q0 += ql
+    seg = torch.tensor(info, dtype=torch.int32, device=dev)
+    slots = torch.arange(1, len(segs) + 1, dtype=torch.int32, device=dev)
+    n_slots, S = len(segs) + 1, len(segs)
+    results = {}
+
+    def add(name, fn, nbytes):
+        us = _time(fn, a.iters, a.warmup, a.profile)
+        results[name] = {"us": round(us, 2), "bytes": nbytes, "gbs": round(nbytes / us / 1e3, 1),
+                         "hbm_frac": round(nbytes / us / 1e3 / HBM_GBS, 3)}
+
+    res = torch.randn(T, C, device=dev, generator=g)
+    rnd = lambda *s: torch.randn(*s, device=dev, generator=g).to(bf)  # noqa: E731
+    y, gate, h, u, shared, passed = rnd(T, C), rnd(T, C), rnd(T, C), rnd(T, C), rnd(T, C), rnd(T, C)
+    u32 = torch.empty(T, C, device=dev)
+    w, bias = torch.ones(C, device=dev), torch.zeros(C, device=dev)
+    cw = torch.randn(C, taps, device=dev, generator=g) * 0.3
+    cstate = torch.zeros(n_slots, max(taps - 1, 1), C, device=dev)[:, : taps - 1]
+    cst = cstate if taps > 1 else None
+    common = dict(groups=a.groups, gate=gate, gate_bias=bias, post_weight=w, post_eps=1e-6, pre_weight=w, pre_eps=1e-6, out=h)
+    state_bytes = 2 * S * (taps - 1) * C * 4
+    conv = dict(conv=(cw, cst, slots, seg, u, u32)) if decode else {}
+    extra = T * C * (2 + 4) + state_bytes + C * taps * 4 if decode else 0
+    add("stream_step (gate, norm, sum, norm" + ("; convolution" if decode else "") + ")",
+        lambda: ops.stream_step(res, x=y, **common, **conv), T * C * (4 + 4 + 2 + 2 + 2) + extra)
+    rows = rnd(T * k, C)
+    pos = torch.randperm(T * k, device=dev, generator=g).to(torch.int32)
+    n_id = a.identity
+    real = torch.rand(T * k, device=dev, generator=g) >= n_id / (a.experts + n_id)
+    pos = torch.where(real, pos, torch.full_like(pos, -1)).view(T, k)
+    aux = torch.rand(T, 2, device=dev, generator=g) * (~real.view(T, k)).any(1, keepdim=True)
+    n_rows, n_pass = int(real.sum()), int((aux[:, 0] != 0).sum())
+    add("stream_step (the same over expert routes, identity experts and a gated shared expert)",
+        lambda: ops.stream_step(res, x=rows, routed=(pos, k, shared, aux, passed), **common, **conv),
+        T * C * (4 + 4 + 2 + 2 + 2) + (n_rows + n_pass) * C * 2 + extra)
+    if not decode:
+        add("conv_act (the sub-layer's input, no bias, no activation)",
+            lambda: ops.conv_act(h, cw, None, None, cst, slots, seg, S, u), T * C * 4)
+    ch = (H + G) * 2 * D + G * Dv
+    P = -(-max(2 * D, Dv) // 16) * 16
+    proj, pw = rnd(T, ch), torch.randn(ch, taps, device=dev, generator=g) * 0.3
+    pst = torch.zeros(n_slots, taps - 1, ch, device=dev) if taps > 1 else None
+    page = 16
+    n_pages = sum(-(-kv // page) for _, kv in segs) + 1
+    ks, vs = (torch.zeros(n_pages, G, page, P, dtype=bf, device=dev) for _ in range(2))
+    positions = torch.cat([torch.arange(kv - ql, kv) for ql, kv in segs]).to(torch.int32).to(dev)
+    smap = (torch.arange(T, device=dev) % (n_pages * page - page) + page).to(torch.int32)
+    table = torch.randn(int(max(kv for _, kv in segs)), D, device=dev, generator=g)
+    q = torch.empty(T, 2 * H, P, dtype=bf, device=dev)
+    add("conv_rope_store (convolution, rotation, cache write of two-map heads)",
+        lambda: ops.conv_rope_store(proj, pw, pst, slots, seg, S, H, G, 2, D, Dv, D, True, positions, table, q, ks, vs, smap),
+        T * (ch + 2 * H * P + 2 * G * P) * 2 + (2 * S * (taps - 1) * ch * 4 if decode else 0))
+    lam, o = torch.full((1,), 0.3, device=dev), torch.empty(T, H, Dv, dtype=bf, device=dev)
+    add("diff_heads (the maps' difference, normed)", lambda: ops.diff_heads(q, lam, 1e-6, 0.7, o), T * H * (2 * P + Dv) * 2)
+    E = a.experts + n_id
+    gw = torch.randn(E + 1, C, device=dev, generator=g) * C ** -0.5
+    corr = torch.randn(E, device=dev, generator=g) * 0.05
+    ids, wts = torch.empty(T, k, dtype=torch.int32, device=dev), torch.empty(T, k, device=dev)
+    auxo = torch.empty(T, 2, device=dev)
+    logits = torch.randn(T, E + 1, device=dev, generator=g)
+    if ops.moe_route_fits(T, C, E, k):
+        x32 = torch.randn(T, C, device=dev, generator=g)
+        sort = (torch.empty(a.experts, dtype=torch.int32, device=dev), torch.empty(a.experts + 1, dtype=torch.int32, device=dev),
+                torch.empty(T * k, dtype=torch.int32, device=dev), torch.empty(T * k, dtype=torch.int32, device=dev))
+        add("moe_route (identity experts, shared gate)",
+            lambda: ops.moe_route(x32, gw, corr, k, "softmax", 1.0, logits, ids, wts, *sort, n_extra=1, n_real=a.experts, aux=auxo),
+            (E + 1 + T) * C * 4)
+    else:
+        add("router_topk (identity experts, shared gate)",
+            lambda: ops.router_topk(logits, corr, k, "softmax", 1.0, ids, wts, n_extra=1, n_real=a.experts, aux=auxo),
+            T * (E + 1) * 4)
+    results["status"] = ops.read_status()
+    return results
+
+
 def bench_few(a) -> dict:
     """The few-token kernels (``csrc/gemv.cu``) at the headline sizes: the qkv and output projections of
     ``--tokens`` tokens, and the routed gate/up and down products of their routes.  Six copies of the dense
@@ -607,7 +703,7 @@ def bench_sample(a) -> dict:
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="microbench")
     sub = ap.add_subparsers(dest="case", required=True)
-    for name in ("moe", "attention", "sample", "sparse", "few", "rows", "gla", "kekopel", "nusudra"):
+    for name in ("moe", "attention", "sample", "sparse", "few", "rows", "gla", "kekopel", "nusudra", "vodatar"):
         p = sub.add_parser(name)
         p.add_argument("--iters", type=int, default=20)
         p.add_argument("--warmup", type=int, default=5)
@@ -639,6 +735,8 @@ def main(argv=None) -> int:
             p.add_argument("--tied", action="store_true", help="the values are the keys (one slab)")
             p.add_argument("--dist-bias", type=int, default=0, help="entries per head of a bias by distance (0 = none)")
             p.add_argument("--window", type=int, default=0, help="a sliding window of this many tokens (0 = none)")
+            p.add_argument("--softcap", type=float, default=0.0, help="scores become cap * tanh(score / cap) (0 = as they are)")
+            p.add_argument("--maps", type=int, default=1, help="softmax maps a head: query rows that are zero outside their map")
             p.add_argument("--sink", action="store_true", help="a sink of logit 0 in the softmax's denominator")
             p.add_argument("--head-sinks", action="store_true", help="a sink with a logit of its own per query head")
         elif name == "rows":
@@ -678,6 +776,20 @@ def main(argv=None) -> int:
             p.add_argument("--groups", type=int, default=8)
             p.add_argument("--taps", type=int, default=4)
             p.add_argument("--chunk", type=int, default=64)
+        elif name == "vodatar":
+            p.add_argument("--tokens", type=int, default=2048)
+            p.add_argument("--batch", type=int, default=0, help="requests with one token each instead of one portion")
+            p.add_argument("--context", type=int, default=2048)
+            p.add_argument("--hidden", type=int, default=3072)
+            p.add_argument("--groups", type=int, default=8)
+            p.add_argument("--taps", type=int, default=4)
+            p.add_argument("--heads", type=int, default=48)
+            p.add_argument("--kv-heads", type=int, default=8)
+            p.add_argument("--dim", type=int, default=64)
+            p.add_argument("--vdim", type=int, default=128)
+            p.add_argument("--experts", type=int, default=64)
+            p.add_argument("--identity", type=int, default=8)
+            p.add_argument("--top-k", type=int, default=8)
         elif name == "few":
             p.add_argument("--tokens", type=int, default=1)
             p.add_argument("--hidden", type=int, default=3072)
@@ -715,7 +827,7 @@ def main(argv=None) -> int:
             p.add_argument("--temperature", type=float, default=0.0)
     a = ap.parse_args(argv)
     res = {"moe": bench_moe, "attention": bench_attention, "sample": bench_sample, "sparse": bench_sparse, "few": bench_few,
-           "rows": bench_rows, "gla": bench_gla, "kekopel": bench_kekopel, "nusudra": bench_nusudra}[a.case](a)
+           "rows": bench_rows, "gla": bench_gla, "kekopel": bench_kekopel, "nusudra": bench_nusudra, "vodatar": bench_vodatar}[a.case](a)
     print(json.dumps({"case": a.case, **{k: v for k, v in vars(a).items() if k != "case"}, "result": res}))
     return 0
 

@@ -501,8 +501,7 @@ def paged_attention(q: torch.Tensor, k_slab: torch.Tensor, v_slab: torch.Tensor,
     one slab for keys and values, and a sink together with a bias by distance.
 
     ``softcap`` (positive, or None): scaled scores ``s`` become ``softcap * tanh(s / softcap)`` before the softmax.  Not with
-    block selection or a bias by distance; of the tcgen05 kernels the ones with one query tile a piece (128 rows, or at most
-    16) take it.
+    block selection or a bias by distance; every tcgen05 form takes it.
     """
     softcap = 0.0 if softcap is None else float(softcap)
     if softcap < 0 or (softcap and (sel is not None or dist_bias is not None)):
@@ -533,8 +532,6 @@ def paged_attention(q: torch.Tensor, k_slab: torch.Tensor, v_slab: torch.Tensor,
         if sel is not None or q.dtype != torch.bfloat16:
             raise KernelError("paged_attention: the tcgen05 kernels take bfloat16 without block selection")
         if window or sink is not None or dist_bias is not None or softcap:
-            if softcap and tile_rows == 256:
-                raise KernelError("paged_attention: of the tcgen05 kernels the ones with one query tile a piece take a soft cap")
             # the form with one 128-row query tile a piece takes a window, a sink and a bias by distance (a bias not
             # together with a window); the form for tiles of at most 16 rows takes the bias alone
             if (window or sink is not None) and (tile_rows != 128 or few_rows):
@@ -552,7 +549,7 @@ def paged_attention(q: torch.Tensor, k_slab: torch.Tensor, v_slab: torch.Tensor,
                 _dev(items, "items", torch.int32), n_items,
                 _dev(part_o, "part_o", torch.float32), _dev(part_ml, "part_ml", torch.float32), n_slots,
                 _dev(out, "out"), T, Hq, Hkv, D, P, pages, float(scale), int(window) if window else 0, ctypes.byref(ex),
-                1 if few_rows else 0, _stream()),
+                1 if few_rows else 2 if tile_rows == 256 else 0, _stream()),
                 f"paged_attention (tcgen05, {what})", 2 if n_slots else 1)
             return
         fn = (_lib().ftk_paged_attention_tc_few if few_rows else

@@ -28,7 +28,7 @@ from ..config.spec import PagedKVNeed, ParamSpec, PartSpec, StateNeed
 from ..engine.attention_plan import DEAL_MOST_PIECES
 from ..errors import ConfigError
 from ..kernels import ops
-from .attention import attention_kernel_form
+from .attention import TC_PAIR_MIN_TOKENS_LONG, attention_kernel_form
 from .base import MIXERS, BuildEnv, Mixer, StepState
 from .rope import shared_position
 
@@ -112,10 +112,9 @@ class DifferentialAttention(Mixer):
 
     # ------------------------------------------------------------------ step
     def kernel_form(self, decode_only: bool, n_tokens: int = 0, page_size: int = 0, longest_span: int = 0):
-        # (of the tcgen05 kernels the ones with one query tile a piece take a soft cap)
         sized = self.kv_split == 1
         return attention_kernel_form(self.env.dtype, decode_only, self.plan_group, n_tokens, self.pad_dim if sized else 0,
-                                     page_size, None, longest_span, one_tile_only=True)
+                                     page_size, None, longest_span)
 
     def plan_key(self, decode_only: bool = False, n_tokens: int = 0, page_size: int = 0, longest_span: int = 0):
         rows, few = self.kernel_form(decode_only, n_tokens, page_size, longest_span)
@@ -125,6 +124,10 @@ class DifferentialAttention(Mixer):
         n_tokens = sum(q for q, _ in builder.seg_lens)
         page_size = builder.engine.config.page_size if builder.engine is not None else 0
         rows, few = self.kernel_form(builder.decode_only, n_tokens, page_size, builder.longest_span())
+        if rows >= 128 and not few and not builder.decode_only and n_tokens >= TC_PAIR_MIN_TOKENS_LONG \
+                and hasattr(builder, "cheaper_attention_rows"):
+            # one or two query tiles a piece: whichever work list the kernel is estimated to get through sooner
+            rows = builder.cheaper_attention_rows(self.plan_group, None, self.plan_kv_heads, self.pad_dim)
         self._step_plan = builder.attention_plan(self.plan_group, rows, None, self.plan_kv_heads, self.pad_dim, few)
 
     def forward(self, h: torch.Tensor, step: StepState, cache: Any, writes_cache: bool) -> torch.Tensor:

@@ -17,6 +17,9 @@ named by a table over token ids) and Pabavik (layers normed on both sides of eve
 with a sink and an output gate, gated linear attention and attention over an earlier layer's cache in turns) and
 Kekopel (a short convolution in front of every sub-layer, norms behind them, a mix over all layers' outputs; latent
 attention with a learned sink per head and matrix memory in turns; dense and input-weighted expert feed-forwards)
+and Nusudra (several residual streams, latent attention, attention beside Mamba-2, the gated delta rule) and Vodatar
+(norms over groups on both sides of every sub-layer, a short convolution in front and a gate behind, differential
+attention with a soft cap and latent attention in turns, identity experts and a gated shared expert, a looped range)
 beside MiniMax-M3 at equal layer sizes, all with random weights: a
 2 048-token prompt in one step and decode steps of eight requests at 2 048 tokens of context, at a few
 sizes that resemble real models' layers.
@@ -190,7 +193,22 @@ def _design_configs(width, heads, kv, dim, experts, top, ff, vocab, layers):
     nusu = {"architecture": "Nusudra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
             "streams": 4, "layers": [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1],
                                       "mlp": {"kind": "dense", "ff": top * ff}} for i in range(layers)]}
-    return {"rumalorn": ruma, "pabavik": paba, "kekopel": keko, "nusudra": nusu, "minimax_m3": m3}
+    # Vodatar: differential attention (two maps of half the head size a head on values of the head size: cached rows as
+    # MiniMax-M3's) and latent attention (the same cached rows as Nusudra's) in turns; the same experts, one identity
+    # expert to eight real ones and a shared expert of an expert's width; the layers behind the first are one pass of a loop,
+    # so that as many layers run as in the other models
+    half = dim // 2
+    vatt = {"heads": heads, "kv_heads": kv, "dim": half, "vdim": dim, "conv": 4, "scale": half ** -0.5, "softcap": 30.0,
+            "diff": 0.3, "rot": {"dims": half, "base": 500000.0}}
+    vlat = dict(nlat, rot={"dims": rot, "base": 500000.0,
+                           "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
+    vmlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "identity": experts // 8, "top": top},
+            "shared": {"ff": ff}}
+    voda = {"architecture": "Vodatar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6, "groups": 8},
+            "residual_mult": 0.5, "canon": {"taps": 4}, "loop": {"start": 1, "stop": layers, "times": 1},
+            "layers": [{"type": "latent_attention" if i % 2 else "attention", "mixer": vlat if i % 2 else vatt, "mlp": vmlp}
+                       for i in range(layers)]}
+    return {"rumalorn": ruma, "pabavik": paba, "kekopel": keko, "nusudra": nusu, "vodatar": voda, "minimax_m3": m3}
 
 
 def _time_design(raw: Dict[str, Any], prompt: int, batch: int, steps: int, warmup: int) -> Dict[str, Any]:
@@ -260,7 +278,7 @@ def designs(raw: Dict[str, Any], layers: int = 4, prompt: int = 2048, batch: int
             row[design] = _time_design(cfg, prompt, batch, steps, warmup)
             gc.collect()
             torch.cuda.empty_cache()
-        for design in ("rumalorn", "pabavik", "kekopel", "nusudra"):
+        for design in ("rumalorn", "pabavik", "kekopel", "nusudra", "vodatar"):
             if design not in row:
                 continue
             row[f"{design}_over_minimax_m3"] = {
