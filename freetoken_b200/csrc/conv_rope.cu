@@ -157,7 +157,7 @@ __global__ void __launch_bounds__(kCrThreads) conv_rope_store_kernel(const __gri
         else for (int i = 0; i < nc; ++i) z[i] = from_float<T>(0.f);
       }
     }
-    if (used < p.pad_dim && map == 0) {
+    if (used < p.pad_dim && (is_q || map == 0)) {  // (a query row belongs to one map, a key row to all)
       const int step = ((is_v ? vq : dq)) * 4;
       for (int z0 = used + d0; z0 < p.pad_dim; z0 += step) {
         if (VEC) Vec4<T>::store(row + z0, zero);
