@@ -339,10 +339,10 @@ int ftk_sparse_select(const void* iq, const void* ik_slab, int dtype, const int3
 // Whether bfloat16 block scores of these sizes can be taken on the tensor cores (`scores [T, n_heads, max_blocks]`
 // float32 scratch must then be given to ftk_sparse_select).
 int ftk_sparse_score_fits(int n_heads, int dim, int block_size);
-// A token's row of logits may hold n_extra values behind the experts' (0 or 1).  aux [n_tokens, 2] or null: the sum of
+// A token's logits (each part) may hold n_extra values behind the experts' (0 or 1) and n_pad ones that mean nothing.  aux [n_tokens, 2] or null: the sum of
 // the weights of the chosen ids >= n_real (experts without tensors), and the sigmoid of the extra logit (1 without).
 int ftk_router_topk(const float* logits, int n_parts, const float* bias, int n_tokens, int n_experts, int top_k,
-                    int scoring, float scale, int32_t* ids, float* weights, int n_extra, int n_real, float* aux,
+                    int scoring, float scale, int32_t* ids, float* weights, int n_extra, int n_pad, int n_real, float* aux,
                     void* stream);
 // Router logits (float32 x [T, hidden] times gate_w [E, hidden]), choice and sort of the routes in one
 // launch, for steps of at most 32 tokens (beyond that the

@@ -209,7 +209,7 @@ __device__ __forceinline__ void route_one(const float* __restrict__ row, int par
 
 __global__ void router_topk_kernel(const float* __restrict__ logits, int n_parts, const float* __restrict__ bias,
                                    int n_tokens, int n_experts, int top_k, int scoring, float scale,
-                                   int32_t* __restrict__ ids, float* __restrict__ weights, int n_extra, int n_real,
+                                   int32_t* __restrict__ ids, float* __restrict__ weights, int n_extra, int n_pad, int n_real,
                                    float* __restrict__ aux) {
   pdl_wait();
   pdl_trigger();
@@ -218,7 +218,7 @@ __global__ void router_topk_kernel(const float* __restrict__ logits, int n_parts
   const int t = blockIdx.x * kRouterWarps + warp;
   if (t >= n_tokens) return;
   float* s = sm + (size_t)warp * 2 * n_experts;  // unbiased scores
-  const int stride = n_experts + n_extra;
+  const int stride = n_experts + n_extra + n_pad;
   const float* row = logits + (size_t)t * n_parts * stride;
   route_one(row, stride, n_parts, bias, n_experts, top_k, scoring, scale, s, ids + (size_t)t * top_k,
             weights + (size_t)t * top_k, nullptr);
@@ -388,9 +388,9 @@ moe_route_kernel(const float* __restrict__ x, const float* __restrict__ w, const
 using namespace ftk;
 
 extern "C" int ftk_router_topk(const float* logits, int n_parts, const float* bias, int n_tokens, int n_experts, int top_k,
-                               int scoring, float scale, int32_t* ids, float* weights, int n_extra, int n_real, float* aux,
+                               int scoring, float scale, int32_t* ids, float* weights, int n_extra, int n_pad, int n_real, float* aux,
                                void* stream) {
-  FTK_REQUIRE((n_extra == 0 || n_extra == 1) && n_real >= 0 && n_real <= n_experts, "router_topk: bad extra logits or expert counts");
+  FTK_REQUIRE((n_extra == 0 || n_extra == 1) && n_pad >= 0 && n_real >= 0 && n_real <= n_experts, "router_topk: bad extra logits or expert counts");
   FTK_REQUIRE(n_parts >= 1 && n_parts <= 4, "router_topk: %d blocks of logits per token (1 to 4)", n_parts);
   FTK_REQUIRE(scoring >= FTK_SCORE_SIGMOID && scoring <= FTK_SCORE_SIGMOID_RAW, "router_topk: unknown scoring %d", scoring);
   FTK_REQUIRE(n_experts >= 1 && top_k >= 1 && top_k <= n_experts, "router_topk: top_k=%d of %d experts", top_k, n_experts);
@@ -403,7 +403,7 @@ extern "C" int ftk_router_topk(const float* logits, int n_parts, const float* bi
   const int blocks = (n_tokens + kRouterWarps - 1) / kRouterWarps;
   note_variant(n_parts > 1 ? "routing: expert choice from logits given in pieces" : "routing: expert choice from given logits");
   FTK_LAUNCH(router_topk_kernel, blocks, kRouterWarps * 32, smem, (cudaStream_t)stream, logits, n_parts, bias, n_tokens, n_experts, top_k,
-                                                                               scoring, scale, ids, weights, n_extra, n_real, aux);
+                                                                               scoring, scale, ids, weights, n_extra, n_pad, n_real, aux);
   FTK_LAUNCH_CHECK("router_topk");
   return 0;
 }

@@ -136,7 +136,7 @@ _SIGNATURES = {
                                    _i, _i, _i, _i, _i, _i, _f, _vp, _i, _i, _vp],
     "ftk_sparse_select": [_vp, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp],
     "ftk_sparse_score_fits": [_i, _i, _i],
-    "ftk_router_topk": [_vp, _i, _vp, _i, _i, _i, _i, _f, _vp, _vp, _i, _i, _vp, _vp],
+    "ftk_router_topk": [_vp, _i, _vp, _i, _i, _i, _i, _f, _vp, _vp, _i, _i, _i, _vp, _vp],
     "ftk_moe_permute": [_vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp],
     "ftk_moe_route_fits": [_i, _i, _i, _i],
     "ftk_moe_route": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _vp],
@@ -652,7 +652,7 @@ def sparse_select(iq: torch.Tensor, ik_slab: torch.Tensor, block_table: torch.Te
 # --------------------------------------------------------------------------- experts
 def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, scoring: str,
                 scale: float, ids: torch.Tensor, weights: torch.Tensor, n_parts: int = 1, n_extra: int = 0,
-                n_real: Optional[int] = None, aux: Optional[torch.Tensor] = None) -> None:
+                n_real: Optional[int] = None, aux: Optional[torch.Tensor] = None, n_pad: int = 0) -> None:
     """Expert choice from float32 router logits ``[T, E]``.
 
     sigmoid: ``s = sigmoid(l)``; choice by ``s + bias``; ``w = s[ids] / (sum + 1e-20) * scale``.
@@ -663,14 +663,15 @@ def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, 
     With ``n_parts > 1`` the logits come as ``[T, n_parts * E]``: a token's logit of expert ``e`` is the
     32-bit sum of ``logits[t, q * E + e]`` over the parts ``q`` in their order.
 
-    A token's logits (each part) may end in ``n_extra`` (0 or 1) values that belong to no expert.  ``aux [T, 2]`` receives
+    A token's logits (each part) may end in ``n_extra`` (0 or 1) values that belong to no expert, and ``n_pad`` behind them
+    that mean nothing (they keep the product's rows aligned).  ``aux [T, 2]`` receives
     the sum of the token's weights that fell on ids from ``n_real`` on (experts without tensors; default: none) and the
     sigmoid of the extra logit (1 without one).  A softmax router's weights are divided by their sum + 1e-20.
     """
     T, PE = logits.shape
     if n_parts < 1 or PE % n_parts or not logits.is_contiguous():
         raise KernelError("router_topk: logits must be contiguous [T, n_parts * E]")
-    E = PE // n_parts - n_extra
+    E = PE // n_parts - n_extra - n_pad
     n_real = E if n_real is None else int(n_real)
     if aux is not None and aux.shape != (T, 2):
         raise KernelError("router_topk: aux must be [T, 2]")
@@ -681,7 +682,8 @@ def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, 
     _check(_lib().ftk_router_topk(_dev(logits, "logits", torch.float32), int(n_parts), _dev(bias, "bias", torch.float32),
                                   T, E, top_k, SCORE_CODES[scoring], float(scale),
                                   _dev(ids, "ids", torch.int32), _dev(weights, "weights", torch.float32),
-                                  int(n_extra), n_real, _dev(aux, "aux", torch.float32), _stream()), "router_topk")
+                                  int(n_extra), int(n_pad), n_real, _dev(aux, "aux", torch.float32), _stream()),
+           "router_topk")
 
 
 def moe_permute(topk_ids: torch.Tensor, n_experts: int, expert_counts: torch.Tensor,

@@ -108,6 +108,7 @@ class MoE(FeedForward):
         if self.by_table and self.vocab < 1:
             raise ConfigError("moe: a token-table router needs the vocabulary size")
         self._gate_pieces: Optional[torch.Tensor] = None
+        self._pad = 0
         self._gate: Optional[torch.Tensor] = None  # the router's rows, and the shared expert's gate behind them
         self.shared_gate = bool(spec.get("shared_gate", False)) and self.shared_inter > 0
         self.has_aux = self.identity > 0 or self.shared_gate
@@ -159,7 +160,9 @@ class MoE(FeedForward):
         if self.on_input:
             self._ones = torch.ones(self.env.max_step_tokens * self.top_k, dtype=torch.float32, device=self.env.device)
         if self.env.dtype == torch.bfloat16 and SPLIT_ROUTER_PRODUCT and not self.by_table:
-            self._gate_pieces = split_in_three(self._gate)
+            # (zero rows up to a multiple of eight: the library's product is several times slower for odd row lengths)
+            self._pad = -self._gate.shape[0] % 8
+            self._gate_pieces = split_in_three(torch.nn.functional.pad(self._gate, (0, 0, 0, self._pad)))
 
     def workspace_bytes(self, n_tokens: int) -> int:
         item = 4 if self.env.dtype == torch.float32 else 2
@@ -235,9 +238,10 @@ class MoE(FeedForward):
                           counts, offsets, routes, pos, **self._aux_args(aux))
         elif self._gate_pieces is not None and h.dtype == torch.bfloat16:
             # the router reads float32(h): the three products below are exact, their 32-bit sums are the logits
-            pieces = ws.get("moe.logit_pieces", (T, 3 * L), torch.float32, (cap, 3 * L))
+            P = L + self._pad
+            pieces = ws.get("moe.logit_pieces", (T, 3 * P), torch.float32, (cap, 3 * P))
             torch.mm(h, self._gate_pieces.t(), out_dtype=torch.float32, out=pieces)
-            ops.router_topk(pieces, bias, k, self.scoring, self.scale, ids, wts, n_parts=3, **self._aux_args(aux))
+            ops.router_topk(pieces, bias, k, self.scoring, self.scale, ids, wts, n_parts=3, n_pad=self._pad, **self._aux_args(aux))
             ops.moe_permute(ids, E, counts, offsets, routes, pos)
         else:
             torch.matmul(h_f32, self._gate.t(), out=logits)

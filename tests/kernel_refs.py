@@ -189,7 +189,7 @@ def sparse_select(iq, ik_slab, block_table, seg_info, n_segs, block_size, local_
             sel[q_start + t, :, : chosen.shape[1]] = chosen.to(torch.int32)
 
 
-def router_topk(logits, bias, top_k, scoring, scale, ids, weights, n_parts=1, n_extra=0, n_real=None, aux=None):
+def router_topk(logits, bias, top_k, scoring, scale, ids, weights, n_parts=1, n_extra=0, n_real=None, aux=None, n_pad=0):
     l = logits.float()
     if n_parts > 1:
         parts = l.view(l.shape[0], n_parts, -1)
@@ -197,6 +197,8 @@ def router_topk(logits, bias, top_k, scoring, scale, ids, weights, n_parts=1, n_
         for q in range(1, n_parts):
             l = l + parts[:, q]
     extra = None
+    if n_pad:
+        l = l[:, :-n_pad]
     if n_extra:
         l, extra = l[:, :-n_extra], l[:, -1]
     if aux is not None:

@@ -356,8 +356,10 @@ def test_routing_with_identity_experts_and_an_extra_logit(T, E, n_id, k, extra):
     ref.router_topk(logits, corr.cpu(), k, "softmax", 1.0, want["ids"], want["wts"], n_extra=extra, n_real=E, aux=want["aux"])
     got = mk(DEV)
     parts = torch.cat([logits * 0.75, logits * 0.25], -1).to(DEV).contiguous()
-    for n_parts, lg in ((1, logits.to(DEV)), (2, parts)):
-        ops.router_topk(lg, corr, k, "softmax", 1.0, got["ids"], got["wts"], n_parts=n_parts, n_extra=extra, n_real=E, aux=got["aux"])
+    padded = torch.cat([torch.nn.functional.pad(logits * f, (0, 3), value=1e9) for f in (0.75, 0.25)], -1).to(DEV).contiguous()
+    for n_parts, lg, pad in ((1, logits.to(DEV), 0), (2, parts, 0), (2, padded, 3)):
+        ops.router_topk(lg, corr, k, "softmax", 1.0, got["ids"], got["wts"], n_parts=n_parts, n_extra=extra, n_real=E, aux=got["aux"],
+                        n_pad=pad)
         torch.testing.assert_close(got["ids"].cpu(), want["ids"], rtol=0, atol=0)
         torch.testing.assert_close(got["wts"].cpu(), want["wts"], rtol=1e-5, atol=1e-6)
         torch.testing.assert_close(got["aux"].cpu(), want["aux"], rtol=1e-5, atol=1e-6)
