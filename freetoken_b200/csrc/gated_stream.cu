@@ -31,6 +31,32 @@ __device__ __forceinline__ float gate_sigmoid(float z) {
   else return __fdividef(1.f, 1.f + __expf(-z));
 }
 
+// Four adjacent elements as they lie in memory: a load that may be left out is kept in this form, since widening it beside
+// the load would make the branch around it wait for the data.
+template <typename T>
+struct Raw4;
+template <>
+struct Raw4<float> {
+  float4 v;
+  __device__ __forceinline__ void widen(float (&y)[4]) const { y[0] = v.x; y[1] = v.y; y[2] = v.z; y[3] = v.w; }
+};
+template <>
+struct Raw4<__nv_bfloat16> {
+  uint2 v;
+  __device__ __forceinline__ void widen(float (&y)[4]) const {
+    y[0] = __uint_as_float(v.x << 16);
+    y[1] = __uint_as_float(v.x & 0xffff0000u);
+    y[2] = __uint_as_float(v.y << 16);
+    y[3] = __uint_as_float(v.y & 0xffff0000u);
+  }
+};
+template <typename T>
+__device__ __forceinline__ Raw4<T> raw_or_zero(const T* p, bool have) {
+  Raw4<T> r{};
+  if (have) r = *reinterpret_cast<const Raw4<T>*>(p);
+  return r;
+}
+
 // One element (or four adjacent ones) of the sub-layer's gated result.
 template <typename T, int W>
 __device__ __forceinline__ void gated_result(const FtkStreamStep& p, int src_row, size_t src, int i, float2 aux, float (&v)[4]) {
@@ -216,11 +242,17 @@ __global__ void __launch_bounds__(MAX_THREADS) stream_step_regs_kernel(const __g
       for (int q = 0; q < PER; ++q) Vec4<T>::load((const T*)p.gate + src + at[q], gv[q]);
     }
     if constexpr (ROUTED) {
+      Raw4<T> through[PER], common[PER];  // the token's own row and the shared expert's
+      const bool passes = p.passed && aux.x != 0.f;
 #pragma unroll
-      for (int q = 0; q < PER; ++q) yv[q][0] = yv[q][1] = yv[q][2] = yv[q][3] = 0.f;
-      constexpr int J = PER <= 1 ? 8 : PER <= 2 ? 4 : 2;  // routes whose rows are asked for before the first is added
+      for (int q = 0; q < PER; ++q) {
+        yv[q][0] = yv[q][1] = yv[q][2] = yv[q][3] = 0.f;
+        common[q] = raw_or_zero((const T*)p.shared + src + at[q], p.shared != nullptr);
+        through[q] = raw_or_zero((const T*)p.passed + src + at[q], passes);
+      }
+      constexpr int J = PER <= 1 ? 8 : PER <= 3 ? 4 : 2;  // routes whose rows are asked for before the first is added
       for (int j0 = 0; j0 < p.top_k; j0 += J) {            // route order
-        float y[J][PER][4];
+        Raw4<T> y[J][PER];
         int pos[J];
 #pragma unroll
         for (int j = 0; j < J; ++j) {
@@ -230,34 +262,24 @@ __global__ void __launch_bounds__(MAX_THREADS) stream_step_regs_kernel(const __g
 #pragma unroll
         for (int j = 0; j < J; ++j)
 #pragma unroll
-          for (int q = 0; q < PER; ++q) {
-            if (pos[j] >= 0) Vec4<T>::load(x + (size_t)pos[j] * p.hidden + at[q], y[j][q]);
-            else y[j][q][0] = y[j][q][1] = y[j][q][2] = y[j][q][3] = 0.f;
-          }
+          for (int q = 0; q < PER; ++q) y[j][q] = raw_or_zero(x + (size_t)pos[j] * p.hidden + at[q], pos[j] >= 0);
 #pragma unroll
         for (int j = 0; j < J; ++j)
 #pragma unroll
-          for (int q = 0; q < PER; ++q)
+          for (int q = 0; q < PER; ++q) {
+            float v[4];
+            y[j][q].widen(v);
 #pragma unroll
-            for (int u = 0; u < 4; ++u) yv[q][u] += y[j][q][u];
+            for (int u = 0; u < 4; ++u) yv[q][u] += v[u];
+          }
       }
-      if (p.passed && aux.x != 0.f) {
 #pragma unroll
-        for (int q = 0; q < PER; ++q) {
-          float y[4];
-          Vec4<T>::load((const T*)p.passed + src + at[q], y);
+      for (int q = 0; q < PER; ++q) {
+        float own[4], sh[4];
+        through[q].widen(own);
+        common[q].widen(sh);
 #pragma unroll
-          for (int u = 0; u < 4; ++u) yv[q][u] = fmaf(aux.x, y[u], yv[q][u]);
-        }
-      }
-      if (p.shared) {
-#pragma unroll
-        for (int q = 0; q < PER; ++q) {
-          float y[4];
-          Vec4<T>::load((const T*)p.shared + src + at[q], y);
-#pragma unroll
-          for (int u = 0; u < 4; ++u) yv[q][u] = fmaf(aux.y, y[u], yv[q][u]);
-        }
+        for (int u = 0; u < 4; ++u) yv[q][u] = fmaf(aux.y, sh[u], fmaf(aux.x, own[u], yv[q][u]));
       }
     } else {
 #pragma unroll

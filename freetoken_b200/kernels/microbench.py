@@ -548,6 +548,14 @@ def bench_vodatar(a) -> dict:
     add("stream_step (the same over expert routes, identity experts and a gated shared expert)",
         lambda: ops.stream_step(res, x=rows, routed=(pos, k, shared, aux, passed), **common, **conv),
         T * C * (4 + 4 + 2 + 2 + 2) + (n_rows + n_pass) * C * 2 + extra)
+    # like kernels of the other designs, in the same call
+    add("like: postnorm_add_norm", lambda: ops.postnorm_add_norm(y, None, w, 1e-6, False, res, w, 1e-6, False, h),
+        T * C * (4 + 4 + 2 + 2))
+    perm = torch.randperm(T * k, device=dev, generator=g).to(torch.int32)
+    add("like: postnorm_add_norm over expert routes and a shared expert",
+        lambda: ops.postnorm_add_norm(rows, (perm, k, shared), w, 1e-6, False, res, w, 1e-6, False, h),
+        T * C * (4 + 4 + 2 + 2) + T * k * C * 2)
+    add("like: short_conv", lambda: ops.short_conv(res, cw, cst, slots, seg, S, u), T * C * (4 + 2) + (state_bytes if decode else 0))
     if not decode:
         add("conv_act (the sub-layer's input, no bias, no activation)",
             lambda: ops.conv_act(h, cw, None, None, cst, slots, seg, S, u), T * C * 4)
