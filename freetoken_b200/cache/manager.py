@@ -3,7 +3,8 @@
 Schedule entries whose mixers declare equal needs form a *group*.  A paged group
 (:class:`PagedGroup`) owns one page pool, one slab per stored quantity and entry, and one
 block table; a group whose need has a ``window`` gives pages back as soon as every position
-in them is older than any query can still read.  Groups with different needs have pools of
+in them is older than any query can still read (a need with ``keep_first`` keeps the pages of its first
+tokens all the same).  Groups with different needs have pools of
 their own, so a windowed group never competes with a full one.  State groups
 (:class:`StateGroup`) hold one fixed-size slot per live request.
 
@@ -62,6 +63,7 @@ class PagedGroup:
         self.entries = entries
         self.page_size = page_size
         self.width = width
+        self.kept_blocks = -(-need.keep_first // page_size) if need.window is not None else 0  # never given back before the end
         self.pool = PagePool(num_pages)
         self.slabs: Dict[str, torch.Tensor] = {}
         for name, heads, dim in need.slabs:
@@ -75,7 +77,7 @@ class PagedGroup:
         self.table_host = np.zeros((max_requests, width), dtype=np.int32)
         self.table_dev = torch.zeros((max_requests, width), dtype=torch.int32, device=device)
         self.updates: List[Tuple[int, int]] = []  # (flat index into the table, page)
-        self.first_live: Dict[int, int] = {}  # row -> first logical block still held
+        self.first_live: Dict[int, int] = {}  # row -> first logical block still held (behind the kept ones)
 
     def bytes_per_page(self, itemsize: int) -> int:
         return sum(h * d for _, h, d in self.need.slabs) * self.page_size * itemsize * len(self.entries)
@@ -162,7 +164,7 @@ class CacheManager:
             if isinstance(need, PagedKVNeed):
                 n = num_pages
                 if need.window is not None:
-                    per_req = -(-(need.window + step) // page_size) + 1
+                    per_req = -(-(need.window + step) // page_size) + 1 + -(-need.keep_first // page_size)
                     n = min(num_pages, max_requests * per_req)
                 g = PagedGroup(len(self.paged), need, entries, page_size, n, max_requests,
                                self.width, dtype, device, poison)
@@ -238,14 +240,14 @@ class CacheManager:
         step size).  A windowed group holds, while a step of ``n`` tokens runs on top of ``L``
         cached ones, the blocks from the first one a query of the step before could still read,
         ``(L - window + 1) // P``, to the last one the step writes, ``ceil((L + n) / P)``: at most
-        ``ceil((window - 1 + n) / P) + 1`` pages, whatever ``L`` is."""
+        ``ceil((window - 1 + n) / P) + 1`` pages, whatever ``L`` is, and the pages of the first tokens it keeps."""
         P = self.page_size
         n_step = min(step_tokens or self.max_step_tokens, self.max_step_tokens, max(1, total_tokens))
         out = []
         for g in self.paged:
             n = -(-total_tokens // P)
             if g.need.window is not None:
-                n = min(n, -(-(g.need.window - 1 + n_step) // P) + 1)
+                n = min(n, -(-(g.need.window - 1 + n_step) // P) + 1 + g.kept_blocks)
             out.append(n)
         return out
 
@@ -260,7 +262,8 @@ class CacheManager:
         for g in self.paged:
             pages = g.held_pages(req.row, n_blocks)
             g.pool.free(pages)
-            for b in range(g.first_live.pop(req.row, 0), n_blocks):
+            first = g.first_live.pop(req.row, 0)
+            for b in list(range(min(g.kept_blocks, first, n_blocks))) + list(range(first, n_blocks)):
                 if g.table_host[req.row, b] != NULL_PAGE:
                     g.set_entry(req.row, b, NULL_PAGE)
         self.slots.free(req.state_slot)
@@ -295,7 +298,7 @@ class CacheManager:
                 for rid, n in entries:
                     r = self.requests[rid]
                     reclaim += max(0, min(g.dead_blocks(r.length), -(-r.length // self.page_size))
-                                   - g.first_live[r.row])
+                                   - max(g.first_live[r.row], g.kept_blocks))
             if want > g.pool.free_count + reclaim:
                 raise CacheError(
                     f"out of pages in cache group {g.index}: the step needs {want}, "
@@ -333,6 +336,7 @@ class CacheManager:
         dead = min(g.dead_blocks(r.length), -(-r.length // self.page_size))
         first = g.first_live[r.row]
         if dead > first:
+            first = max(first, g.kept_blocks)
             pages = [int(p) for p in g.table_host[r.row, first:dead] if p != NULL_PAGE]
             g.pool.free(pages)
             for b in range(first, dead):
@@ -383,9 +387,10 @@ class CacheManager:
                 if np.any(g.table_host[r.row, n_blocks:] != NULL_PAGE):
                     raise CacheError(f"request {rid!r} holds pages beyond its length")
                 first = g.first_live[r.row]
-                if np.any(g.table_host[r.row, :first] != NULL_PAGE):
+                kept = min(g.kept_blocks, n_blocks)
+                if np.any(g.table_host[r.row, kept:first] != NULL_PAGE):
                     raise CacheError(f"request {rid!r} holds pages its window has passed")
-                if np.any(g.table_host[r.row, first:n_blocks] == NULL_PAGE):
+                if np.any(g.table_host[r.row, :kept] == NULL_PAGE) or np.any(g.table_host[r.row, first:n_blocks] == NULL_PAGE):
                     raise CacheError(f"request {rid!r} misses a page inside its length")
             g.pool.check(held)
             live_rows = {r.row for r in self.requests.values()}

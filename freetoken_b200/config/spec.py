@@ -78,15 +78,17 @@ class PagedKVNeed:
     (``("k", Hkv, D), ("v", Hkv, D)`` for attention; an indexer adds ``("index_k", 1, Di)``).
     A slab is laid out ``[pages, heads, page_size, dim]`` per owning schedule entry.
     ``window`` is ``None`` when every earlier token stays readable, else the number
-    of most recent tokens that do; pages wholly older than that are given back.
+    of most recent tokens that do; pages wholly older than that are given back, but for the ones that
+    hold any of the first ``keep_first`` tokens, which stay readable.
     Mixers with equal needs share a group (one page pool, one block table).
     """
 
     slabs: Tuple[Tuple[str, int, int], ...]
     window: Optional[int] = None
+    keep_first: int = 0
 
     def group_key(self) -> Tuple:
-        return ("paged", self.slabs, self.window)
+        return ("paged", self.slabs, self.window, self.keep_first)
 
 
 @dataclass(frozen=True)

@@ -15,6 +15,7 @@
 // the bias belongs to the logit: choice by logit + bias, weights = softmax of logit + bias over the chosen experts
 #define FTK_SCORE_SOFTMAX_OF_CHOSEN 2
 #define FTK_SCORE_SIGMOID_RAW 3  // sigmoid scores, the chosen experts' scores as weights without renormalising
+#define FTK_SCORE_SOFTMAX_RAW 4  // softmax scores over all experts, the chosen ones as they are
 
 #ifdef __cplusplus
 extern "C" {
@@ -81,6 +82,9 @@ typedef struct {
   // scores (scaled) become softcap * tanh(score / softcap); 0 = as they are.  Not with block selection or a bias by
   // distance.
   float softcap;
+  // with a window: queries also read the positions below keep_first (work items number the keys as build_plan does with
+  // keep_first); not with block selection, a bias by distance or a soft cap.  0 = none
+  int keep_first;
 } FtkAttnExtras;
 
 // What ftk_stream_step does to the rows of the 32-bit stream (see gated_stream.cu).  x, passed, shared, gate, raw_out,
@@ -89,6 +93,8 @@ typedef struct {
   float* residual;           // [T, hidden]
   const float* vec;          // [hidden] added to every row first, or null
   const void* x;             // [*, hidden] the sub-layer's rows, or the experts' rows with route_pos; null: none
+  const void* x2;            // [T, hidden] or null: the result is x_scale * x + x2_scale * x2 (dense rows only)
+  float x_scale, x2_scale;   // (used with x2)
   const int32_t* route_pos;  // [T, top_k] or null; negative: a route without a row
   int top_k;
   int n_routes;
@@ -105,6 +111,7 @@ typedef struct {
   float pre_eps;
   void* out;                 // [n_rows, hidden] or null
   float* norm_f32;           // [n_rows, hidden] the same, not rounded, or null (may be the stream)
+  int f32_rounded;           // norm_f32 takes the rounded values instead (float32(out))
   const float* conv_w;       // [hidden, taps] or null; rows are then one token per segment
   int taps;
   float* state;              // [n_slots, taps - 1, hidden]
@@ -206,7 +213,10 @@ int ftk_gla_scan(const void* q, long long q_stride, const void* k, long long k_s
                  float* state, int n_slots, const int32_t* state_slots, const int32_t* seg_info, int n_segs,
                  const int32_t* chunks, int n_chunks, const int32_t* seg_chunks, int any_single, int any_multi,
                  float* carry, float* decay_prod, float* out, int n_tokens, int n_heads, int dim, int vdim,
-                 const float* k_fac, const float* a_head, int ones_col, float* out_ones, int qk_div, void* stream);
+                 const float* k_fac, const float* a_head, int a_head_stride, int ones_col, float* out_ones, int qk_div,
+                 const float* rope, int n_rot, int rope_neighbours, int max_pos, void* stream);
+// (a_head_stride 0: a_head [n_heads], the same decays for every token.  rope [max_pos, n_rot] cos || sin: queries and keys
+// are rotated by their position, in 32 bits, as they are read; pairs of neighbours or of halves of the n_rot dimensions.)
 // (qk_div > 1: head h reads the queries and keys of head h / qk_div, and q, k hold n_heads / qk_div heads; with a_head)
 
 // One pass over S <= 8 residual streams (hyper.cu), streams [S][T, C] float32, stream_stride floats apart; each step
@@ -239,10 +249,12 @@ int ftk_ssm_output(const float* o32, const void* x, long long x_stride, const fl
 // (x / sqrt(sum x^2 + unit_eps), q then times q_scale).  q, k hold n_kv_heads heads of `dim`; state [n_slots, n_heads,
 // vdim, dim] float32 (column by column); out [T, n_heads, vdim] float32.
 int ftk_delta_scan(const void* q, long long q_stride, const void* k, long long k_stride, const void* v, long long v_stride,
-                   const void* b, long long b_stride, const void* a, long long a_stride, int dtype, const float* a_log,
+                   const void* b, long long b_stride, const void* a, long long a_stride, float* z, int dtype, const float* a_log,
                    const float* dt_bias, float q_scale, float unit_eps, float* state, int n_slots,
                    const int32_t* state_slots, const int32_t* seg_info, int n_segs, float* out, int n_tokens,
                    int n_heads, int n_kv_heads, int dim, int vdim, void* stream);
+// (z [n_tokens, n_heads * dim] float32 instead of a: logits of one decay per head and key channel; dt_bias is then
+// [n_heads * dim].  When a segment has several tokens z is overwritten with the decays.)
 // Short causal convolution over time with a residual (shortconv.cu): out[t, c] = x[t, c] + sum_j w[c, j] *
 // in(t - taps + 1 + j, c) over the request's own inputs; the last taps - 1 inputs of every request live in its
 // state slot (state [n_slots, taps - 1, channels] float32, oldest first; zeros before the sequence's start) and are
@@ -287,7 +299,7 @@ int ftk_copy_tokens(int32_t* dst, int dst_len, const int32_t* pairs, const int32
                     int vocab, void* stream);
 int ftk_norm_rope_store(const void* x, int dtype, int n_tokens, int row_elems, int head_dim,
                         int rotary_dim, const int32_t* positions, const float* rope_table, int max_pos,
-                        float eps, int gemma, int n_sections, const FtkSection* sections, void* stream);
+                        float eps, int gemma, int neighbours, int n_sections, const FtkSection* sections, void* stream);
 int ftk_paged_attention(const void* q, const void* k_slab, const void* v_slab, int dtype,
                         const int32_t* block_table, int bt_stride, const int32_t* seg_info, int n_segs,
                         const int32_t* items, int n_items, float* part_o, float* part_ml, int n_slots,
@@ -341,9 +353,11 @@ int ftk_sparse_select(const void* iq, const void* ik_slab, int dtype, const int3
 int ftk_sparse_score_fits(int n_heads, int dim, int block_size);
 // A token's logits (each part) may hold n_extra values behind the experts' (0 or 1) and n_pad ones that mean nothing.  aux [n_tokens, 2] or null: the sum of
 // the weights of the chosen ids >= n_real (experts without tensors), and the sigmoid of the extra logit (1 without).
+// The experts may form n_groups equal groups of neighbours: only those of the keep_groups groups with the largest choice
+// in them can be chosen (1, 1: all experts).
 int ftk_router_topk(const float* logits, int n_parts, const float* bias, int n_tokens, int n_experts, int top_k,
                     int scoring, float scale, int32_t* ids, float* weights, int n_extra, int n_pad, int n_real, float* aux,
-                    void* stream);
+                    int n_groups, int keep_groups, void* stream);
 // Router logits (float32 x [T, hidden] times gate_w [E, hidden]), choice and sort of the routes in one
 // launch, for steps of at most 32 tokens (beyond that the
 // separate kernels are faster); ftk_moe_route_fits says whether the sizes are taken.
@@ -351,7 +365,7 @@ int ftk_moe_route_fits(int n_tokens, int hidden, int n_experts, int top_k);
 int ftk_moe_route(const float* x, const float* gate_w, const float* bias, int n_tokens, int hidden, int n_experts,
                   int top_k, int scoring, float scale, float* logits, int32_t* ids, float* weights,
                   int32_t* counts, int32_t* offsets, int32_t* routes, int32_t* pos, int do_sort, int n_extra,
-                  int n_real, float* aux, void* stream);
+                  int n_real, float* aux, int n_groups, int keep_groups, void* stream);
 // Products of very few tokens (bfloat16): the weights are streamed once by warps of every SM (gemv.cu).
 int ftk_small_linear_fits(int n_tokens, int n_out, int k);
 int ftk_small_linear(const void* x, const void* w, void* out, int n_tokens, int n_out, int k, void* stream);

@@ -65,6 +65,10 @@ struct AttnParams {
   const float* sink_heads;
   // scaled scores s become softcap * tanh(s / softcap); 0: as they are
   float softcap;
+  // first tokens that a window keeps: a query also reads positions below keep_first.  Key numbers of the work items then
+  // run over the first keep_span positions (keep_first rounded up to keep_quantum) and, right behind them, the tile's window
+  // from the multiple of keep_quantum at or before its first key (see Item::jump).  keep_span 0: none
+  int keep_first, keep_span, keep_quantum;
 };
 
 // Soft-capped scores of the bfloat16 kernels: raw products s become softcap * log2(e) * tanh(s * scale / softcap), scores
@@ -173,7 +177,11 @@ constexpr int kMaxMergeSplits = 64;  // most splits of one tile that the merge s
 struct Item {
   int seg, tok0, ntok, kb, ke, nsplit, split, base;
   int q_start, q_len, kv_len, bt_row;
+  int lo;    // first key inside the window of the tile's first token (0 without a window)
+  int jump;  // positions left out between the kept first tokens and the tile's window
   bool ok;
+  // how far the keys' positions are ahead of their numbers from key number `v` on, up to the end of v's keep_quantum
+  __device__ __forceinline__ int shift(const AttnParams& p, int v) const { return v < p.keep_span ? 0 : jump; }
 };
 
 __device__ __forceinline__ Item load_item(const AttnParams& p, int idx) {
@@ -185,6 +193,8 @@ __device__ __forceinline__ Item load_item(const AttnParams& p, int idx) {
   if (it.ok) {
     const int32_t* s = p.seg_info + (size_t)it.seg * 4;
     it.q_start = s[0]; it.q_len = s[1]; it.kv_len = s[2]; it.bt_row = s[3];
+    it.lo = p.window > 0 ? max(0, it.kv_len - it.q_len + it.tok0 - p.window + 1) : 0;
+    it.jump = p.keep_span > 0 ? max(0, it.lo / p.keep_quantum * p.keep_quantum - p.keep_span) : 0;
     const int key_limit = p.sel ? p.sel_stride * p.block_size : it.kv_len;
     it.ok = it.tok0 >= 0 && it.tok0 + it.ntok <= it.q_len && it.kb >= 0 && it.ke <= key_limit &&
             (!p.sel || it.ntok == 1) &&
@@ -200,7 +210,11 @@ __device__ __forceinline__ Item load_item(const AttnParams& p, int idx) {
 // Position in the sequence of key number `v` of the tile's range: `v` itself, or, in a block-sparse
 // layer, the v-th key of the chosen blocks of the tile's (single) token; -1 when there is none.
 __device__ __forceinline__ int key_position(const AttnParams& p, const Item& it, int kvh, int v) {
-  if (!p.sel) return v;
+  if (!p.sel) {
+    if (p.keep_span == 0) return v;
+    const int pos = v + it.shift(p, v);
+    return pos >= p.keep_first && pos < it.lo ? -1 : pos;  // (neither kept nor in any row's window: its page may be gone)
+  }
   const int32_t* chosen = p.sel + ((size_t)(it.q_start + it.tok0) * p.Hkv + kvh) * p.sel_stride;
   const int slot = v / p.block_size;
   if (slot >= p.sel_stride) return -1;
@@ -280,7 +294,7 @@ __global__ void __launch_bounds__(kF32Rows * 32) attention_f32_kernel(AttnParams
     __syncthreads();
     if (!active) continue;
     const int key = lane < nk ? spos[lane] : -1;
-    const bool vis = key >= 0 && key <= q_pos && key >= lo_row;
+    const bool vis = key >= 0 && key <= q_pos && (key >= lo_row || key < p.keep_first);
     float s = -INFINITY;
     if (vis) {
       const float* qr = sq + warp * D;
@@ -604,7 +618,7 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(AttnParams p) {
       cap_scores(*reinterpret_cast<float (*)[kBN / 2]>(&s), cap, qp0 >= 0 || qp1 >= 0);
     }
     // mask, running max
-    const int c0 = it.kb + iter * kBN;
+    const int c0 = it.kb + iter * kBN, shift = it.shift(p, c0);
     float mx0 = -INFINITY, mx1 = -INFINITY;
     // a key tile that lies as far behind every row of the warp as the bias table's last entry reaches has one
     // bias per row; the others look every key's distance up
@@ -616,10 +630,10 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(AttnParams p) {
     for (int n = 0; n < kBN / 8; ++n) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const int key = c0 + n * 8 + (lane & 3) * 2 + e;
-        const bool in = key < it.ke;
-        const bool v0 = in && key <= qp0 && key >= lo0;
-        const bool v1 = in && key <= qp1 && key >= lo1;
+        const int key = c0 + shift + n * 8 + (lane & 3) * 2 + e;
+        const bool in = key - shift < it.ke;
+        const bool v0 = in && key <= qp0 && (key >= lo0 || key < p.keep_first);
+        const bool v1 = in && key <= qp1 && (key >= lo1 || key < p.keep_first);
         s[n][e] = v0 ? s[n][e] * sl2 + (far ? fb0 : dist_bias_at(brow0, p.dist_len, qp0 - key) * kLog2e) : -INFINITY;
         s[n][2 + e] = v1 ? s[n][2 + e] * sl2 + (far ? fb1 : dist_bias_at(brow1, p.dist_len, qp1 - key) * kLog2e) : -INFINITY;
         mx0 = fmaxf(mx0, s[n][e]);
@@ -871,7 +885,7 @@ __global__ void __launch_bounds__(128) attention_decode_bf16_kernel(AttnParams p
     if (p.softcap > 0.f) {
       cap_scores(*reinterpret_cast<float (*)[8]>(&s), cap, qp0 >= 0 || qp1 >= 0);
     }
-    const int c0 = it.kb + iter * kBN + warp * 16;
+    const int c0 = it.kb + iter * kBN + warp * 16, shift = it.shift(p, c0);
     float mx0 = -INFINITY, mx1 = -INFINITY;
     // a 16-key slice that every row of the tile may read in full needs no mask (rows beyond the
     // tile's last are never stored, so what they compute does not matter)
@@ -896,11 +910,11 @@ __global__ void __launch_bounds__(128) attention_decode_bf16_kernel(AttnParams p
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int col = n * 8 + (lane & 3) * 2 + e;
-          int key = c0 + col;
-          const bool in = key < it.ke;
+          int key = c0 + shift + col;
+          const bool in = c0 + col < it.ke;
           if (p.sel) key = in ? row_pos[iter & 3][warp * 16 + col] : -1;
-          const bool v0 = in && key >= 0 && key <= qp0 && key >= lo0;
-          const bool v1 = in && key >= 0 && key <= qp1 && key >= lo1;
+          const bool v0 = in && key >= 0 && key <= qp0 && (key >= lo0 || key < p.keep_first);
+          const bool v1 = in && key >= 0 && key <= qp1 && (key >= lo1 || key < p.keep_first);
           s[n][e] = v0 ? s[n][e] * sl2 + dist_bias_at(brow0, p.dist_len, qp0 - key) * kLog2e : -INFINITY;
           s[n][2 + e] = v1 ? s[n][2 + e] * sl2 + dist_bias_at(brow1, p.dist_len, qp1 - key) * kLog2e : -INFINITY;
           mx0 = fmaxf(mx0, s[n][e]);
@@ -1073,6 +1087,14 @@ extern "C" int ftk_attention_tc_few_fits(int head_dim, int page_size, int group)
   return attention_tc_few_fits(head_dim, page_size, group) ? 1 : 0;
 }
 
+// Kept first tokens of a window (see AttnParams): false if the options do not go together.
+static bool set_kept(AttnParams& p, const FtkAttnExtras* extras, int quantum) {
+  p.keep_first = extras ? extras->keep_first : 0;
+  p.keep_quantum = quantum;
+  p.keep_span = (p.keep_first + quantum - 1) / quantum * quantum;
+  return p.keep_first >= 0 && (p.keep_first == 0 || (p.window > 0 && !p.sel && !p.dist_bias && !(p.softcap > 0.f)));
+}
+
 enum TcForm { kTcSingle = 0, kTcPair = 1, kTcFew = 2 };
 
 // bfloat16 steps on the tensor-core kernels: tiles of 128 query rows (`items` planned for tile_rows =
@@ -1125,6 +1147,7 @@ static int paged_attention_tc_impl(const void* q, const void* k_slab, const void
   p.softcap = extras ? extras->softcap : 0.f;
   FTK_REQUIRE(!(p.softcap > 0.f) || (!p.dist_bias && scale > 0.f),
               "paged_attention_tc: a soft cap goes with a positive scale and no distance bias");
+  FTK_REQUIRE(set_kept(p, extras, kTcKeys), "paged_attention_tc: kept first tokens go with a window, without bias or soft cap");
   FTK_REQUIRE(!p.has_sink || form == kTcSingle,
               "paged_attention_tc: of the tcgen05 kernels the one with 128-row tiles takes a softmax sink");
   cudaStream_t s = (cudaStream_t)stream;
@@ -1233,6 +1256,7 @@ static int paged_attention_impl(const void* q, const void* k_slab, const void* v
   p.softcap = extras ? extras->softcap : 0.f;
   FTK_REQUIRE(!(p.softcap > 0.f) || (!sel && !p.dist_bias),
               "paged_attention: a soft cap cannot be combined with block selection or a distance bias");
+  FTK_REQUIRE(set_kept(p, extras, kBN), "paged_attention: kept first tokens go with a window, without bias, soft cap or block selection");
   FTK_REQUIRE(!p.has_sink || !sel, "paged_attention: a sink cannot be combined with block selection");
   if (extras && extras->kv_split > 1) {
     FTK_REQUIRE(!sel && p.G % extras->kv_split == 0 && (long long)n_kv_heads * extras->kv_split <= 65535,

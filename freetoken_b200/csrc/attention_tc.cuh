@@ -623,7 +623,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           const int key = it.kb + j * kTcKeys + 16 * box;
           int page = 0;
           if (j < n_tiles && key < it.ke) {
-            const int slot = key / p.P;
+            const int slot = (key + it.shift(p, key)) / p.P;
             page = slot < p.bt_stride ? bt[slot] : 0;
             if (page < 0 || page >= p.num_pages) page = 0;
           }
@@ -638,7 +638,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           const int key = key0 + 16 * box;
           const int page = page_next;
           page_next = page_of(j + 1);
-          const int row = (page * p.Hkv + kvh) * p.P + key % p.P;
+          const int row = (page * p.Hkv + kvh) * p.P + (key + it.shift(p, key)) % p.P;
           if (FEW && !waited && (key0 + kTcKeys > fresh_from || (!kv && j == q_at))) {
             pdl_wait();
             waited = true;
@@ -718,11 +718,13 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           const int live = it.ke - key0;  // keys of the request in this tile
           if (p.window > 0) {
             // a windowed piece starts at a multiple of the key tile at or before the first key that its first row
-            // sees: the value rows before that key are zeroed too (their pages may have gone back to the pool)
-            const int dead = min(kTcKeys, max(0, it.kv_len - it.q_len + it.tok0 - p.window + 1) - key0);
-            if (dead > 0) {
-              for (int x = lane; x < dead * 16; x += 32) {
-                const int r = x / 16, h = (x / 8) & 1, c = x & 7;
+            // sees: the value rows before that key are zeroed too (their pages may have gone back to the pool), but the
+            // ones that the window keeps stay
+            const int first = key0 + it.shift(p, key0);
+            const int from = max(0, p.keep_first - first), dead = min(kTcKeys, it.lo - first);
+            if (dead > from) {
+              for (int x = lane; x < (dead - from) * 16; x += 32) {
+                const int r = from + x / 16, h = (x / 8) & 1, c = x & 7;
                 *reinterpret_cast<uint4*>(tiles + (v_tile0 + vs) * kTcTile + h * kTcHalf + r * 128 + c * 16) =
                     make_uint4(0u, 0u, 0u, 0u);
               }
@@ -782,9 +784,13 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int pos_base = it.kv_len - it.q_len + it.tok0;
     const int qpos = r < R ? pos_base + r / G : -1;
     // last key this row may read; rows past the tile's last are never stored and must not hold the others up
-    const int hi = r < R ? min(it.ke - 1, qpos) : 0x7fffffff;
+    // (with kept first tokens a piece's end is no position, but whole key tiles behind its start, or the request's end)
+    const int hi = r < R ? (p.keep_span ? qpos : min(it.ke - 1, qpos)) : 0x7fffffff;
     // first key the row may read (a sliding window); rows that the tile does not have need no mask
-    const int lo = (p.window > 0 && r < R) ? qpos - p.window + 1 : 0;
+    const int lo = (p.window > 0 && r < R) ? max(0, qpos - p.window + 1) : 0;
+    // keys from `keep` on are hidden for `hidden` places (0 and lo, unless the window keeps first tokens)
+    const int keep = p.keep_first;
+    const unsigned int hidden = (unsigned int)max(0, lo - keep);
     // a learned bias by distance (see AttnParams::dist_bias): the row of this thread's head, and the factor that
     // turns a bias into raw-score units (the scores are scaled after the maximum is taken)
     const float* brow = (BIASED && r < R) ? p.dist_bias + (size_t)(kvh * G + r % G) * p.dist_len : nullptr;
@@ -799,11 +805,11 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       }
       tc_fence_after();
       const uint32_t s_addr = lane_addr + (uint32_t)(sb * kTcKeys);
-      const int key0 = it.kb + j * kTcKeys;
+      const int key0 = it.kb + j * kTcKeys + it.shift(p, it.kb + j * kTcKeys);
       // the row's 128 scores, in registers for both passes (with a soft cap they are read once per pass instead)
       float v0[32], v1[32], v2[32], v3[32];
       // a tile that every row of the warp reads in full needs no mask (most tiles of a long prompt)
-      const bool interior = __all_sync(0xffffffffu, key0 + kTcKeys - 1 <= hi && key0 >= lo);
+      const bool interior = __all_sync(0xffffffffu, key0 + kTcKeys - 1 <= hi && (key0 >= lo || key0 + kTcKeys <= keep));
       float tile_bias = 0.f;  // what every score of this tile and row gets added, in the exp2 domain
       float mx = -INFINITY;
       float vb[CAPPED == kCapBounded ? 128 : 1];
@@ -828,10 +834,10 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       if (!interior) {
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          if (key0 + i > hi || key0 + i < lo) v0[i] = -INFINITY;
-          if (key0 + 32 + i > hi || key0 + 32 + i < lo) v1[i] = -INFINITY;
-          if (key0 + 64 + i > hi || key0 + 64 + i < lo) v2[i] = -INFINITY;
-          if (key0 + 96 + i > hi || key0 + 96 + i < lo) v3[i] = -INFINITY;
+          if (key0 + i > hi || (unsigned int)(key0 + i - keep) < hidden) v0[i] = -INFINITY;
+          if (key0 + 32 + i > hi || (unsigned int)(key0 + 32 + i - keep) < hidden) v1[i] = -INFINITY;
+          if (key0 + 64 + i > hi || (unsigned int)(key0 + 64 + i - keep) < hidden) v2[i] = -INFINITY;
+          if (key0 + 96 + i > hi || (unsigned int)(key0 + 96 + i - keep) < hidden) v3[i] = -INFINITY;
         }
       }
       if constexpr (BIASED) {

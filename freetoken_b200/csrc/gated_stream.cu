@@ -2,10 +2,10 @@
 //
 // stream_step, one pass over a token's row (every part optional):
 //   r <- r + vec                                            a vector for every token (what a pass of a loop adds)
-//   y  = dense row, or the sum over the token's expert routes in route order, plus pass_w * passed (experts that hand
+//   y  = dense row (or x_scale times it plus x2_scale times a second one), or the sum over the token's expert routes in route order, plus pass_w * passed (experts that hand
 //        their input back) and shared_w * shared             (32-bit sums)
 //   y <- y * sigmoid(gate + gate_bias)                       element by element
-//   r <- r + groupnorm(y) * w_post                           (a factor on the result is folded into w_post)
+//   r <- r + groupnorm(y) * w_post                           (a factor on the result is folded into w_post), or r <- r + y
 //   raw = r rounded to the engine's type                     rows of another tensor (its own row stride)
 //   h  = groupnorm(r) * w_pre                                into `out`, as float32 into `norm_f32`
 //   u  = h + sum_j conv_w[:, j] h(t - taps + 1 + j)          steps of one token per request: the earlier h come from the
@@ -98,6 +98,12 @@ __device__ __forceinline__ void gated_result(const FtkStreamStep& p, int src_row
     }
   } else {
     load(x + src + i, v);
+    if (p.x2) {
+      float y[4];
+      load((const T*)p.x2 + src + i, y);
+#pragma unroll
+      for (int u = 0; u < W; ++u) v[u] = fmaf(p.x2_scale, y[u], p.x_scale * v[u]);
+    }
   }
   if (p.gate) {
     float g[4], b[4];
@@ -284,6 +290,15 @@ __global__ void __launch_bounds__(MAX_THREADS) stream_step_regs_kernel(const __g
     } else {
 #pragma unroll
       for (int q = 0; q < PER; ++q) Vec4<T>::load(x + src + at[q], yv[q]);
+      if (p.x2) {
+        float second[PER][4];
+#pragma unroll
+        for (int q = 0; q < PER; ++q) Vec4<T>::load((const T*)p.x2 + src + at[q], second[q]);
+#pragma unroll
+        for (int q = 0; q < PER; ++q)
+#pragma unroll
+          for (int u = 0; u < 4; ++u) yv[q][u] = fmaf(p.x2_scale, second[q][u], p.x_scale * yv[q][u]);
+      }
     }
     if (p.gate) {
 #pragma unroll
@@ -315,7 +330,12 @@ __global__ void __launch_bounds__(MAX_THREADS) stream_step_regs_kernel(const __g
     for (int w = 0; w < a.warps_per_group; ++w) t += scratch[team * a.warps_per_group + w];
     return t;
   };
-  if (has_y) {
+  if (has_y && !p.post_w) {
+#pragma unroll
+    for (int q = 0; q < PER; ++q)
+#pragma unroll
+      for (int u = 0; u < 4; ++u) zv[q][u] += yv[q][u];
+  } else if (has_y) {
     const float inv = rsqrtf(team_sum(ss, red[0]) / (float)a.group_size + p.post_eps);
 #pragma unroll
     for (int q = 0; q < PER; ++q)
@@ -341,9 +361,10 @@ __global__ void __launch_bounds__(MAX_THREADS) stream_step_regs_kernel(const __g
     float y[4];
 #pragma unroll
     for (int u = 0; u < 4; ++u) y[u] = zv[q][u] * inv * wr[q][u];
-    if (p.norm_f32) Vec4<float>::store(p.norm_f32 + dst + i, y);
+    if (p.norm_f32 && !p.f32_rounded) Vec4<float>::store(p.norm_f32 + dst + i, y);
 #pragma unroll
     for (int u = 0; u < 4; ++u) y[u] = to_float(from_float<T>(y[u]));
+    if (p.norm_f32 && p.f32_rounded) Vec4<float>::store(p.norm_f32 + dst + i, y);
     if (p.out) Vec4<T>::store((T*)p.out + dst + i, y);
     if constexpr (CONV && TAPS == 4) {
       float acc[4];
@@ -403,10 +424,10 @@ __global__ void __launch_bounds__(256) stream_step_any_kernel(const __grid_const
     }
     __syncthreads();
   };
-  if (has_y) factors(yrow, p.post_eps);
+  if (has_y && p.post_w) factors(yrow, p.post_eps);
   const bool changed = (has_y || p.vec) && !p.rows;
   for (int i = threadIdx.x; i < p.hidden; i += blockDim.x) {
-    if (has_y) zrow[i] = fmaf(yrow[i] * inv[i / a.group_size], p.post_w[i], zrow[i]);
+    if (has_y) zrow[i] = p.post_w ? fmaf(yrow[i] * inv[i / a.group_size], p.post_w[i], zrow[i]) : zrow[i] + yrow[i];
     if (changed) p.residual[src + i] = zrow[i];
     if (p.raw_out) ((T*)p.raw_out)[(size_t)r * p.raw_stride + i] = from_float<T>(zrow[i]);
   }
@@ -418,8 +439,9 @@ __global__ void __launch_bounds__(256) stream_step_any_kernel(const __grid_const
   for (int i = threadIdx.x; i < p.hidden; i += blockDim.x) {
     float y[4];
     y[0] = zrow[i] * inv[i / a.group_size] * p.pre_w[i];
-    if (p.norm_f32) p.norm_f32[dst + i] = y[0];
+    const float exact = y[0];
     y[0] = to_float(from_float<T>(y[0]));
+    if (p.norm_f32) p.norm_f32[dst + i] = p.f32_rounded ? y[0] : exact;
     if (p.out) ((T*)p.out)[dst + i] = from_float<T>(y[0]);
     if (p.conv_w) step_conv<T, 1>(p, r, dst, i, y, live, st, before);
   }
@@ -437,7 +459,7 @@ extern "C" int ftk_stream_step(const FtkStreamStep* args, void* stream) {
               "stream_step: %d channels do not divide into %d groups", p.hidden, p.groups);
   if (p.n_rows == 0) return 0;
   FTK_REQUIRE(p.residual, "stream_step: null stream");
-  FTK_REQUIRE(!p.x || p.post_w, "stream_step: a sub-layer's result needs its norm's weight");
+  FTK_REQUIRE(!p.x2 || (p.x && !p.route_pos), "stream_step: a second dense row goes with a first");
   FTK_REQUIRE(!p.route_pos || (p.x && p.top_k >= 1 && p.n_routes >= 0), "stream_step: bad routes");
   FTK_REQUIRE(!p.passed || p.aux, "stream_step: passed rows need their weights");
   FTK_REQUIRE(p.pre_w || (!p.out && !p.norm_f32 && !p.conv_w), "stream_step: an output needs the weight of the stream's norm");
@@ -451,7 +473,7 @@ extern "C" int ftk_stream_step(const FtkStreamStep* args, void* stream) {
   a.group_size = p.hidden / p.groups;
   const int item = dtype_size(p.dtype);
   auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
-  const bool vec = a.group_size % 4 == 0 && al16(p.residual) && al16(p.x) && al16(p.passed) && al16(p.shared) && al16(p.gate) &&
+  const bool vec = a.group_size % 4 == 0 && al16(p.residual) && al16(p.x) && al16(p.x2) && al16(p.passed) && al16(p.shared) && al16(p.gate) &&
                    al16(p.gate_bias) && al16(p.post_w) && al16(p.pre_w) && al16(p.vec) && al16(p.out) && al16(p.norm_f32) &&
                    al16(p.conv_out) && al16(p.conv_out_f32) && al16(p.state) && al16(p.conv_w) && (p.raw_stride * item) % (4 * item) == 0 &&
                    (reinterpret_cast<uintptr_t>(p.raw_out) % (4 * item)) == 0;

@@ -8,7 +8,7 @@
 //
 // One warp handles one (token, head).  The head vector is normed in registers, parked in shared
 // memory so that a lane can read its rotation partner, rotated with the cos/sin row of the token's
-// position, and written to its destination: a dense [T, heads, D] tensor (queries) or the row of a
+// position (pairs of halves of the rotated span, or of neighbours), and written to its destination: a dense [T, heads, D] tensor (queries) or the row of a
 // paged slab [pages, heads, page_size, D] that the token's slot names (keys, values).
 //
 // A section may also add a bias to its heads first (projections whose bias is not added by the matrix
@@ -34,7 +34,7 @@ template <typename T>
 __global__ void norm_rope_store_kernel(const T* __restrict__ x, int n_tokens, int row_elems, int head_dim,
                                        int rotary_dim, const int32_t* __restrict__ positions,
                                        const float* __restrict__ rope_table, int max_pos, float eps, int gemma,
-                                       Sections sec) {
+                                       int neighbours, Sections sec) {
   pdl_wait();
   pdl_trigger();
   __shared__ float park[kWarpsPerBlock][kMaxHeadDim];
@@ -89,7 +89,12 @@ __global__ void norm_rope_store_kernel(const T* __restrict__ x, int n_tokens, in
 #pragma unroll
     for (int i = 0; i < kPer; ++i) {
       const int d = lane + 32 * i;
-      if (d < half) {
+      if (neighbours) {  // (2i, 2i + 1)
+        if (d < rotary_dim) {
+          const float c = cs[d >> 1], s = cs[half + (d >> 1)], other = park[warp][d ^ 1];
+          v[i] = (d & 1) ? park[warp][d] * c + other * s : park[warp][d] * c - other * s;
+        }
+      } else if (d < half) {
         v[i] = park[warp][d] * cs[d] - park[warp][d + half] * cs[half + d];
       } else if (d < rotary_dim) {
         v[i] = park[warp][d] * cs[d - half] + park[warp][d - half] * cs[d];
@@ -128,7 +133,7 @@ template <int LPH>
 __global__ void __launch_bounds__(kWarpsPerBlock * 32)
 norm_rope_store_vec_kernel(const __nv_bfloat16* __restrict__ x, int n_tokens, int row_elems, int rotary_dim,
                            const int32_t* __restrict__ positions, const float* __restrict__ rope_table, int max_pos,
-                           float eps, int gemma, Sections sec) {
+                           float eps, int gemma, int neighbours, Sections sec) {
   pdl_wait();
   pdl_trigger();
   constexpr int kHeadDim = LPH * 8;
@@ -166,12 +171,18 @@ norm_rope_store_vec_kernel(const __nv_bfloat16* __restrict__ x, int n_tokens, in
     pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
     const float* cs = rope_table + (size_t)pos * rotary_dim;
     const int d0 = l * 8;
-    const float* a = low ? cs + d0 : cs + d0 - half;  // cos of this element's pair
-    const float* b = low ? cs + half + d0 : cs + d0;  // sin of this element's pair
+    // cos and sin of these elements' pairs (neighbours: four pairs of them)
+    const float* a = neighbours ? cs + (d0 >> 1) : low ? cs + d0 : cs + d0 - half;
+    const float* b = neighbours ? cs + half + (d0 >> 1) : low ? cs + half + d0 : cs + d0;
+    if (neighbours) {
+      *reinterpret_cast<float4*>(ca) = *reinterpret_cast<const float4*>(a);
+      *reinterpret_cast<float4*>(cb) = *reinterpret_cast<const float4*>(b);
+    } else {
     *reinterpret_cast<float4*>(ca) = *reinterpret_cast<const float4*>(a);
     *reinterpret_cast<float4*>(ca + 4) = *reinterpret_cast<const float4*>(a + 4);
     *reinterpret_cast<float4*>(cb) = *reinterpret_cast<const float4*>(b);
     *reinterpret_cast<float4*>(cb + 4) = *reinterpret_cast<const float4*>(b + 4);
+    }
   }
   float factor = 1.f;
   if (S.pos_scale) {
@@ -214,7 +225,16 @@ norm_rope_store_vec_kernel(const __nv_bfloat16* __restrict__ x, int n_tokens, in
       for (int j = 0; j < 8; ++j) v[j] = v[j] * inv * (w[j] + one);
     }
   }
-  {
+  if (neighbours) {
+    if (rot && in) {
+#pragma unroll
+      for (int j = 0; j < 8; j += 2) {
+        const float x = v[j], y = v[j + 1], c = ca[j >> 1], s = cb[j >> 1];
+        v[j] = x * c - y * s;
+        v[j + 1] = y * c + x * s;
+      }
+    }
+  } else {
     // rotation partners: the lane half a rotary span away, on either side
     const int hop = half >> 3;  // lanes per half span
     float partner[8];
@@ -261,7 +281,7 @@ using namespace ftk;
 
 extern "C" int ftk_norm_rope_store(const void* x, int dtype, int n_tokens, int row_elems, int head_dim,
                                    int rotary_dim, const int32_t* positions, const float* rope_table,
-                                   int max_pos, float eps, int gemma, int n_sections,
+                                   int max_pos, float eps, int gemma, int neighbours, int n_sections,
                                    const FtkSection* sections, void* stream) {
   FTK_REQUIRE(dtype_ok(dtype), "norm_rope_store: bad dtype %d", dtype);
   FTK_REQUIRE(n_sections >= 1 && n_sections <= kMaxSections, "norm_rope_store: %d sections (1..%d allowed)",
@@ -322,22 +342,22 @@ extern "C" int ftk_norm_rope_store(const void* x, int dtype, int n_tokens, int r
       const int32_t* ps = positions ? positions + t0 : nullptr;
       if (lph == 8)
         FTK_LAUNCH(norm_rope_store_vec_kernel<8>, vgrid, kWarpsPerBlock * 32, 0, s, xs, nt, row_elems, rotary_dim, ps,
-                   rope_table, max_pos, eps, gemma, part);
+                   rope_table, max_pos, eps, gemma, neighbours, part);
       else if (lph == 16)
         FTK_LAUNCH(norm_rope_store_vec_kernel<16>, vgrid, kWarpsPerBlock * 32, 0, s, xs, nt, row_elems, rotary_dim, ps,
-                   rope_table, max_pos, eps, gemma, part);
+                   rope_table, max_pos, eps, gemma, neighbours, part);
       else
         FTK_LAUNCH(norm_rope_store_vec_kernel<32>, vgrid, kWarpsPerBlock * 32, 0, s, xs, nt, row_elems, rotary_dim, ps,
-                   rope_table, max_pos, eps, gemma, part);
+                   rope_table, max_pos, eps, gemma, neighbours, part);
     } else if (dtype == FTK_F32)
       (note_variant("head norm + rotation + cache write: a warp per head"),
        FTK_LAUNCH(norm_rope_store_kernel<float>, grid, kWarpsPerBlock * 32, 0, s, 
           (const float*)x + (size_t)t0 * row_elems, nt, row_elems, head_dim, rotary_dim,
-          positions ? positions + t0 : nullptr, rope_table, max_pos, eps, gemma, part));
+          positions ? positions + t0 : nullptr, rope_table, max_pos, eps, gemma, neighbours, part));
     else
       FTK_LAUNCH(norm_rope_store_kernel<__nv_bfloat16>, grid, kWarpsPerBlock * 32, 0, s, 
           (const __nv_bfloat16*)x + (size_t)t0 * row_elems, nt, row_elems, head_dim, rotary_dim,
-          positions ? positions + t0 : nullptr, rope_table, max_pos, eps, gemma, part);
+          positions ? positions + t0 : nullptr, rope_table, max_pos, eps, gemma, neighbours, part);
   }
   FTK_LAUNCH_CHECK("norm_rope_store");
   return 0;

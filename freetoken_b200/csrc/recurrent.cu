@@ -16,6 +16,9 @@
 // The recurrence itself is the plain one, token by token, so the result differs from a pure scan only
 // by the rounding of step 2's sums.
 //
+// Variants of the same recurrence: one decay per (token, head), or per head alone (a_head); a factor on the keys; queries and
+// keys that are rotated by their position on the way in (32-bit, never rounded: they enter the recurrence).
+//
 // A block owns 64 (or 32) value columns of one (chunk, head): per group of that many columns, 4 warps split the
 // key channels, a thread keeps its share of two (or one) state columns in registers, and the tokens' q, k and
 // decays are staged in shared memory 16 tokens at a time for all of the block's columns (float4 reads, the same
@@ -53,6 +56,11 @@ struct GlaArgs {
   int H, D, Dv, n_tokens, groups;
   const float* k_fac;      // [T, H] or null: a factor on token t's keys of head h (applied in 32 bits while they are staged)
   const float* a_head;     // [T, H] or null: one decay per (token, head) for all key channels, in place of z
+  int a_head_stride;       // H, or 0: the same decays for every token ([H])
+  // rotary positions on the leading n_rot dimensions of queries and keys, applied in 32 bits while they are staged:
+  // [max_pos, n_rot] rows cos | sin, null: none; pairs (i, i + n_rot / 2), or neighbours
+  const float* rope;
+  int n_rot, rope_neighbours, max_pos;
   int ones_col;            // 1: the last of the Dv value columns is 1 for every token, and v holds Dv - 1 columns per head
   float* out_ones;         // [T, H] or null: with ones_col, that column's outputs go here and out is [T, H, Dv - 1]
   int qk_div;              // queries and keys are shared by groups of this many heads: head h reads q/k head h / qk_div
@@ -68,6 +76,38 @@ __device__ __forceinline__ void gla_cp4(void* dst, const void* src) {
 }
 __device__ __forceinline__ void gla_cp_commit() { asm volatile("cp.async.commit_group;\n" ::); }
 __device__ __forceinline__ void gla_cp_wait_all() { asm volatile("cp.async.wait_group 0;\n" ::: "memory"); }
+
+// Element d of a head's row, rotated.
+template <typename R>
+__device__ __forceinline__ float rotated1(const R* row, const float* cs, int d, int n_rot, bool neighbours) {
+  const float x = to_float(row[d]);
+  if (d >= n_rot) return x;
+  const int half = n_rot >> 1;
+  const bool low = neighbours ? (d & 1) == 0 : d < half;
+  const int i = neighbours ? d >> 1 : low ? d : d - half;  // the pair's index
+  const float o = to_float(row[neighbours ? d ^ 1 : low ? d + half : d - half]);
+  return low ? x * cs[i] - o * cs[half + i] : x * cs[i] + o * cs[half + i];
+}
+// Four adjacent elements d .. d + 3 of a head's row, rotated (`cs`: the position's cosines, then sines).
+template <typename R>
+__device__ __forceinline__ void rotated4(const R* row, const float* cs, int d, int n_rot, bool neighbours, float (&y)[4]) {
+  const int half = n_rot >> 1;
+  if (d >= n_rot) {
+    Vec4<R>::load(row + d, y);
+  } else if (!neighbours && (half & 3) == 0) {  // the four lie in one half
+    const bool low = d < half;
+    float x[4], o[4], c[4], s[4];
+    Vec4<R>::load(row + d, x);
+    Vec4<R>::load(row + (low ? d + half : d - half), o);
+    Vec4<float>::load(cs + (low ? d : d - half), c);
+    Vec4<float>::load(cs + (low ? d + half : d), s);
+#pragma unroll
+    for (int u = 0; u < 4; ++u) y[u] = low ? x[u] * c[u] - o[u] * s[u] : x[u] * c[u] + o[u] * s[u];
+  } else {
+#pragma unroll
+    for (int u = 0; u < 4; ++u) y[u] = rotated1(row, cs, d + u, n_rot, neighbours);
+  }
+}
 
 __device__ __forceinline__ float decay_of(float z, float inv_tau) {
   // sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau)
@@ -168,6 +208,11 @@ __global__ void __launch_bounds__(gla_max_groups(DPT) * kGlaSlices * 32) gla_chu
   float* zraw = reinterpret_cast<float*>(qraw + kGlaBatch * Dp);                                  // [batch][Dp]
   __nv_bfloat16* vraw = reinterpret_cast<__nv_bfloat16*>(zraw + kGlaBatch * Dp);                  // [batch][cols]
   float* hraw = reinterpret_cast<float*>(vraw + kGlaBatch * cols);                                // [2][batch]: key factors, head decays
+  // the rotation table's row of the chunk's token t
+  auto rope_row = [&](int t) {
+    const int pos = kv_len - q_len + tok0 + t;
+    return a.rope + (size_t)(pos < a.max_pos ? pos : a.max_pos - 1) * a.n_rot;
+  };
   auto fetch = [&](int b0n) {
     const int nbn = min(kGlaBatch, ntok - b0n);
     const int per_row = Dp / 8;
@@ -186,11 +231,25 @@ __global__ void __launch_bounds__(gla_max_groups(DPT) * kGlaSlices * 32) gla_chu
         gla_cp16(zraw + t * Dp + d + 4, in ? zr + 4 : zr, in);
       }
     }
+    if (a.rope) {  // the positions' rows of the rotation table, where the decay logits would lie
+      if ((a.n_rot & 3) == 0) {
+        const int per_rot = a.n_rot >> 2;
+        for (int i = threadIdx.x; i < nbn * per_rot; i += blockDim.x) {
+          const int t = i / per_rot, d = (i % per_rot) * 4;
+          gla_cp16(zraw + t * Dp + d, rope_row(b0n + t) + d, true);
+        }
+      } else {
+        for (int i = threadIdx.x; i < nbn * a.n_rot; i += blockDim.x) {
+          const int t = i / a.n_rot, d = i % a.n_rot;
+          gla_cp4(zraw + t * Dp + d, rope_row(b0n + t) + d);
+        }
+      }
+    }
     if (a.k_fac || a.a_head) {
       for (int t = threadIdx.x; t < nbn; t += blockDim.x) {
-        const size_t at = (size_t)(q_start + tok0 + b0n + t) * a.H + h;
-        if (a.k_fac) gla_cp4(hraw + t, a.k_fac + at);
-        if (a.a_head) gla_cp4(hraw + kGlaBatch + t, a.a_head + at);
+        const size_t tok = (size_t)(q_start + tok0 + b0n + t);
+        if (a.k_fac) gla_cp4(hraw + t, a.k_fac + tok * a.H + h);
+        if (a.a_head) gla_cp4(hraw + kGlaBatch + t, a.a_head + tok * a.a_head_stride + h);
       }
     }
     const int vper = cols / 8;
@@ -211,6 +270,15 @@ __global__ void __launch_bounds__(gla_max_groups(DPT) * kGlaSlices * 32) gla_chu
       for (int i = threadIdx.x * 4; i < nb * Dp; i += blockDim.x * 4) {
         const int d = i % Dp, t = i / Dp;
         const float kf = a.k_fac ? hraw[t] : 1.f;
+        if (a.rope) {
+          float y[4];
+          rotated4(kraw + t * Dp, zraw + t * Dp, d, a.n_rot, a.rope_neighbours, y);
+          *reinterpret_cast<float4*>(sk + i) = make_float4(y[0] * kf, y[1] * kf, y[2] * kf, y[3] * kf);
+          if (MODE != 1) {
+            rotated4(qraw + t * Dp, zraw + t * Dp, d, a.n_rot, a.rope_neighbours, y);
+            *reinterpret_cast<float4*>(sq + i) = make_float4(y[0] * a.q_scale, y[1] * a.q_scale, y[2] * a.q_scale, y[3] * a.q_scale);
+          }
+        } else {
         const __nv_bfloat162* k2 = reinterpret_cast<const __nv_bfloat162*>(kraw + i);
         const float2 k01 = __bfloat1622float2(k2[0]), k23 = __bfloat1622float2(k2[1]);
         *reinterpret_cast<float4*>(sk + i) = make_float4(k01.x * kf, k01.y * kf, k23.x * kf, k23.y * kf);
@@ -218,6 +286,7 @@ __global__ void __launch_bounds__(gla_max_groups(DPT) * kGlaSlices * 32) gla_chu
           const __nv_bfloat162* q2 = reinterpret_cast<const __nv_bfloat162*>(qraw + i);
           const float2 q01 = __bfloat1622float2(q2[0]), q23 = __bfloat1622float2(q2[1]);
           *reinterpret_cast<float4*>(sq + i) = make_float4(q01.x * a.q_scale, q01.y * a.q_scale, q23.x * a.q_scale, q23.y * a.q_scale);
+        }
         }
         float4 av;
         if (d >= D) {
@@ -254,10 +323,26 @@ __global__ void __launch_bounds__(gla_max_groups(DPT) * kGlaSlices * 32) gla_chu
 #pragma unroll
         for (int u = 0; u < 8; ++u) { qv[u] = 0.f; kv[u] = 0.f; av[u] = 1.f; }
         if (d < D) {
+          const float kf = a.k_fac ? a.k_fac[tok * a.H + h] : 1.f;
+          if (a.rope) {
+            const T* krow = kb + tok * a.k_stride + (size_t)hqk * D;
+            const T* qrow = qb + tok * a.q_stride + (size_t)hqk * D;
+            const float* cs = rope_row(b0 + t);
+#pragma unroll
+            for (int g4 = 0; g4 < 8; g4 += 4) {
+              float y[4];
+              rotated4(krow, cs, d + g4, a.n_rot, a.rope_neighbours, y);
+#pragma unroll
+              for (int u = 0; u < 4; ++u) kv[g4 + u] = y[u] * kf;
+              if (MODE != 1) {
+                rotated4(qrow, cs, d + g4, a.n_rot, a.rope_neighbours, y);
+#pragma unroll
+                for (int u = 0; u < 4; ++u) qv[g4 + u] = y[u] * a.q_scale;
+              }
+            }
+          } else {
           const uint4 kr = *reinterpret_cast<const uint4*>(kb + tok * a.k_stride + (size_t)hqk * D + d);
           const __nv_bfloat162* k2 = reinterpret_cast<const __nv_bfloat162*>(&kr);
-#pragma unroll
-          const float kf = a.k_fac ? a.k_fac[tok * a.H + h] : 1.f;
 #pragma unroll
           for (int u = 0; u < 4; ++u) { const float2 f = __bfloat1622float2(k2[u]); kv[2 * u] = f.x * kf; kv[2 * u + 1] = f.y * kf; }
           if (MODE != 1) {
@@ -266,8 +351,9 @@ __global__ void __launch_bounds__(gla_max_groups(DPT) * kGlaSlices * 32) gla_chu
 #pragma unroll
             for (int u = 0; u < 4; ++u) { const float2 f = __bfloat1622float2(q2[u]); qv[2 * u] = f.x * a.q_scale; qv[2 * u + 1] = f.y * a.q_scale; }
           }
+          }
           if (a.a_head) {
-            const float ah = a.a_head[tok * a.H + h];
+            const float ah = a.a_head[tok * a.a_head_stride + h];
 #pragma unroll
             for (int u = 0; u < 8; ++u) av[u] = ah;
           } else {
@@ -294,9 +380,18 @@ __global__ void __launch_bounds__(gla_max_groups(DPT) * kGlaSlices * 32) gla_chu
         const size_t tok = (size_t)(q_start + tok0 + b0 + t);
         float qv = 0.f, kv = 0.f, av = 1.f;
         if (d < D) {
-          if (MODE != 1) qv = to_float(qb[tok * a.q_stride + (size_t)hqk * D + d]) * a.q_scale;
-          kv = to_float(kb[tok * a.k_stride + (size_t)hqk * D + d]) * (a.k_fac ? a.k_fac[tok * a.H + h] : 1.f);
-          av = a.a_head ? a.a_head[tok * a.H + h] : a.z[(tok * a.H + h) * D + d];
+          const T* krow = kb + tok * a.k_stride + (size_t)hqk * D;
+          const T* qrow = qb + tok * a.q_stride + (size_t)hqk * D;
+          if (a.rope) {
+            const float* cs = rope_row(b0 + t);
+            kv = rotated1(krow, cs, d, a.n_rot, a.rope_neighbours);
+            if (MODE != 1) qv = rotated1(qrow, cs, d, a.n_rot, a.rope_neighbours) * a.q_scale;
+          } else {
+            if (MODE != 1) qv = to_float(qrow[d]) * a.q_scale;
+            kv = to_float(krow[d]);
+          }
+          kv *= a.k_fac ? a.k_fac[tok * a.H + h] : 1.f;
+          av = a.a_head ? a.a_head[tok * a.a_head_stride + h] : a.z[(tok * a.H + h) * D + d];
           if (!a.a_head && !a.z_is_decay) av = decay_of(av + (a.z_bias ? a.z_bias[(size_t)h * D + d] : 0.f), a.inv_tau);
         }
         sq[i] = qv; sk[i] = kv; sa[i] = av;
@@ -490,8 +585,8 @@ extern "C" int ftk_gla_scan(const void* q, long long q_stride, const void* k, lo
                             const int32_t* seg_info, int n_segs, const int32_t* chunks, int n_chunks,
                             const int32_t* seg_chunks, int any_single, int any_multi, float* carry,
                             float* decay_prod, float* out, int n_tokens, int n_heads, int dim, int vdim,
-                            const float* k_fac, const float* a_head, int ones_col, float* out_ones, int qk_div,
-                            void* stream) {
+                            const float* k_fac, const float* a_head, int a_head_stride, int ones_col, float* out_ones,
+                            int qk_div, const float* rope, int n_rot, int rope_neighbours, int max_pos, void* stream) {
   FTK_REQUIRE(dtype_ok(dtype), "gla_scan: bad dtype %d", dtype);
   FTK_REQUIRE(n_tokens >= 0 && n_segs >= 0 && n_chunks >= 0, "gla_scan: bad counts");
   if (n_tokens == 0 || n_chunks == 0) return 0;
@@ -512,6 +607,10 @@ extern "C" int ftk_gla_scan(const void* q, long long q_stride, const void* k, lo
   FTK_REQUIRE(!out_ones || ones_col, "gla_scan: outputs of a column of ones that is not there");
   FTK_REQUIRE(qk_div >= 1 && n_heads % qk_div == 0 && (qk_div == 1 || a_head),
               "gla_scan: heads that share queries and keys come in groups that divide the heads, with a decay per head");
+  FTK_REQUIRE(!a_head || a_head_stride == 0 || a_head_stride == n_heads, "gla_scan: decays per head for every token, or one row for all");
+  FTK_REQUIRE(!rope || (a_head && n_rot >= 2 && n_rot % 2 == 0 && n_rot <= dim && max_pos >= 1 && ((uintptr_t)rope & 15) == 0),
+              "gla_scan: a rotation goes with a decay per head, an even number of dimensions (at most %d) and an aligned table", dim);
+  a.a_head_stride = a_head_stride; a.rope = rope; a.n_rot = n_rot; a.rope_neighbours = rope_neighbours; a.max_pos = max_pos;
   a.k_fac = k_fac; a.a_head = a_head; a.ones_col = ones_col; a.out_ones = out_ones; a.qk_div = qk_div;
   a.out = out; a.H = n_heads; a.D = dim; a.Dv = vdim; a.n_tokens = n_tokens;
   cudaStream_t s = (cudaStream_t)stream;

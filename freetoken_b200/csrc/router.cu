@@ -3,6 +3,8 @@
 // sigmoid form (python/freetoken/models/minimax_m3/moe.py:71-81): s = sigmoid(logits); the experts
 // are chosen by s + bias, weighted by the unbiased s, divided by their sum (+1e-20) and multiplied by
 // the scaling factor.  softmax form (python/freetoken/moe/fused.py:27-31): s = softmax(logits).
+// Raw forms leave the chosen scores as they are.  Experts may form equal groups of neighbours of which only the best few
+// (by their largest choice) may be chosen from.
 // One warp per token; the largest choice goes first and the lower expert index wins a tie.
 // For long steps the logits are a library matrix product in float32, as in the reference (F.linear),
 // and router_topk_kernel takes them; for short steps moe_route_kernel computes them itself and also
@@ -37,9 +39,44 @@ __device__ __forceinline__ void token_aux(const float* __restrict__ row, int par
   }
 }
 
+// Experts in `count` equal groups of neighbours, of which the `keep` with the largest choice in them are open (count 1: all).
+struct RouteGroups {
+  int count, keep;
+};
+
+// What the chosen scores are divided by: nothing (1) in the raw forms.
+__device__ __forceinline__ float weight_denominator(int scoring, float wsum) {
+  if (scoring == FTK_SCORE_SIGMOID_RAW || scoring == FTK_SCORE_SOFTMAX_RAW) return 1.f;
+  return scoring == FTK_SCORE_SOFTMAX_OF_CHOSEN ? wsum : wsum + 1e-20f;
+}
+
+// The largest of c[0 .. n_experts) whose group is not in `closed` (a bit per group; size 0: no groups), by one warp; the
+// lowest index of equal ones; 0x7fffffff when every value is NaN or -inf.
+__device__ __forceinline__ int best_choice(const float* c, int n_experts, int size, unsigned long long closed) {
+  float best = -INFINITY;
+  int bi = 0x7fffffff;
+  for (int e = threadIdx.x & 31; e < n_experts; e += 32) {
+    const float v = size && (closed >> (e / size) & 1) ? -INFINITY : c[e];
+    if (v > best) {  // ascending e within a lane: the first of equal values stays
+      best = v;
+      bi = e;
+    }
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+    if (ob > best || (ob == best && oi < bi)) {
+      best = ob;
+      bi = oi;
+    }
+  }
+  return bi;
+}
+
 // Scores, choice and weights of one token, by one warp.  `s` and `c` hold n_experts floats each.
 __device__ __forceinline__ void route_token(const float* __restrict__ row, int part_stride, int n_parts, const float* __restrict__ bias,
-                                            int n_experts, int top_k, int scoring, float scale, float* s, float* c,
+                                            int n_experts, RouteGroups groups, int top_k, int scoring, float scale, float* s, float* c,
                                             int32_t* __restrict__ ids, float* __restrict__ weights,
                                             int32_t* ids_copy) {
   const int lane = threadIdx.x & 31;
@@ -64,26 +101,21 @@ __device__ __forceinline__ void route_token(const float* __restrict__ row, int p
   }
   for (int e = lane; e < n_experts; e += 32) c[e] = bias ? s[e] + bias[e] : s[e];
   __syncwarp();
+  if (groups.keep < groups.count) {  // the best expert of all is in the best group, the best of the rest in the next, ...
+    const int size = n_experts / groups.count;
+    unsigned long long open = 0;
+    for (int g = 0; g < groups.keep; ++g) {
+      const int e = best_choice(c, n_experts, size, open);
+      if (e != 0x7fffffff) open |= 1ull << (e / size);
+    }
+    __syncwarp();
+    for (int e = lane; e < n_experts; e += 32)
+      if (!(open >> (e / size) & 1)) c[e] = -INFINITY;
+    __syncwarp();
+  }
   float wsum = 0.f;
   for (int j = 0; j < top_k; ++j) {
-    float best = -INFINITY;
-    int bi = 0x7fffffff;
-    for (int e = lane; e < n_experts; e += 32) {
-      const float v = c[e];
-      if (v > best) {  // ascending e within a lane: the first of equal values stays
-        best = v;
-        bi = e;
-      }
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ob > best || (ob == best && oi < bi)) {
-        best = ob;
-        bi = oi;
-      }
-    }
+    int bi = best_choice(c, n_experts, 0, 0);
     if (bi == 0x7fffffff) bi = 0;  // every remaining choice is NaN or -inf
     const float w = s[bi];
     wsum += w;
@@ -95,7 +127,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ row, int p
     }
     __syncwarp();
   }
-  const float denom = scoring == FTK_SCORE_SIGMOID_RAW ? 1.f : scoring == FTK_SCORE_SOFTMAX_OF_CHOSEN ? wsum : wsum + 1e-20f;  // (raw: the scores as they are)
+  const float denom = weight_denominator(scoring, wsum);
   for (int j = lane; j < top_k; j += 32) weights[j] = weights[j] / denom * scale;
 }
 
@@ -110,7 +142,7 @@ __device__ __forceinline__ unsigned int order_key(float v) {
 
 template <int PER>
 __device__ __forceinline__ void route_token_regs(const float* __restrict__ row, int part_stride, int n_parts, const float* __restrict__ bias,
-                                                 int n_experts, int top_k, int scoring, float scale, float* wbuf,
+                                                 int n_experts, RouteGroups groups, int top_k, int scoring, float scale, float* wbuf,
                                                  int32_t* __restrict__ ids, float* __restrict__ weights,
                                                  int32_t* ids_copy) {
   const int lane = threadIdx.x & 31;
@@ -156,6 +188,31 @@ __device__ __forceinline__ void route_token_regs(const float* __restrict__ row, 
     const int e = q * 32 + lane;
     key[q] = e < n_experts ? order_key(bias ? sv[q] + bias[e] : sv[q]) : 0u;
   }
+  if (groups.keep < groups.count) {  // (see route_token)
+    const int size = n_experts / groups.count;
+    unsigned int open = 0;  // a bit per slot of the lane
+    for (int g = 0; g < groups.keep; ++g) {
+      unsigned int best = 0u;
+      int slot = 0;
+#pragma unroll
+      for (int q = 0; q < PER; ++q)
+        if (key[q] > best && !(open >> q & 1)) {
+          best = key[q];
+          slot = q;
+        }
+      const unsigned int top = __reduce_max_sync(0xffffffffu, best);
+      if (top <= floor_key) break;
+      const int first = (int)__reduce_min_sync(0xffffffffu, best == top ? (unsigned)(slot * 32 + lane) : 0x7fffffffu) / size * size;
+#pragma unroll
+      for (int q = 0; q < PER; ++q) {
+        const int e = q * 32 + lane;
+        if (e >= first && e < first + size) open |= 1u << q;
+      }
+    }
+#pragma unroll
+    for (int q = 0; q < PER; ++q)
+      if (!(open >> q & 1)) key[q] = 0u;
+  }
   float wsum = 0.f;
   for (int j = 0; j < top_k; ++j) {
     unsigned int best = 0u;
@@ -188,29 +245,29 @@ __device__ __forceinline__ void route_token_regs(const float* __restrict__ row, 
     }
   }
   __syncwarp();
-  const float denom = scoring == FTK_SCORE_SIGMOID_RAW ? 1.f : scoring == FTK_SCORE_SOFTMAX_OF_CHOSEN ? wsum : wsum + 1e-20f;  // (raw: the scores as they are)
+  const float denom = weight_denominator(scoring, wsum);
   for (int j = lane; j < top_k; j += 32) weights[j] = wbuf[j] / denom * scale;
   __syncwarp();
 }
 
 // One token by one warp, in registers where the experts fit; `s` holds 2 * n_experts floats.
 __device__ __forceinline__ void route_one(const float* __restrict__ row, int part_stride, int n_parts, const float* __restrict__ bias, int n_experts,
-                                          int top_k, int scoring, float scale, float* s, int32_t* __restrict__ ids,
+                                          RouteGroups groups, int top_k, int scoring, float scale, float* s, int32_t* __restrict__ ids,
                                           float* __restrict__ weights, int32_t* ids_copy) {
   if (n_experts <= 128)
-    route_token_regs<4>(row, part_stride, n_parts, bias, n_experts, top_k, scoring, scale, s, ids, weights, ids_copy);
+    route_token_regs<4>(row, part_stride, n_parts, bias, n_experts, groups, top_k, scoring, scale, s, ids, weights, ids_copy);
   else if (n_experts <= 256)
-    route_token_regs<8>(row, part_stride, n_parts, bias, n_experts, top_k, scoring, scale, s, ids, weights, ids_copy);
+    route_token_regs<8>(row, part_stride, n_parts, bias, n_experts, groups, top_k, scoring, scale, s, ids, weights, ids_copy);
   else if (n_experts <= 512)
-    route_token_regs<16>(row, part_stride, n_parts, bias, n_experts, top_k, scoring, scale, s, ids, weights, ids_copy);
+    route_token_regs<16>(row, part_stride, n_parts, bias, n_experts, groups, top_k, scoring, scale, s, ids, weights, ids_copy);
   else
-    route_token(row, part_stride, n_parts, bias, n_experts, top_k, scoring, scale, s, s + n_experts, ids, weights, ids_copy);
+    route_token(row, part_stride, n_parts, bias, n_experts, groups, top_k, scoring, scale, s, s + n_experts, ids, weights, ids_copy);
 }
 
 __global__ void router_topk_kernel(const float* __restrict__ logits, int n_parts, const float* __restrict__ bias,
                                    int n_tokens, int n_experts, int top_k, int scoring, float scale,
                                    int32_t* __restrict__ ids, float* __restrict__ weights, int n_extra, int n_pad, int n_real,
-                                   float* __restrict__ aux) {
+                                   float* __restrict__ aux, RouteGroups groups) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ float sm[];
@@ -220,7 +277,7 @@ __global__ void router_topk_kernel(const float* __restrict__ logits, int n_parts
   float* s = sm + (size_t)warp * 2 * n_experts;  // unbiased scores
   const int stride = n_experts + n_extra + n_pad;
   const float* row = logits + (size_t)t * n_parts * stride;
-  route_one(row, stride, n_parts, bias, n_experts, top_k, scoring, scale, s, ids + (size_t)t * top_k,
+  route_one(row, stride, n_parts, bias, n_experts, groups, top_k, scoring, scale, s, ids + (size_t)t * top_k,
             weights + (size_t)t * top_k, nullptr);
   if (aux)
     token_aux(row, stride, n_parts, n_experts, n_extra, n_real, ids + (size_t)t * top_k, weights + (size_t)t * top_k, top_k,
@@ -272,7 +329,7 @@ moe_route_kernel(const float* __restrict__ x, const float* __restrict__ w, const
                  int n_tokens, int hidden, int n_experts, int top_k, int scoring, float scale,
                  float* __restrict__ logits, int32_t* __restrict__ ids, float* __restrict__ weights,
                  int32_t* __restrict__ counts, int32_t* __restrict__ offsets, int32_t* __restrict__ routes,
-                 int32_t* __restrict__ pos, int do_sort, int n_extra, int n_real, float* __restrict__ aux) {
+                 int32_t* __restrict__ pos, int do_sort, int n_extra, int n_real, float* __restrict__ aux, RouteGroups groups) {
   const int n_rows = n_experts + n_extra;  // rows of the weight, logits of a token
   extern __shared__ float sm[];
   __shared__ float part[kRouteVals][kRouteWarps + 1];
@@ -346,7 +403,7 @@ moe_route_kernel(const float* __restrict__ x, const float* __restrict__ w, const
   float* s = sm + (size_t)warp * 2 * n_experts;
   for (int t = warp; t < n_tokens; t += kRouteWarps) {
     const float* row = logits + (size_t)t * n_rows;
-    route_one(row, n_rows, 1, bias ? sbias : nullptr, n_experts, top_k, scoring, scale, s, ids + (size_t)t * top_k,
+    route_one(row, n_rows, 1, bias ? sbias : nullptr, n_experts, groups, top_k, scoring, scale, s, ids + (size_t)t * top_k,
               weights + (size_t)t * top_k, do_sort ? sid + (size_t)t * top_k : nullptr);
     if (aux)
       token_aux(row, n_rows, 1, n_experts, n_extra, n_real, ids + (size_t)t * top_k, weights + (size_t)t * top_k, top_k,
@@ -387,12 +444,20 @@ moe_route_kernel(const float* __restrict__ x, const float* __restrict__ w, const
 
 using namespace ftk;
 
+// (more than 512 experts are chosen from with a bit per group: at most 64 of them)
+static bool groups_ok(int n_experts, int count, int keep, int top_k) {
+  return count >= 1 && keep >= 1 && keep <= count && n_experts % count == 0 && (n_experts <= 512 || count <= 64) &&
+         (keep == count || top_k <= n_experts / count * keep);
+}
+
 extern "C" int ftk_router_topk(const float* logits, int n_parts, const float* bias, int n_tokens, int n_experts, int top_k,
                                int scoring, float scale, int32_t* ids, float* weights, int n_extra, int n_pad, int n_real, float* aux,
-                               void* stream) {
+                               int n_groups, int keep_groups, void* stream) {
+  FTK_REQUIRE(groups_ok(n_experts, n_groups, keep_groups, top_k), "router_topk: %d of %d groups of %d experts, top %d", keep_groups,
+              n_groups, n_experts, top_k);
   FTK_REQUIRE((n_extra == 0 || n_extra == 1) && n_pad >= 0 && n_real >= 0 && n_real <= n_experts, "router_topk: bad extra logits or expert counts");
   FTK_REQUIRE(n_parts >= 1 && n_parts <= 4, "router_topk: %d blocks of logits per token (1 to 4)", n_parts);
-  FTK_REQUIRE(scoring >= FTK_SCORE_SIGMOID && scoring <= FTK_SCORE_SIGMOID_RAW, "router_topk: unknown scoring %d", scoring);
+  FTK_REQUIRE(scoring >= FTK_SCORE_SIGMOID && scoring <= FTK_SCORE_SOFTMAX_RAW, "router_topk: unknown scoring %d", scoring);
   FTK_REQUIRE(n_experts >= 1 && top_k >= 1 && top_k <= n_experts, "router_topk: top_k=%d of %d experts", top_k, n_experts);
   FTK_REQUIRE(n_tokens >= 0, "router_topk: bad token count");
   if (n_tokens == 0) return 0;
@@ -403,7 +468,7 @@ extern "C" int ftk_router_topk(const float* logits, int n_parts, const float* bi
   const int blocks = (n_tokens + kRouterWarps - 1) / kRouterWarps;
   note_variant(n_parts > 1 ? "routing: expert choice from logits given in pieces" : "routing: expert choice from given logits");
   FTK_LAUNCH(router_topk_kernel, blocks, kRouterWarps * 32, smem, (cudaStream_t)stream, logits, n_parts, bias, n_tokens, n_experts, top_k,
-                                                                               scoring, scale, ids, weights, n_extra, n_pad, n_real, aux);
+                                                                               scoring, scale, ids, weights, n_extra, n_pad, n_real, aux, RouteGroups{n_groups, keep_groups});
   FTK_LAUNCH_CHECK("router_topk");
   return 0;
 }
@@ -420,9 +485,12 @@ extern "C" int ftk_moe_route_fits(int n_tokens, int hidden, int n_experts, int t
 extern "C" int ftk_moe_route(const float* x, const float* gate_w, const float* bias, int n_tokens, int hidden,
                              int n_experts, int top_k, int scoring, float scale, float* logits, int32_t* ids,
                              float* weights, int32_t* counts, int32_t* offsets, int32_t* routes, int32_t* pos,
-                             int do_sort, int n_extra, int n_real, float* aux, void* stream) {
+                             int do_sort, int n_extra, int n_real, float* aux, int n_groups, int keep_groups,
+                             void* stream) {
+  FTK_REQUIRE(groups_ok(n_experts, n_groups, keep_groups, top_k), "moe_route: %d of %d groups of %d experts, top %d", keep_groups,
+              n_groups, n_experts, top_k);
   FTK_REQUIRE((n_extra == 0 || n_extra == 1) && n_real >= 0 && n_real <= n_experts, "moe_route: bad extra logits or expert counts");
-  FTK_REQUIRE(scoring >= FTK_SCORE_SIGMOID && scoring <= FTK_SCORE_SIGMOID_RAW, "moe_route: unknown scoring %d", scoring);
+  FTK_REQUIRE(scoring >= FTK_SCORE_SIGMOID && scoring <= FTK_SCORE_SOFTMAX_RAW, "moe_route: unknown scoring %d", scoring);
   FTK_REQUIRE(ftk_moe_route_fits(n_tokens, hidden, n_experts, top_k),
               "moe_route: %d tokens, width %d, %d experts, top %d do not fit the one-launch routing (at most 32 tokens, "
               "a width that is a multiple of 4); use the matrix product + router_topk + moe_permute",
@@ -436,7 +504,7 @@ extern "C" int ftk_moe_route(const float* x, const float* gate_w, const float* b
   note_variant(do_sort ? "routing: product, choice and sort in one launch" : "routing: product and choice in one launch");
   FTK_LAUNCH(moe_route_kernel, blocks, kRouteWarps * 32, smem, (cudaStream_t)stream, 
       x, gate_w, bias, n_tokens, hidden, n_experts, top_k, scoring, scale, logits, ids, weights, counts, offsets, routes, pos,
-      do_sort, n_extra, n_real, aux);
+      do_sort, n_extra, n_real, aux, RouteGroups{n_groups, keep_groups});
   FTK_LAUNCH_CHECK("moe_route");
   return 0;
 }

@@ -125,8 +125,13 @@ def build_plan(segments: Sequence[Tuple[int, int]], group: int, tile_rows: int,
                max_splits: int = 32, min_split_keys: int = 256,
                fixed_splits: Optional[int] = None,
                sparse: Optional[Tuple[int, int]] = None, key_tile: Optional[int] = None,
-               costs: Optional[PieceCosts] = None) -> AttentionPlan:
+               costs: Optional[PieceCosts] = None, keep_first: int = 0) -> AttentionPlan:
     """``segments`` holds (q_len, kv_len) per segment, in step order.
+
+    ``keep_first`` (with a window): every query also reads the positions below it.  A tile's keys are then numbered: first
+    the positions ``0 .. K - 1``, ``K`` being ``keep_first`` rounded up to the kernel's key quantum (``key_tile`` or
+    ``SPLIT_QUANTUM``), then the tile's window from the quantum that holds its first key on (nothing is left out where that
+    lies within the first ``K``); the kernels turn numbers back into positions.
 
     ``fixed_splits`` fixes the number of item rows at that many per tile on average: the rows are dealt
     to the tiles in proportion to their key spans (:func:`deal_rows`; a request of 20,000 tokens beside one
@@ -165,6 +170,10 @@ def build_plan(segments: Sequence[Tuple[int, int]], group: int, tile_rows: int,
         block, topk = sparse
         lo = np.zeros_like(hi)
         hi = np.minimum(topk, (pos0 + tok0) // block + 1) * block
+    if window is not None and keep_first:
+        q = key_tile if key_tile else SPLIT_QUANTUM
+        jump = np.maximum(0, lo // q * q - -(-keep_first // q) * q)  # positions between the kept tokens and the window
+        lo, hi = np.zeros_like(lo), hi - jump
     spans = hi - lo
     n_tiles = int(spans.shape[0])
     target = 2 * sm_count

@@ -109,24 +109,30 @@ class StepBuilder:
         longest = max(kv for _, kv in self.seg_lens)
         return 1 << max(6, (longest - 1).bit_length())
 
-    def fixed_splits(self, n_kv_heads: int, ctas_per_sm: int = 2) -> int:
+    def fixed_splits(self, n_kv_heads: int, ctas_per_sm: int = 2, most_keys: Optional[int] = None) -> int:
         """Splits per tile of a graph-replayed decode step: enough CTAs to fill the GPU at
-        this batch size, independent of the requests' exact lengths."""
+        this batch size, independent of the requests' exact lengths.  ``most_keys``: what a window leaves a
+        tile at most; pieces are then no shorter than a split's worth."""
         b = max(1, len(self.seg_lens))
-        return wave_splits(b * n_kv_heads, ctas_per_sm * self.sm_count, 16, self.longest_span())
+        span, limit = self.longest_span(), 16
+        if most_keys is not None and most_keys < span:
+            span, limit = most_keys, max(1, min(limit, most_keys // 256))
+        return wave_splits(b * n_kv_heads, ctas_per_sm * self.sm_count, limit, span)
 
     def attention_plan(self, group: int, tile_rows: int, window: Optional[int], n_kv_heads: int,
-                       head_dim: int, few_rows: bool = False) -> Any:
-        """``few_rows``: the work list is for the tcgen05 kernel in its form for tiles of at most 16 rows (key tiles of 128)."""
-        key = ("attention", group, tile_rows, window, n_kv_heads, head_dim, few_rows)
+                       head_dim: int, few_rows: bool = False, keep_first: int = 0) -> Any:
+        """``few_rows``: the work list is for the tcgen05 kernel in its form for tiles of at most 16 rows (key tiles of 128).
+        ``keep_first``: first tokens that the window keeps."""
+        key = ("attention", group, tile_rows, window, n_kv_heads, head_dim, few_rows) + ((keep_first,) if keep_first else ())
         if key not in self.plans:
-            plan = self._drafts.pop(key, None) or self._draft(group, tile_rows, window, n_kv_heads, few_rows)
+            plan = self._drafts.pop(key, None) or self._draft(group, tile_rows, window, n_kv_heads, few_rows, keep_first)
             self.plans[key] = plan
             self.plan_dims[key] = (n_kv_heads, tile_rows, head_dim)
             self.add(f"plan.{len(self.plans) - 1}", plan.items)
         return key
 
-    def _draft(self, group: int, tile_rows: int, window: Optional[int], n_kv_heads: int, few_rows: bool) -> AttentionPlan:
+    def _draft(self, group: int, tile_rows: int, window: Optional[int], n_kv_heads: int, few_rows: bool,
+               keep_first: int = 0) -> AttentionPlan:
         tensor_core = tile_rows >= 128 or few_rows
         per_sm = 1 if tensor_core else 2  # the tcgen05 kernels fill an SM with one CTA
         costs = None
@@ -134,8 +140,9 @@ class StepBuilder:
             costs = TC_TWO_TILE_COSTS if tile_rows == 256 else TC_ONE_TILE_COSTS
         return build_plan(self.seg_lens, group, tile_rows, window, n_kv_heads,
                           sm_count=self.sm_count if per_sm == 2 else max(1, self.sm_count // 2),
-                          fixed_splits=self.fixed_splits(n_kv_heads, per_sm) if self.fixed else None,
-                          key_tile=128 if tensor_core else 0, costs=costs)
+                          fixed_splits=self.fixed_splits(n_kv_heads, per_sm, None if window is None else window + keep_first)
+                          if self.fixed else None,
+                          key_tile=128 if tensor_core else 0, costs=costs, keep_first=keep_first)
 
     def cheaper_attention_rows(self, group: int, window: Optional[int], n_kv_heads: int, head_dim: int) -> int:
         """128 or 256: the tcgen05 attention kernel (one or two query tiles a piece) whose work list for this step

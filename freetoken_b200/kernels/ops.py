@@ -59,7 +59,7 @@ ACT_SILU, ACT_SWIGLUOAI = 0, 1
 SCORE_SIGMOID, SCORE_SOFTMAX, SCORE_SOFTMAX_OF_CHOSEN = 0, 1, 2
 ACT_CODES = {"silu": ACT_SILU, "swigluoai": ACT_SWIGLUOAI}
 SCORE_CODES = {"sigmoid": SCORE_SIGMOID, "softmax": SCORE_SOFTMAX, "softmax_of_chosen": SCORE_SOFTMAX_OF_CHOSEN,
-               "sigmoid_raw": 3}
+               "sigmoid_raw": 3, "softmax_raw": 4}
 
 _vp = ctypes.c_void_p
 _i = ctypes.c_int
@@ -84,15 +84,16 @@ class _StreamNorm(ctypes.Structure):
 
 class _AttnExtras(ctypes.Structure):
     _fields_ = [("dist_bias", _vp), ("dist_len", _i), ("kv_split", _i), ("has_sink", _i), ("sink_logit", _f),
-                ("sink_heads", _vp), ("softcap", _f)]
+                ("sink_heads", _vp), ("softcap", _f), ("keep_first", _i)]
 
 
 class _StreamStep(ctypes.Structure):
     _fields_ = [
-        ("residual", _vp), ("vec", _vp), ("x", _vp), ("route_pos", _vp), ("top_k", _i), ("n_routes", _i), ("aux", _vp),
+        ("residual", _vp), ("vec", _vp), ("x", _vp), ("x2", _vp), ("x_scale", _f), ("x2_scale", _f), ("route_pos", _vp),
+        ("top_k", _i), ("n_routes", _i), ("aux", _vp),
         ("passed", _vp), ("shared", _vp), ("gate", _vp), ("gate_bias", _vp), ("post_w", _vp), ("post_eps", _f),
         ("raw_out", _vp), ("raw_stride", ctypes.c_longlong), ("pre_w", _vp), ("pre_eps", _f), ("out", _vp),
-        ("norm_f32", _vp), ("conv_w", _vp), ("taps", _i), ("state", _vp), ("n_slots", _i), ("state_slots", _vp),
+        ("norm_f32", _vp), ("f32_rounded", _i), ("conv_w", _vp), ("taps", _i), ("state", _vp), ("n_slots", _i), ("state_slots", _vp),
         ("seg_info", _vp), ("conv_out", _vp), ("conv_out_f32", _vp), ("rows", _vp), ("n_rows", _i), ("hidden", _i),
         ("groups", _i), ("dtype", _i),
     ]
@@ -112,7 +113,7 @@ _SIGNATURES = {
     "ftk_embedding_gather": [_vp, _i, _vp, _i, _i, _i, _vp, _vp],
     "ftk_add_rmsnorm": [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _f, _i, _vp],
     "ftk_add_rmsnorm_routes": [_vp, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _f, _i, _vp],
-    "ftk_norm_rope_store": [_vp, _i, _i, _i, _i, _i, _vp, _vp, _i, _f, _i, _i,
+    "ftk_norm_rope_store": [_vp, _i, _i, _i, _i, _i, _vp, _vp, _i, _f, _i, _i, _i,
                             ctypes.POINTER(_Section), _vp],
     "ftk_paged_attention": [_vp, _vp, _vp, _i, _vp, _i, _vp, _i, _vp, _i, _vp, _vp, _i, _vp,
                             _i, _i, _i, _i, _i, _i, _f, _i, _vp],
@@ -136,10 +137,11 @@ _SIGNATURES = {
                                    _i, _i, _i, _i, _i, _i, _f, _vp, _i, _i, _vp],
     "ftk_sparse_select": [_vp, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp],
     "ftk_sparse_score_fits": [_i, _i, _i],
-    "ftk_router_topk": [_vp, _i, _vp, _i, _i, _i, _i, _f, _vp, _vp, _i, _i, _i, _vp, _vp],
+    "ftk_router_topk": [_vp, _i, _vp, _i, _i, _i, _i, _f, _vp, _vp, _i, _i, _i, _vp, _i, _i, _vp],
     "ftk_moe_permute": [_vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp],
     "ftk_moe_route_fits": [_i, _i, _i, _i],
-    "ftk_moe_route": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _vp],
+    "ftk_moe_route": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _i,
+                      _vp],
     "ftk_small_linear_fits": [_i, _i, _i],
     "ftk_small_linear": [_vp, _vp, _vp, _i, _i, _i, _vp],
     "ftk_moe_small_fits": [_i, _i, _i, _i],
@@ -177,11 +179,12 @@ _SIGNATURES = {
     "ftk_mlstm_gates": [_vp, _vp, _vp, _f, _vp, _i, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp],
     "ftk_mlstm_output": [_vp, _vp, _vp, _vp, ctypes.c_longlong, _vp, _f, _vp, _i, _i, _i, _i, _vp],
     "ftk_gla_scan": [_vp, ctypes.c_longlong, _vp, ctypes.c_longlong, _vp, ctypes.c_longlong, _i, _vp, _vp, _f, _f,
-                     _vp, _i, _vp, _vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _i, _vp, _i, _vp],
+                     _vp, _i, _vp, _vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _i, _i, _vp, _i,
+                     _vp, _i, _i, _i, _vp],
     "ftk_hyper_step": [_vp, ctypes.c_longlong, _i, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _f, _vp, _i, _vp, _vp],
     "ftk_conv_act": [_vp, ctypes.c_longlong, _i, _vp, _vp, _i, _i, _vp, _i, _vp, _vp, _i, _vp, _i, _i, _vp],
     "ftk_delta_scan": [_vp, ctypes.c_longlong, _vp, ctypes.c_longlong, _vp, ctypes.c_longlong, _vp, ctypes.c_longlong,
-                       _vp, ctypes.c_longlong, _i, _vp, _vp, _f, _f, _vp, _i, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _vp],
+                       _vp, ctypes.c_longlong, _vp, _i, _vp, _vp, _f, _f, _vp, _i, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _vp],
     "ftk_ssm_gates": [_vp, ctypes.c_longlong, _i, _vp, _vp, _vp, _vp, _i, _i, _vp],
     "ftk_ssm_output": [_vp, _vp, ctypes.c_longlong, _vp, _vp, ctypes.c_longlong, _i, _vp, _i, _f, _vp, _i, _i, _i, _vp],
     "ftk_norm_mean": [ctypes.POINTER(_vp), ctypes.POINTER(_vp), _i, _i, _f, _vp, _i, _i, _vp],
@@ -397,7 +400,7 @@ def cast(src: torch.Tensor, dst: torch.Tensor) -> None:
 # --------------------------------------------------------------------------- attention
 def norm_rope_store(x: torch.Tensor, head_dim: int, rotary_dim: int, positions: torch.Tensor,
                     rope_table: Optional[torch.Tensor], eps: float, gemma: bool,
-                    sections: Sequence[dict]) -> None:
+                    sections: Sequence[dict], neighbours: bool = False) -> None:
     """Per-head RMSNorm, partial NeoX rotation and scatter of projected heads, in one pass.
 
     ``x [T, n_heads_total * head_dim]`` is cut into sections of whole heads.  A section is a
@@ -405,7 +408,8 @@ def norm_rope_store(x: torch.Tensor, head_dim: int, rotary_dim: int, positions: 
     ``rotate`` (bool), and one destination: ``dense_out [T, n_heads, head_dim]`` or
     ``slab [pages, n_heads, page_size, head_dim]`` with ``slot_map [T]`` (slot = page *
     page_size + offset, negative = skip).  ``rope_table [max_pos, rotary_dim]`` holds
-    cos then sin of ``position * inv_freq`` in float32.
+    cos then sin of ``position * inv_freq`` in float32; pairs that turn together are the halves of the rotated span,
+    or with ``neighbours`` the dimensions ``(2i, 2i + 1)``.  ``x`` may be a view of adjacent columns of a wider tensor.
 
     Optional keys of a section: ``bias`` (float32 ``[n_heads * head_dim]``, added first),
     ``pos_scale`` (float32 ``[positions]``, the heads are multiplied last by the entry of the
@@ -453,10 +457,12 @@ def norm_rope_store(x: torch.Tensor, head_dim: int, rotary_dim: int, positions: 
         if rope_table is None or rope_table.shape[1] != rotary_dim:
             raise KernelError("norm_rope_store: rope_table must be [max_pos, rotary_dim]")
     max_pos = rope_table.shape[0] if rope_table is not None else 0
-    _check(_lib().ftk_norm_rope_store(_dev(x, "x"), _code(x, "x"), T, x.shape[1], head_dim, rotary_dim,
+    if not x.is_cuda or x.stride(1) != 1:
+        raise KernelError("norm_rope_store: x must be rows of adjacent elements on the device")
+    _check(_lib().ftk_norm_rope_store(x.data_ptr(), _code(x, "x"), T, x.stride(0) if T > 1 else x.shape[1], head_dim, rotary_dim,
                                       _dev(positions, "positions", torch.int32),
                                       _dev(rope_table, "rope_table", torch.float32), max_pos,
-                                      float(eps), 1 if gemma else 0, len(sections), arr, _stream()),
+                                      float(eps), 1 if gemma else 0, 1 if neighbours else 0, len(sections), arr, _stream()),
            "norm_rope_store")
 
 
@@ -466,7 +472,7 @@ def paged_attention(q: torch.Tensor, k_slab: torch.Tensor, v_slab: torch.Tensor,
                     part_ml: Optional[torch.Tensor], out: torch.Tensor, tile_rows: int, scale: float,
                     window: Optional[int], sel: Optional[torch.Tensor] = None, block_size: int = 0,
                     few_rows: bool = False, dist_bias: Optional[torch.Tensor] = None, kv_split: int = 1,
-                    sink: Any = None, softcap: Optional[float] = None) -> None:
+                    sink: Any = None, softcap: Optional[float] = None, keep_first: int = 0) -> None:
     """Causal softmax attention of the step's queries over the paged keys and values.
 
     ``q, out [T, Hq, D]``; slabs ``[pages, Hkv, page_size, D]``; ``block_table [rows, width]``
@@ -502,7 +508,14 @@ def paged_attention(q: torch.Tensor, k_slab: torch.Tensor, v_slab: torch.Tensor,
 
     ``softcap`` (positive, or None): scaled scores ``s`` become ``softcap * tanh(s / softcap)`` before the softmax.  Not with
     block selection or a bias by distance; every tcgen05 form takes it.
+
+    ``keep_first`` (with a window; the work list from ``build_plan(..., keep_first=...)``): positions below it stay visible
+    however far back they are.  Of the tcgen05 kernels the one with 128-row tiles takes it; not with a bias by distance,
+    block selection or a soft cap.
     """
+    keep_first = int(keep_first or 0)
+    if keep_first and (keep_first < 0 or not window or sel is not None or dist_bias is not None or softcap):
+        raise KernelError("paged_attention: kept first tokens go with a window, without bias, soft cap or block selection")
     softcap = 0.0 if softcap is None else float(softcap)
     if softcap < 0 or (softcap and (sel is not None or dist_bias is not None)):
         raise KernelError("paged_attention: a soft cap is positive, without block selection or a distance bias")
@@ -540,7 +553,8 @@ def paged_attention(q: torch.Tensor, k_slab: torch.Tensor, v_slab: torch.Tensor,
                 raise KernelError("paged_attention: of the tcgen05 kernels the ones with one query tile a piece take a "
                                   "distance bias [Hq, L] (no window)")
             ex = _AttnExtras(_dev(dist_bias, "dist_bias", torch.float32), dist_bias.shape[1] if dist_bias is not None else 0,
-                             1, 0 if sink is None else 1, 0.0 if sink is None else float(sink), sink_heads, softcap)
+                             1, 0 if sink is None else 1, 0.0 if sink is None else float(sink), sink_heads, softcap,
+                             keep_first)
             what = "soft cap" if softcap else "distance bias" if dist_bias is not None else "window or sink"
             _check(_lib().ftk_paged_attention_tc_ex(
                 _dev(q, "q"), _dev(k_slab, "k_slab"), _dev(v_slab, "v_slab"),
@@ -578,11 +592,12 @@ def paged_attention(q: torch.Tensor, k_slab: torch.Tensor, v_slab: torch.Tensor,
             _dev(sel, "sel", torch.int32), sel.shape[2], int(block_size), _stream()),
             "paged_attention (block-sparse)", 2 if n_slots else 1)
         return
-    if dist_bias is not None or kv_split > 1 or sink is not None or softcap:
+    if dist_bias is not None or kv_split > 1 or sink is not None or softcap or keep_first:
         if dist_bias is not None and (dist_bias.dim() != 2 or dist_bias.shape[0] != Hq or dist_bias.shape[1] < 1):
             raise KernelError("paged_attention: dist_bias must be [Hq, L]")
         ex = _AttnExtras(_dev(dist_bias, "dist_bias", torch.float32), dist_bias.shape[1] if dist_bias is not None else 0,
-                         kv_split, 0 if sink is None else 1, 0.0 if sink is None else float(sink), sink_heads, softcap)
+                         kv_split, 0 if sink is None else 1, 0.0 if sink is None else float(sink), sink_heads, softcap,
+                             keep_first)
         _check(_lib().ftk_paged_attention_ex(
             _dev(q, "q"), _dev(k_slab, "k_slab"), _dev(v_slab, "v_slab"), _code(q, "q"),
             _dev(block_table, "block_table", torch.int32), block_table.shape[1],
@@ -652,13 +667,18 @@ def sparse_select(iq: torch.Tensor, ik_slab: torch.Tensor, block_table: torch.Te
 # --------------------------------------------------------------------------- experts
 def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, scoring: str,
                 scale: float, ids: torch.Tensor, weights: torch.Tensor, n_parts: int = 1, n_extra: int = 0,
-                n_real: Optional[int] = None, aux: Optional[torch.Tensor] = None, n_pad: int = 0) -> None:
+                n_real: Optional[int] = None, aux: Optional[torch.Tensor] = None, n_pad: int = 0,
+                groups: Sequence[int] = (1, 1)) -> None:
     """Expert choice from float32 router logits ``[T, E]``.
 
     sigmoid: ``s = sigmoid(l)``; choice by ``s + bias``; ``w = s[ids] / (sum + 1e-20) * scale``.
     softmax: ``s = softmax(l)``; choice by ``s (+ bias)``; ``w = s[ids] / sum * scale``.
     softmax_of_chosen: the bias belongs to the logit: choice by ``l + bias``; ``w = softmax((l + bias)[ids]) * scale``.
+    softmax_raw, sigmoid_raw: the chosen experts' scores (times ``scale``) as they are.
     The largest goes first; the lower expert index wins a tie.
+
+    ``groups = (count, keep)``: the experts form ``count`` equal groups of neighbours, and only experts of the ``keep`` groups
+    with the largest choice in them can be chosen.
 
     With ``n_parts > 1`` the logits come as ``[T, n_parts * E]``: a token's logit of expert ``e`` is the
     32-bit sum of ``logits[t, q * E + e]`` over the parts ``q`` in their order.
@@ -682,8 +702,8 @@ def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, 
     _check(_lib().ftk_router_topk(_dev(logits, "logits", torch.float32), int(n_parts), _dev(bias, "bias", torch.float32),
                                   T, E, top_k, SCORE_CODES[scoring], float(scale),
                                   _dev(ids, "ids", torch.int32), _dev(weights, "weights", torch.float32),
-                                  int(n_extra), int(n_pad), n_real, _dev(aux, "aux", torch.float32), _stream()),
-           "router_topk")
+                                  int(n_extra), int(n_pad), n_real, _dev(aux, "aux", torch.float32), int(groups[0]),
+                                  int(groups[1]), _stream()), "router_topk")
 
 
 def moe_permute(topk_ids: torch.Tensor, n_experts: int, expert_counts: torch.Tensor,
@@ -750,7 +770,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[t
             raise KernelError("linear: bias must be [N] of x's dtype")
         torch.addmm(bias, x, w.t(), out=out)
         return
-    if (T <= SMALL_LINEAR_MAX_TOKENS and x.dtype == torch.bfloat16 and x.is_cuda and x.is_contiguous()
+    if (T <= SMALL_LINEAR_MAX_TOKENS and x.dtype == torch.bfloat16 and x.is_cuda and x.is_contiguous() and x.data_ptr() % 16 == 0
             and w.is_contiguous() and out.is_contiguous() and small_linear_fits(T, N, K)):
         small_linear(x, w, out)
         return
@@ -789,10 +809,10 @@ def moe_route(x: torch.Tensor, gate_w: torch.Tensor, bias: Optional[torch.Tensor
               scale: float, logits: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
               expert_counts: Optional[torch.Tensor] = None, expert_offsets: Optional[torch.Tensor] = None,
               sorted_routes: Optional[torch.Tensor] = None, route_pos: Optional[torch.Tensor] = None, n_extra: int = 0,
-              n_real: Optional[int] = None, aux: Optional[torch.Tensor] = None) -> None:
+              n_real: Optional[int] = None, aux: Optional[torch.Tensor] = None, groups: Sequence[int] = (1, 1)) -> None:
     """``logits = x @ gate_w^T`` in float32, then :func:`router_topk` and :func:`moe_permute`, in one launch.
     Without the four outputs of the sort only ids and weights are made (the few-token expert kernels take
-    the routes in token order).  ``n_extra``, ``n_real`` and ``aux`` as in :func:`router_topk` (``gate_w`` and ``logits`` then
+    the routes in token order).  ``n_extra``, ``n_real``, ``aux`` and ``groups`` as in :func:`router_topk` (``gate_w`` and ``logits`` then
     have ``n_extra`` more rows and columns); routes to ids from ``n_real`` on are sorted behind the others and get the
     place -1, and the sort's outputs count ``n_real`` experts."""
     T, H = x.shape
@@ -818,7 +838,7 @@ def moe_route(x: torch.Tensor, gate_w: torch.Tensor, bias: Optional[torch.Tensor
                                 _dev(expert_offsets, "expert_offsets", torch.int32),
                                 _dev(sorted_routes, "sorted_routes", torch.int32),
                                 _dev(route_pos, "route_pos", torch.int32), 1 if sort else 0, int(n_extra), n_real,
-                                _dev(aux, "aux", torch.float32), _stream()), "moe_route")
+                                _dev(aux, "aux", torch.float32), int(groups[0]), int(groups[1]), _stream()), "moe_route")
 
 
 def moe_small_fits(n_tokens: int, hidden: int, inter: int, top_k: int) -> bool:
@@ -1125,12 +1145,13 @@ def gated_heads(x: torch.Tensor, gates: torch.Tensor, out: torch.Tensor, dim: in
         GATE_CODES[act], _dev(out, "out"), out.shape[2], _code(out, "out"), T, H, dim, _stream()), "gated_heads")
 
 
-def gla_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, z_bias: Optional[torch.Tensor],
+def gla_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: Optional[torch.Tensor], z_bias: Optional[torch.Tensor],
              tau: float, q_scale: float, state: torch.Tensor, state_slots: torch.Tensor, seg_info: torch.Tensor,
              n_segs: int, chunks: torch.Tensor, n_chunks: int, seg_chunks: torch.Tensor, any_single: bool,
              any_multi: bool, carry: Optional[torch.Tensor], decay_prod: Optional[torch.Tensor],
              out: torch.Tensor, k_fac: Optional[torch.Tensor] = None, a_head: Optional[torch.Tensor] = None,
-             ones_col: bool = False, out_ones: Optional[torch.Tensor] = None, qk_div: int = 1) -> None:
+             ones_col: bool = False, out_ones: Optional[torch.Tensor] = None, qk_div: int = 1,
+             rope_table: Optional[torch.Tensor] = None, neighbours: bool = False) -> None:
     """Gated linear attention of the step's tokens, per (request, head):
     ``S <- diag(a_t) S + k_t v_t^T``, ``o_t = S^T (q_t q_scale)``, ``a_t = sigmoid(z_t + z_bias)^(1 / tau)``.
 
@@ -1142,13 +1163,18 @@ def gla_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor,
     ``out [T, H, Dv]`` float32.
 
     ``k_fac [T, H]`` float32 multiplies a token's keys of a head (in 32 bits, as they are read); ``a_head [T, H]``
-    float32 gives one decay per (token, head) for all key channels, and ``z`` is then ``None``; with ``ones_col``
+    float32 gives one decay per (token, head) for all key channels (``[H]``: the same for every token), and ``z`` is then
+    ``None``; with ``ones_col``
     the state's last value column belongs to a value that is 1 for every token, and ``v`` is ``[T, H * (Dv - 1)]``
     (the sum of the keys under the same decays: a normaliser); with ``out_ones [T, H]`` that column's outputs go
     there and ``out`` is ``[T, H, Dv - 1]``.
 
     ``qk_div > 1``: queries and keys are shared by groups of that many heads (head ``h`` reads q/k head
-    ``h // qk_div``), and ``q, k`` are ``[T, (H / qk_div) * D]``; with ``a_head`` only."""
+    ``h // qk_div``), and ``q, k`` are ``[T, (H / qk_div) * D]``; with ``a_head`` only.
+
+    ``rope_table [max_pos, n_rot]`` (cos then sin, with ``a_head`` only): the first ``n_rot`` dimensions of every query and
+    key are rotated by the token's position as they are read, in 32 bits (they are never rounded); pairs as in
+    :func:`norm_rope_store`."""
     T = out.shape[0]
     H, D, Dv = state.shape[1], state.shape[2], state.shape[3]
     qk_div = int(qk_div)
@@ -1160,7 +1186,12 @@ def gla_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor,
         raise KernelError("gla_scan: shapes do not agree")
     if out_ones is not None and not ones_col:
         raise KernelError("gla_scan: out_ones goes with ones_col")
-    for name, f in (("k_fac", k_fac), ("a_head", a_head), ("out_ones", out_ones)):
+    one_row = a_head is not None and a_head.dim() == 1
+    if one_row and a_head.shape != (H,):
+        raise KernelError("gla_scan: a_head must be [T, H] or [H]")
+    if rope_table is not None and (a_head is None or rope_table.dim() != 2 or rope_table.shape[1] % 2 or not 2 <= rope_table.shape[1] <= D):
+        raise KernelError("gla_scan: rope_table must be [max_pos, n_rot <= D], with a decay per head")
+    for name, f in (("k_fac", k_fac), ("a_head", None if one_row else a_head), ("out_ones", out_ones)):
         if f is not None and (f.shape != (T, H) or not f.is_contiguous()):
             raise KernelError(f"gla_scan: {name} must be a contiguous [T, H]")
     if q.dtype != k.dtype or q.dtype != v.dtype or q.stride(1) != 1 or k.stride(1) != 1 or v.stride(1) != 1:
@@ -1181,8 +1212,10 @@ def gla_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor,
         _dev(seg_chunks, "seg_chunks", torch.int32), 1 if any_single else 0, 1 if any_multi else 0,
         _dev(carry, "carry", torch.float32), _dev(decay_prod, "decay_prod", torch.float32),
         _dev(out, "out", torch.float32), T, H, D, Dv, _dev(k_fac, "k_fac", torch.float32),
-        _dev(a_head, "a_head", torch.float32), 1 if ones_col else 0, _dev(out_ones, "out_ones", torch.float32),
-        qk_div, _stream()), "gla_scan", max(1, launches))
+        _dev(a_head, "a_head", torch.float32), 0 if one_row else H, 1 if ones_col else 0,
+        _dev(out_ones, "out_ones", torch.float32), qk_div, _dev(rope_table, "rope_table", torch.float32),
+        rope_table.shape[1] if rope_table is not None else 0, 1 if neighbours else 0,
+        rope_table.shape[0] if rope_table is not None else 0, _stream()), "gla_scan", max(1, launches))
 
 
 # --------------------------------------------------------------------------- short convolution, depth mix
@@ -1412,7 +1445,8 @@ def stream_step(residual: torch.Tensor, groups: int = 1, vec: Optional[torch.Ten
                 gate_bias: Optional[torch.Tensor] = None, post_weight: Optional[torch.Tensor] = None, post_eps: float = 0.0,
                 raw_out: Optional[torch.Tensor] = None, pre_weight: Optional[torch.Tensor] = None, pre_eps: float = 0.0,
                 out: Optional[torch.Tensor] = None, norm_f32: Optional[torch.Tensor] = None,
-                conv: Optional[tuple] = None, rows: Optional[torch.Tensor] = None, dtype: Optional[torch.dtype] = None) -> None:
+                conv: Optional[tuple] = None, rows: Optional[torch.Tensor] = None, dtype: Optional[torch.dtype] = None,
+                x2: Optional[torch.Tensor] = None, scales: Sequence[float] = (1.0, 1.0), f32_rounded: bool = False) -> None:
     """One pass over the rows of the 32-bit stream; every part is optional.
 
     ``r += vec``; ``y`` = row ``t`` of ``x``, or, with ``routed = (route_pos, top_k, shared, aux, passed)``, the 32-bit sum
@@ -1420,7 +1454,8 @@ def stream_step(residual: torch.Tensor, groups: int = 1, vec: Optional[torch.Ten
     ``aux`` and ``passed`` may be None); ``y *= sigmoid(gate + gate_bias)``; ``r += groupnorm(y) post_weight``;
     ``raw_out = r`` (rows of the engine's type, any row stride); ``out = groupnorm(r) pre_weight`` and the same unrounded
     in ``norm_f32`` (float32, may be the stream itself).  ``groupnorm`` divides each of ``groups`` equal consecutive parts
-    of a row by its own ``sqrt(mean(part^2) + eps)``.
+    of a row by its own ``sqrt(mean(part^2) + eps)``.  With ``x2``, ``y = scales[0] x + scales[1] x2`` (dense rows);
+    without ``post_weight``, ``r += y``; with ``f32_rounded``, ``norm_f32`` receives ``float32(out)``.
 
     ``conv = (weight [H, taps], state, state_slots, seg_info, conv_out, conv_out_f32 or None)``, for steps of one token per
     request: ``conv_out = h + sum_j weight[:, j] h(t - taps + 1 + j)`` of the normed values as ``out`` stores them, the
@@ -1434,7 +1469,7 @@ def stream_step(residual: torch.Tensor, groups: int = 1, vec: Optional[torch.Ten
     for name, t in (("vec", vec), ("post_weight", post_weight), ("pre_weight", pre_weight), ("gate_bias", gate_bias)):
         if t is not None and t.shape != (H,):
             raise KernelError(f"stream_step: {name} must be [{H}]")
-    for name, t in (("x", x), ("gate", gate), ("out", out), ("raw_out", raw_out)):
+    for name, t in (("x", x), ("x2", x2), ("gate", gate), ("out", out), ("raw_out", raw_out)):
         if t is not None and (t.dtype != dtype or t.shape[-1] != H):
             raise KernelError(f"stream_step: {name} must hold rows of {H} elements of {dtype}")
     for name, t in (("out", out), ("norm_f32", norm_f32)):
@@ -1444,6 +1479,10 @@ def stream_step(residual: torch.Tensor, groups: int = 1, vec: Optional[torch.Ten
         raise KernelError("stream_step: gate has fewer rows than the stream")
     a = _StreamStep()
     a.residual, a.vec = _dev(residual, "residual", torch.float32), _dev(vec, "vec", torch.float32)
+    if x2 is not None and (x is None or routed is not None or x2.numel() < T * H):
+        raise KernelError("stream_step: a second dense tensor goes with a first of as many rows")
+    a.x2, a.x_scale, a.x2_scale = _dev(x2, "x2"), float(scales[0]), float(scales[1])
+    a.f32_rounded = 1 if f32_rounded else 0
     a.x, a.gate, a.gate_bias = _dev(x, "x"), _dev(gate, "gate"), _dev(gate_bias, "gate_bias", torch.float32)
     if routed is not None:
         pos, top_k, shared, aux, passed = routed
@@ -1563,9 +1602,10 @@ def ssm_output(o32: torch.Tensor, x: torch.Tensor, d_skip: torch.Tensor, z: torc
                                  int(norm_groups), float(eps), _dev(out, "out"), T, H, P, _stream()), "ssm_output")
 
 
-def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, b_raw: torch.Tensor, a_raw: torch.Tensor,
+def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, b_raw: torch.Tensor, a_raw: Optional[torch.Tensor],
                a_log: torch.Tensor, dt_bias: torch.Tensor, q_scale: float, unit_eps: float, state: torch.Tensor,
-               state_slots: torch.Tensor, seg_info: torch.Tensor, n_segs: int, out: torch.Tensor) -> None:
+               state_slots: torch.Tensor, seg_info: torch.Tensor, n_segs: int, out: torch.Tensor,
+               z: Optional[torch.Tensor] = None) -> None:
     """The gated delta rule over the step's tokens, per (request, head), a request's tokens in order:
     ``S <- g S``, ``u = beta (v - S^T k)``, ``S <- S + k u^T``, ``o = S^T q``, with ``beta = sigmoid(b_raw)``,
     ``g = exp(-exp(a_log) softplus(a_raw + dt_bias))``, and ``q``, ``k`` first made unit vectors per head
@@ -1574,20 +1614,28 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, b_raw: torch.T
     ``q, k [T, G * D]``, ``v [T, H * Dv]``, ``b_raw, a_raw [T, H]`` of the engine's dtype (views of adjacent columns
     are fine; head ``h`` reads q/k head ``h // (H / G)``); ``a_log, dt_bias [H]`` float32; ``state [slots, H, Dv, D]``
     float32 (``S`` column by column: a value column's key channels are neighbours), read from and left in the slot ``state_slots[segment]`` (a segment with ``kv_len == q_len`` starts from
-    zero); ``out [T, H, Dv]`` float32.  Everything but the reading of the rows is 32-bit."""
+    zero); ``out [T, H, Dv]`` float32.  Everything but the reading of the rows is 32-bit.
+
+    ``z [T, H * D]`` (float32, ``a_raw`` is then None and ``dt_bias [H * D]``): one decay per head and key channel,
+    ``g[d] = exp(-exp(a_log) softplus(z[d] + dt_bias[d]))``, on the rows of ``S`` that belong to key channels; when a segment
+    has several tokens, ``z`` is overwritten with the decays."""
     T, H, Dv = out.shape
     D = state.shape[3]
+    if (a_raw is None) == (z is None) or (z is not None and z.shape != (T, H * D)):
+        raise KernelError("delta_scan: either a_raw [T, H] or z [T, H * D]")
     if state.shape[1] != H or state.shape[2] != Dv or q.shape[1] % D or H % (q.shape[1] // D) or D > 256:
         raise KernelError("delta_scan: shapes do not agree (keys of at most 256 channels)")
     G = q.shape[1] // D
     qs, ks = _cols(q, "delta_scan: q", (T, G * D)), _cols(k, "delta_scan: k", (T, G * D), q.dtype)
     vs = _cols(v, "delta_scan: v", (T, H * Dv), q.dtype)
-    bs, as_ = _cols(b_raw, "delta_scan: b_raw", (T, H), q.dtype), _cols(a_raw, "delta_scan: a_raw", (T, H), q.dtype)
-    if a_log.shape != (H,) or dt_bias.shape != (H,):
-        raise KernelError("delta_scan: a_log and dt_bias must be [H]")
+    bs = _cols(b_raw, "delta_scan: b_raw", (T, H), q.dtype)
+    as_ = _cols(a_raw, "delta_scan: a_raw", (T, H), q.dtype) if z is None else 0
+    if a_log.shape != (H,) or dt_bias.shape != ((H,) if z is None else (H * D,)):
+        raise KernelError("delta_scan: a_log must be [H], dt_bias [H] (or [H * D] with a decay per channel)")
     _check(_lib().ftk_delta_scan(
-        q.data_ptr(), qs, k.data_ptr(), ks, v.data_ptr(), vs, b_raw.data_ptr(), bs, a_raw.data_ptr(), as_, _code(q, "q"),
+        q.data_ptr(), qs, k.data_ptr(), ks, v.data_ptr(), vs, b_raw.data_ptr(), bs,
+        a_raw.data_ptr() if z is None else None, as_, _dev(z, "z", torch.float32), _code(q, "q"),
         _dev(a_log, "a_log", torch.float32), _dev(dt_bias, "dt_bias", torch.float32), float(q_scale), float(unit_eps),
         _dev(state, "state", torch.float32), state.shape[0], _dev(state_slots, "state_slots", torch.int32),
         _dev(seg_info, "seg_info", torch.int32), n_segs, _dev(out, "out", torch.float32), T, H, G, D, Dv, _stream()),
-        "delta_scan")
+        "delta_scan", 2 if z is not None and T > n_segs else 1)

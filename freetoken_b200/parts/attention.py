@@ -19,7 +19,9 @@ schedule entry names the owner) and a cache that outlives the layer's own window
 look farther back (``cache_window``), biases on the q, k and v projections (``proj_bias``), one learned sink
 logit per head (``sink="learned"``), and a bias by the logarithm of the distance that is taken off the scaled score,
 ``r1_h ln(1 + r2_h (i - j))`` with two learned numbers per head (``log_dist_bias``; the kernels read it from a table
-by distance that covers the engine's longest sequence, made in float64 and rounded once).
+by distance that covers the engine's longest sequence, made in float64 and rounded once), and first tokens
+that the window keeps (``keep_first``: query ``i`` reads key ``j <= i`` if ``i - j < window`` or ``j < keep_first``).  The
+rotation is any of the rotary position encodings (pairs of halves or of neighbours, scaled frequencies).
 """
 
 from __future__ import annotations
@@ -94,7 +96,8 @@ class GQAttention(Mixer):
     ``eps``, ``gemma`` (bool), ``position`` (PartSpec of a position encoding), ``window``
     (None or tokens), ``scale`` (None = head_dim^-0.5); ``v_head_dim`` (head_dim), ``sink`` (None, a
     logit, or "learned": a tensor of one logit per head), ``proj_bias`` (bool), ``log_dist_bias`` (bool), ``out_gate`` (None | "sigmoid" | "silu"), ``own_kv`` (True), ``cache_window`` (how long the
-    cache keeps a token: ``window``, or more, or None for ever, when other layers read it), ``init_std``."""
+    cache keeps a token: ``window``, or more, or None for ever, when other layers read it), ``keep_first`` (0; with a window,
+    not with ``log_dist_bias``), ``init_std``."""
 
     graph_safe = True  # running a step twice writes the same keys and values again
 
@@ -122,6 +125,9 @@ class GQAttention(Mixer):
             raise ConfigError("gqa_attention: a window holds at least the token itself")
         if self.cache_window is not None and (self.window is None or self.cache_window < self.window):
             raise ConfigError("gqa_attention: the cache must keep a token at least as long as the layer's window")
+        self.keep_first = int(spec.get("keep_first", 0) or 0)
+        if self.keep_first < 0 or (self.keep_first and (self.window is None or spec.get("log_dist_bias", False))):
+            raise ConfigError("gqa_attention: kept first tokens go with a window, without a bias by distance")
         self.learned_sink = spec.get("sink") == "learned"
         self.sink: Optional[float] = None if spec.get("sink") is None or self.learned_sink else float(spec["sink"])
         self.proj_bias = bool(spec.get("proj_bias", False))
@@ -134,6 +140,7 @@ class GQAttention(Mixer):
         self.scale = float(spec.get("scale") or self.head_dim ** -0.5)
         self.position = shared_position(spec.get("position") or PartSpec("none"), env)
         self.rotary_dim = int(getattr(self.position, "rotary_dim", 0))
+        self.neighbours = bool(getattr(self.position, "interleaved", False))
         if self.rotary_dim > self.head_dim:
             raise ConfigError("gqa_attention: rotary_dim exceeds head_dim")
         # more query heads per KV head than the kernels' tiles have rows: every KV head is taken as `kv_split` heads of
@@ -153,7 +160,8 @@ class GQAttention(Mixer):
         self.g_row = self.v_row + (self.vv_dim if self.own_kv else 0)
         self.proj_rows = self.g_row + self.gate_dim
         self.plain = not (self.padded or self.sink is not None or self.out_gate or self.kv_split > 1 or not self.own_kv
-                          or self.learned_sink or self.proj_bias or self.log_dist_bias)
+                          or self.learned_sink or self.proj_bias or self.log_dist_bias or self.neighbours
+                          or self.keep_first)
         self._o_weight: Optional[torch.Tensor] = None
 
     # ------------------------------------------------------------------ tensors
@@ -209,13 +217,14 @@ class GQAttention(Mixer):
         if not self.own_kv:
             return None
         return PagedKVNeed((("k", self.n_kv_heads, self.pad_dim),
-                            ("v", self.n_kv_heads, self.pad_dim)), self.cache_window)
+                            ("v", self.n_kv_heads, self.pad_dim)), self.cache_window,
+                           self.keep_first if self.cache_window is not None else 0)
 
     def workspace_bytes(self, n_tokens: int) -> int:
         item = 4 if self.env.dtype == torch.float32 else 2
         # qkv, q, o, out; and the 32-bit partial results of tiles split along the keys (at most
         # attention_plan.DEAL_MOST_PIECES pieces per SM, 256 rows each at most)
-        rows = n_tokens * (self.proj_rows + self.vv_dim + 2 * self.n_heads * self.pad_dim + self.hidden) * item
+        rows = n_tokens * (self.proj_rows + 2 * self.n_heads * self.pad_dim + self.hidden) * item
         return rows + DEAL_MOST_PIECES * 148 * 256 * (self.pad_dim + 2) * 4
 
     # ------------------------------------------------------------------ step
@@ -247,7 +256,7 @@ class GQAttention(Mixer):
             # one or two query tiles a piece: whichever work list the kernel is estimated to get through sooner
             rows = builder.cheaper_attention_rows(self.plan_group, self.window, self.plan_kv_heads, self.pad_dim)
         self._step_plan = builder.attention_plan(self.plan_group, rows, self.window, self.plan_kv_heads, self.pad_dim,
-                                                 few_rows)
+                                                 few_rows, self.keep_first)
 
     def forward(self, h: torch.Tensor, step: StepState, cache: Any, writes_cache: bool) -> torch.Tensor:
         if not self.plain:
@@ -303,11 +312,9 @@ class GQAttention(Mixer):
                                      slab=cache.slabs["v"], slot_map=cache.slot_map, dst_head_dim=Dp,
                                      bias=self.params.get("v_bias")))
         ops.norm_rope_store(proj, D, self.rotary_dim, step.positions, self.position.table(), self.eps, self.gemma,
-                            sections)
-        if self.own_kv and not v_too:  # values of another size: a pass of their own over a copy of their columns
-            v = ws.get("attn.v", (T, self.vv_dim), dt, (cap, self.vv_dim))
-            v.copy_(proj[:, self.v_row: self.g_row])
-            ops.norm_rope_store(v, Dv, 0, step.positions, None, self.eps, self.gemma,
+                            sections, neighbours=self.neighbours)
+        if self.own_kv and not v_too:  # values of another size: a pass of their own over their columns
+            ops.norm_rope_store(proj[:, self.v_row: self.g_row], Dv, 0, step.positions, None, self.eps, self.gemma,
                                 [dict(first_head=0, n_heads=G, norm_weight=None, rotate=False, slab=cache.slabs["v"],
                                       slot_map=cache.slot_map, dst_head_dim=Dp, bias=self.params.get("v_bias"))])
         plan = step.attention_plans[self._step_plan]
@@ -316,7 +323,7 @@ class GQAttention(Mixer):
                             len(step.segments), plan.items_dev, plan.n_items, plan.part_o, plan.part_ml,
                             o, self._step_plan[2], self.scale, self.window, few_rows=self._step_plan[6],
                             kv_split=self.kv_split, sink=self.params["sink"] if self.learned_sink else self.sink,
-                            dist_bias=self.dist_table())
+                            dist_bias=self.dist_table(), keep_first=self.keep_first)
         if self.out_gate:
             ops.gated_heads(o, proj[:, self.g_row:], o, Dv, self.out_gate)
         out = ws.get("attn.out", (T, self.hidden), dt, (cap, self.hidden))

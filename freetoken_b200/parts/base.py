@@ -181,8 +181,8 @@ class RouteSum:
     residual without the sum's trip through memory; for any other consumer :func:`as_rows` takes it.
 
     With ``aux [T, 2]`` the row also has ``aux[t, 0] passed[t]`` (experts that hand the token's input back) and the shared
-    part counts ``aux[t, 1]`` times; negative places have no row.  Only a :class:`GatedSum` keeps those terms to itself;
-    for every other consumer :meth:`plain` takes the whole sum first."""
+    part counts ``aux[t, 1]`` times; negative places have no row.  A :class:`GatedSum` and a norm with ``takes_aux_sum`` keep
+    those terms to themselves; for every other consumer :meth:`plain` takes the whole sum first."""
 
     def __init__(self, y: torch.Tensor, pos: torch.Tensor, top_k: int, shared: Optional[torch.Tensor],
                  n_tokens: int, out: torch.Tensor, aux: Optional[torch.Tensor] = None,
@@ -333,6 +333,24 @@ class GatedSum:
         ops.stream_step(residual, raw_out=raw_out, **self.kernel_args())
 
 
+class ScaledSum:
+    """Two mixers' outputs that are added with constant factors: ``scales[0] x + scales[1] x2`` is still to be added to the
+    stream, in 32 bits.  A norm with ``takes_scaled_sum`` adds it in the pass that norms the stream; for any other consumer
+    :meth:`fold` adds it first."""
+
+    def __init__(self, x: torch.Tensor, x2: torch.Tensor, scales: Tuple[float, float]):
+        self.x, self.x2, self.scales = x, x2, scales
+
+    def kernel_args(self) -> Dict[str, Any]:
+        """Keyword arguments of ``ops.stream_step``."""
+        return dict(x=self.x, x2=self.x2, scales=self.scales)
+
+    def fold(self, residual: torch.Tensor) -> None:
+        from ..kernels import ops
+
+        ops.stream_step(residual, **self.kernel_args())
+
+
 class HyperSum:
     """A sub-layer output that is still to be written into a layer stack's several residual streams
     (hyper-connections): ``x_t <- sum_s mix[s, t] x_s + out[t] y`` for the streams ``streams [S, T, hidden]``
@@ -363,6 +381,11 @@ def as_rows(x: Any, consumer: Any = None, residual: Optional[torch.Tensor] = Non
             raise ConfigError("a GatedSum needs the stream to be added to")
         x.fold(residual)
         return None
+    if isinstance(x, ScaledSum) and not getattr(consumer, "takes_scaled_sum", False):
+        if residual is None:
+            raise ConfigError("a ScaledSum needs the stream to be added to")
+        x.fold(residual)
+        return None
     if isinstance(x, NormedSum) and not getattr(consumer, "takes_normed_sum", False):
         if residual is None:
             raise ConfigError("a NormedSum needs the stream to be added to")
@@ -376,7 +399,7 @@ def as_rows(x: Any, consumer: Any = None, residual: Optional[torch.Tensor] = Non
     if isinstance(x, RouteSum) and not getattr(consumer, "takes_route_sum", False):
         return x.rows()
     if isinstance(x, RouteSum):
-        return x.plain()
+        return x if getattr(consumer, "takes_aux_sum", False) else x.plain()
     return x
 
 
@@ -385,6 +408,8 @@ class Norm(Part):
     takes_stream_sum: bool = False  # add_forward accepts a StreamSum as x
     takes_normed_sum: bool = False  # add_forward accepts a NormedSum as x
     takes_gated_sum: bool = False  # add_forward accepts a GatedSum as x
+    takes_scaled_sum: bool = False  # add_forward accepts a ScaledSum as x
+    takes_aux_sum: bool = False  # ... and a RouteSum with terms beside the routes' and the plain shared part
 
     def forward(self, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
         """``out = norm(x)`` row by row."""

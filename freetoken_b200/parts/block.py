@@ -3,7 +3,8 @@
 ``prenorm_residual`` (python/freetoken/models/minimax_m3/model.py:53-61): every norm call is
 "add the previous sub-layer's output to the residual, then norm the sum":
 ``r += x; h = N_in(r); a = mixer(h); r += a; h = N_post(r); f = ffn(h)`` and ``f`` travels to
-the next layer's first norm.  The residual stream is 32-bit.
+the next layer's first norm.  The residual stream is 32-bit.  A layer whose feed-forward is ``none`` has no second norm and
+hands on ``a``.
 
 ``parallel_residual``: one norm feeds both sub-layers, ``r += x; h = N(r); a = mixer(h); f = ffn(h)``,
 and ``a + f`` travels to the next layer's norm as a :class:`StreamSum`, so that both are added to
@@ -45,7 +46,8 @@ import torch
 from ..config.spec import ParamSpec, PartSpec, StateNeed
 from ..errors import ConfigError
 from ..kernels import ops
-from .base import (BLOCKS, FEED_FORWARDS, NORMS, Block, BuildEnv, FeedForward, GatedSum, HyperSum, Mixer, NormedSum, Part, RouteSum, StepState,
+from .base import (BLOCKS, FEED_FORWARDS, NORMS, Block, BuildEnv, FeedForward, GatedSum, HyperSum, Mixer, NormedSum, Part, RouteSum,
+                   ScaledSum, StepState,
                    StreamSum, as_rows, nvtx_range)
 
 
@@ -59,13 +61,16 @@ class PreNormResidualBlock(Block):
         super().__init__(spec, env, mixer, ffn, mixer_name, ffn_name)
         self.hidden = int(spec["hidden"])
         self.input_norm = NORMS.build(spec["norm"], env)
-        self.post_norm = NORMS.build(spec["norm"], env)
+        self.has_ffn = not isinstance(ffn, NoFeedForward)
+        self.post_norm = NORMS.build(spec["norm"], env) if self.has_ffn else None
         self.input_norm_name = spec.get("input_norm_name", "input_layernorm")
         self.post_norm_name = spec.get("post_norm_name", "post_attention_layernorm")
 
     def children(self) -> Dict[str, Part]:
-        return {self.input_norm_name: self.input_norm, self.mixer_name: self.mixer,
-                self.post_norm_name: self.post_norm, self.ffn_name: self.ffn}
+        out = {self.input_norm_name: self.input_norm, self.mixer_name: self.mixer}
+        if self.has_ffn:
+            out.update({self.post_norm_name: self.post_norm, self.ffn_name: self.ffn})
+        return out
 
     def workspace_bytes(self, n_tokens: int) -> int:
         item = 4 if self.env.dtype == torch.float32 else 2
@@ -79,10 +84,13 @@ class PreNormResidualBlock(Block):
         self.input_norm.add_forward(as_rows(x, self.input_norm, residual), residual, h)
         with nvtx_range(f"mixer {self.mixer.kind}"):
             a = self.mixer.forward(h, step, cache, writes_cache)
+        if not self.has_ffn:
+            return a
         h2 = ws.get("block.h2", (T, self.hidden), dt, (cap, self.hidden))
         h32 = None
         if self.ffn.f32_input_needed(T) and dt != torch.float32:
             h32 = ws.get("block.h2_f32", (T, self.hidden), torch.float32, (cap, self.hidden))
+        a = as_rows(a, self.post_norm, residual)
         self.post_norm.add_forward(a, residual, h2, out_f32=h32)
         lazy = getattr(self.ffn, "forward_lazy", None)
         with nvtx_range(f"feed-forward {self.ffn.kind}"):
@@ -368,7 +376,7 @@ class ConvPostNormResidualBlock(Block):
             ops.postnorm_add_norm(y, None, weight, self.eps, False, residual)
 
     def forward(self, x, residual: torch.Tensor, step: StepState, cache: Any, writes_cache: bool):
-        if isinstance(x, NormedSum):  # (whatever a block of another kind left to be added)
+        if isinstance(x, (NormedSum, ScaledSum)):  # (whatever a block of another kind left to be added)
             x.fold(residual)
         elif x is not None:
             StreamSum.of(x).fold(residual)

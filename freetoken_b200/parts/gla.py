@@ -52,6 +52,21 @@ def chunk_list(seg_lens: Sequence[Tuple[int, int]], chunk: int) -> Tuple[np.ndar
     return np.asarray(chunks, dtype=np.int32).reshape(-1, 4), per_seg, single, multi
 
 
+def prepare_chunks(builder, chunk: int) -> Tuple[str, int, bool, bool]:
+    """Put the step's chunk lists into its metadata (once per chunk size, whatever the number of layers); returns their
+    name there, the number of chunks, and whether any segment has one chunk / several."""
+    name = f"gla.chunks.{chunk}"
+    found = getattr(builder, "_gla_lists", None)
+    if found is None:
+        found = builder._gla_lists = {}
+    if name not in found:
+        chunks, per_seg, single, multi = chunk_list(builder.seg_lens, chunk)
+        builder.add(name, chunks)
+        builder.add(name + ".segments", per_seg)
+        found[name] = (chunks.shape[0], single, multi)
+    return (name,) + found[name]
+
+
 @MIXERS.register("gated_linear_attention")
 class GatedLinearAttention(Mixer):
     """params: ``hidden``, ``n_heads``, ``head_dim`` (keys and queries), ``v_head_dim``, ``tau``, ``decay_rank``
@@ -112,17 +127,7 @@ class GatedLinearAttention(Mixer):
 
     # ------------------------------------------------------------------ step
     def prepare(self, builder) -> None:
-        """Put the step's chunk lists into its metadata (once per chunk size, whatever the number of layers)."""
-        name = f"gla.chunks.{self.chunk}"
-        found = getattr(builder, "_gla_lists", None)
-        if found is None:
-            found = builder._gla_lists = {}
-        if name not in found:
-            chunks, per_seg, single, multi = chunk_list(builder.seg_lens, self.chunk)
-            builder.add(name, chunks)
-            builder.add(name + ".segments", per_seg)
-            found[name] = (chunks.shape[0], single, multi)
-        self._step_lists = (name,) + found[name]
+        self._step_lists = prepare_chunks(builder, self.chunk)
 
     def forward(self, h: torch.Tensor, step: StepState, cache: Any, writes_cache: bool) -> torch.Tensor:
         if not writes_cache:

@@ -31,7 +31,7 @@ from ..config.spec import ParamSpec, PartSpec, StateNeed
 from ..errors import ConfigError
 from ..kernels import ops
 from .base import MIXERS, BuildEnv, Mixer, StepState
-from .gla import DEFAULT_CHUNK, chunk_list
+from .gla import DEFAULT_CHUNK, prepare_chunks
 
 
 @MIXERS.register("mlstm")
@@ -87,16 +87,7 @@ class MatrixMemory(Mixer):
 
     def prepare(self, builder) -> None:
         """Put the step's chunk lists into its metadata (once per chunk size; the recurrence's other users share them)."""
-        name = f"gla.chunks.{self.chunk}"
-        found = getattr(builder, "_gla_lists", None)
-        if found is None:
-            found = builder._gla_lists = {}
-        if name not in found:
-            chunks, per_seg, single, multi = chunk_list(builder.seg_lens, self.chunk)
-            builder.add(name, chunks)
-            builder.add(name + ".segments", per_seg)
-            found[name] = (chunks.shape[0], single, multi)
-        self._step_lists = (name,) + found[name]
+        self._step_lists = prepare_chunks(builder, self.chunk)
 
     def forward(self, h: torch.Tensor, step: StepState, cache: Any, writes_cache: bool) -> torch.Tensor:
         if not writes_cache:

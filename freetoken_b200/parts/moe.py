@@ -23,6 +23,10 @@ weight).  Their routes get no rows; a token's weights on them are one number (``
 :class:`RouteSum` applies to the input row.  ``shared_gate``: the shared expert's output is multiplied by
 ``sigmoid(w_sg . h)``, whose logit is one more row of the router product (``aux[t, 1]``).  The reference has neither.
 
+``scoring="softmax_raw"``: the chosen experts' softmax scores as they are.  ``groups=(count, keep)``: the experts form ``count``
+equal groups of neighbours, and a token's experts come from the ``keep`` groups with the largest choice in them.  The
+reference has neither.
+
 ``router="token_table"`` has no router matrix: a table ``[vocab, top_k]`` of expert ids (the ids of a
 row differ) names each token id's experts, each with weight ``1 / top_k``; the expert products are
 the same kernels.  The reference has no such router.
@@ -68,7 +72,7 @@ def split_in_three(w: torch.Tensor) -> Optional[torch.Tensor]:
 @FEED_FORWARDS.register("moe")
 class MoE(FeedForward):
     """params: ``hidden``, ``inter``, ``n_experts``, ``top_k``, ``scoring`` ("sigmoid" |
-    "softmax"), ``bias`` (bool), ``scale``, ``act``, ``alpha``, ``limit``,
+    "softmax" | ...), ``groups`` (None, or (count, keep)), ``bias`` (bool), ``scale``, ``act``, ``alpha``, ``limit``,
     ``shared_inter`` (0 = no shared expert), ``shared_limit`` (the shared expert's clamp; ``limit`` when absent), ``router`` ("learned" | "token_table"; the table also needs
     ``vocab``), ``weight_on`` ("output" | "input"), ``identity`` (experts behind the ``n_experts`` real ones that hand the
     input back, 0), ``shared_gate`` (bool), ``router_store`` (dtype of router and bias in written files), ``bias_std``.  ``h_f32`` given to the forward calls of a bfloat16 model
@@ -89,6 +93,11 @@ class MoE(FeedForward):
         self.scoring = spec.get("scoring", "sigmoid")
         if self.scoring not in ops.SCORE_CODES:
             raise ConfigError(f"moe: unknown scoring '{self.scoring}'")
+        self.groups = tuple(int(x) for x in (spec.get("groups") or (1, 1)))
+        count, keep = self.groups
+        if not 1 <= keep <= count or self.n_choices % count or self.top_k > self.n_choices // count * keep \
+                or (self.n_choices > 512 and count > 64):
+            raise ConfigError(f"moe: the best {keep} of {count} groups of {self.n_choices} experts, {self.top_k} a token")
         self.has_bias = bool(spec.get("bias", False))
         self.scale = float(spec.get("scale", 1.0))
         self.act = spec.get("act", "swigluoai")
@@ -199,8 +208,11 @@ class MoE(FeedForward):
         return RouteSum(y, pos, k, shared, T, out, aux, h if self.identity else None)
 
     def _aux_args(self, aux: Optional[torch.Tensor]) -> dict:
-        """What the routing kernels are told about identity experts and the shared expert's gate."""
-        return {} if aux is None else dict(n_extra=int(self.shared_gate), n_real=self.n_experts, aux=aux)
+        """What the routing kernels are told about groups, identity experts and the shared expert's gate."""
+        args = {} if self.groups[0] == 1 else dict(groups=self.groups)
+        if aux is not None:
+            args.update(n_extra=int(self.shared_gate), n_real=self.n_experts, aux=aux)
+        return args
 
     def forward_lazy(self, h: torch.Tensor, step: StepState, h_f32: Optional[torch.Tensor] = None) -> RouteSum:
         """The experts' rows and where each token's routes lie among them; the sum over a token's routes

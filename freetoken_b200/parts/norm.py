@@ -18,7 +18,7 @@ import torch
 from ..config.spec import ParamSpec, PartSpec
 from ..kernels import ops
 from ..errors import ConfigError
-from .base import NORMS, BuildEnv, GatedSum, Norm, NormedSum, RouteSum, StreamSum
+from .base import NORMS, BuildEnv, GatedSum, Norm, NormedSum, RouteSum, ScaledSum, StreamSum
 
 
 @NORMS.register("rmsnorm")
@@ -30,6 +30,8 @@ class RMSNorm(Norm):
     takes_route_sum = True
     takes_normed_sum = True
     takes_gated_sum = True
+    takes_scaled_sum = True
+    takes_aux_sum = True
 
     def __init__(self, spec: PartSpec, env: BuildEnv):
         super().__init__(spec, env)
@@ -76,11 +78,18 @@ class RMSNorm(Norm):
         if isinstance(x, GatedSum) and x.groups != self.groups:
             x.fold(residual)
             x = None
+        if self.groups == 1 and (isinstance(x, ScaledSum) or (isinstance(x, RouteSum) and x.aux is not None)):
+            # two scaled results, or an expert layer's sum with all its terms: added in 32 bits by the pass that norms
+            args = x.kernel_args() if isinstance(x, ScaledSum) else \
+                dict(x=x.y, routed=(x.pos, x.top_k, x.shared, x.aux, x.passed))
+            ops.stream_step(residual, pre_weight=self._w, pre_eps=self.eps, out=out, norm_f32=out_f32, f32_rounded=True,
+                            rows=rows, **args)
+            return out
         if isinstance(x, GatedSum) or self.groups > 1:  # gate, the sub-layer's own norm, the sum and this norm in one pass
             if out_f32 is not None:
                 raise ConfigError("rmsnorm: no 32-bit copy of the output of a norm over groups")
             if x is not None and not isinstance(x, GatedSum):
-                (x if isinstance(x, NormedSum) else StreamSum.of(x)).fold(residual)
+                (x if isinstance(x, (NormedSum, ScaledSum)) else StreamSum.of(x)).fold(residual)
                 x = None
             args = x.kernel_args() if x is not None else dict(groups=self.groups)
             ops.stream_step(residual, pre_weight=self._w, pre_eps=self.eps, out=out, rows=rows, **args)

@@ -18,6 +18,10 @@ the original context, ``lo = max(floor(index(fast)), 0)`` and ``hi = min(ceil(in
 turns at ``f_i / factor`` with the share ``ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1)`` and at ``f_i`` with the
 rest; cosines and sines are multiplied by ``0.1 ln(factor) + 1``.
 
+``band_scaling`` (a parameter of both, as Llama 3.1 stretches its frequencies): ``(factor, low, high, original)``.  A pair whose
+wavelength ``2 pi / f`` is shorter than ``original / high`` keeps ``f``, one longer than ``original / low`` turns at
+``f / factor``, and in between the two are blended with ``s = (original f / (2 pi) - low) / (high - low)`` on ``f``.
+
 ``none``: no position encoding (a mixer that needs none asks for this kind).
 
 ``log_temperature``: no rotation; the table holds one factor per position,
@@ -42,7 +46,8 @@ from .base import POSITIONS, BuildEnv, PositionEncoding
 class NeoxRope(PositionEncoding):
     """params: ``rotary_dim`` (even, <= head_dim; 0 disables), ``theta``, ``precise`` (False: the reference's
     float32 operations; True: angles, cosines and sines in float64, rounded to float32 once), ``yarn`` (None, or
-    ``(factor, original, fast, slow)``; needs ``precise``)."""
+    ``(factor, original, fast, slow)``; needs ``precise``), ``band_scaling`` (None, or ``(factor, low, high, original)``; needs
+    ``precise``; not with ``yarn``)."""
 
     interleaved = False
 
@@ -55,12 +60,21 @@ class NeoxRope(PositionEncoding):
         self.yarn = spec.get("yarn")
         if self.yarn is not None and not spec.get("precise", False):
             raise ConfigError("rope: stretched frequencies are computed in float64 (precise)")
+        self.bands = spec.get("band_scaling")
+        if self.bands is not None and (self.yarn is not None or not spec.get("precise", False)):
+            raise ConfigError("rope: frequencies are scaled in one way, in float64 (precise)")
         self._table: Optional[torch.Tensor] = None
 
     def frequencies(self) -> torch.Tensor:
         """One per pair, float64."""
         rd = self.rotary_dim
         f = self.theta ** (-torch.arange(0, rd, 2, dtype=torch.float64) / rd)
+        if self.bands is not None:
+            factor, low, high, original = (float(x) for x in self.bands)
+            wave = 2.0 * math.pi / f
+            s = (original / wave - low) / (high - low) if high != low else torch.zeros_like(f)
+            mixed = (1.0 - s) * f / factor + s * f
+            return torch.where(wave < original / high, f, torch.where(wave > original / low, f / factor, mixed))
         if self.yarn is None:
             return f
         factor, original, fast, slow = (float(x) for x in self.yarn)

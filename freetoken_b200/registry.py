@@ -41,6 +41,7 @@ _LAZY: Dict[str, str] = {
     "Kekopel": "freetoken_b200.models.kekopel",
     "Nusudra": "freetoken_b200.models.nusudra",
     "Vodatar": "freetoken_b200.models.vodatar",
+    "Gizulorn": "freetoken_b200.models.gizulorn",
 }
 
 

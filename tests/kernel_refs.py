@@ -75,7 +75,7 @@ def table_update(table, updates, n_updates):
     table.view(-1)[u[ok, 0].long()] = u[ok, 1]
 
 
-def norm_rope_store(x, head_dim, rotary_dim, positions, rope_table, eps, gemma, sections):
+def norm_rope_store(x, head_dim, rotary_dim, positions, rope_table, eps, gemma, sections, neighbours=False):
     T = x.shape[0]
     whole = x.shape[1] // head_dim * head_dim  # a row may end in columns that belong to no head
     xs = x[:, :whole].reshape(T, -1, head_dim).float()
@@ -91,7 +91,10 @@ def norm_rope_store(x, head_dim, rotary_dim, positions, rope_table, eps, gemma, 
         if w is not None:
             scale = w.float() + 1.0 if gemma else w.float()
             u = u * torch.rsqrt((u * u).sum(-1, keepdim=True) / head_dim + eps) * scale
-        if s.get("rotate") and rotary_dim:
+        if s.get("rotate") and rotary_dim and neighbours:
+            a, b = u[..., 0:rotary_dim:2], u[..., 1:rotary_dim:2]
+            u = torch.cat([torch.stack([a * cos - b * sin, b * cos + a * sin], dim=-1).flatten(-2), u[..., rotary_dim:]], dim=-1)
+        elif s.get("rotate") and rotary_dim:
             a, b, rest = u[..., :half], u[..., half:rotary_dim], u[..., rotary_dim:]
             u = torch.cat([a * cos - b * sin, b * cos + a * sin, rest], dim=-1)
         if s.get("pos_scale") is not None:
@@ -112,10 +115,11 @@ def norm_rope_store(x, head_dim, rotary_dim, positions, rope_table, eps, gemma, 
 
 def paged_attention(q, k_slab, v_slab, block_table, seg_info, n_segs, items, n_items, part_o, part_ml,
                     out, tile_rows, scale, window, sel=None, block_size=0, few_rows=False, dist_bias=None, kv_split=1,
-                    sink=None, softcap=None):
+                    sink=None, softcap=None, keep_first=0):
     """Per query token, softmax over the visible keys gathered through the block table; the
     work list and the scratch are ignored (they only steer how the kernel splits the work).
-    With ``sel`` a query reads only the keys of its chosen blocks."""
+    With ``sel`` a query reads only the keys of its chosen blocks.  Pages that a window has passed may hold anything (they are
+    not read), but for the ones of the first ``keep_first`` positions."""
     T, Hq, D = q.shape
     P = k_slab.shape[2]
     Hkv = k_slab.shape[1]
@@ -132,6 +136,9 @@ def paged_attention(q, k_slab, v_slab, block_table, seg_info, n_segs, items, n_i
             qq = q[q_start + t].float().view(-1, G, D)  # [Hkv, G, D]
             if sel is None:
                 kk, vv = K[lo:p_q + 1], V[lo:p_q + 1]
+                if keep_first and lo > 0:
+                    n = min(keep_first, lo)
+                    kk, vv = torch.cat([K[:n], kk]), torch.cat([V[:n], vv])
                 s = torch.einsum("hgd,khd->hgk", qq, kk) * scale
                 if softcap:
                     s = softcap * torch.tanh(s / softcap)
@@ -189,7 +196,8 @@ def sparse_select(iq, ik_slab, block_table, seg_info, n_segs, block_size, local_
             sel[q_start + t, :, : chosen.shape[1]] = chosen.to(torch.int32)
 
 
-def router_topk(logits, bias, top_k, scoring, scale, ids, weights, n_parts=1, n_extra=0, n_real=None, aux=None, n_pad=0):
+def router_topk(logits, bias, top_k, scoring, scale, ids, weights, n_parts=1, n_extra=0, n_real=None, aux=None, n_pad=0,
+                groups=(1, 1)):
     l = logits.float()
     if n_parts > 1:
         parts = l.view(l.shape[0], n_parts, -1)
@@ -202,32 +210,43 @@ def router_topk(logits, bias, top_k, scoring, scale, ids, weights, n_parts=1, n_
     if n_extra:
         l, extra = l[:, :-n_extra], l[:, -1]
     if aux is not None:
-        _choose(l, bias, top_k, scoring, scale, ids, weights)
+        _choose(l, bias, top_k, scoring, scale, ids, weights, groups)
         real = l.shape[1] if n_real is None else n_real
         aux[:, 0] = torch.where(ids >= real, weights, torch.zeros_like(weights)).sum(-1)
         aux[:, 1] = torch.sigmoid(extra) if extra is not None else 1.0
         return
-    _choose(l, bias, top_k, scoring, scale, ids, weights)
+    _choose(l, bias, top_k, scoring, scale, ids, weights, groups)
 
 
-def _choose(l, bias, top_k, scoring, scale, ids, weights):
+def _open_groups(c, groups):
+    """The choices of experts outside the best groups (by their largest choice) become -inf."""
+    count, keep = groups
+    if keep >= count:
+        return c
+    best = c.view(c.shape[0], count, -1).amax(-1)
+    order = torch.argsort(best, dim=-1, descending=True, stable=True)[:, :keep]
+    ok = torch.zeros_like(best, dtype=torch.bool).scatter(-1, order, True)
+    return c.masked_fill(~ok.repeat_interleave(c.shape[1] // count, dim=-1), float("-inf"))
+
+
+def _choose(l, bias, top_k, scoring, scale, ids, weights, groups=(1, 1)):
     if scoring == "softmax_of_chosen":  # the bias belongs to the logit; the softmax runs over the chosen logits only
         l = l + bias.float() if bias is not None else l
-        idx = torch.argsort(l, dim=-1, descending=True, stable=True)[:, :top_k]
+        idx = torch.argsort(_open_groups(l, groups), dim=-1, descending=True, stable=True)[:, :top_k]
         ids.copy_(idx.to(torch.int32))
         weights.copy_(torch.softmax(l.gather(-1, idx), dim=-1) * scale)
         return
     if scoring == "sigmoid_raw":  # the chosen experts' sigmoid scores as they are
         sg = torch.sigmoid(l)
-        idx = torch.argsort(sg, dim=-1, descending=True, stable=True)[:, :top_k]
+        idx = torch.argsort(_open_groups(sg, groups), dim=-1, descending=True, stable=True)[:, :top_k]
         ids.copy_(idx.to(torch.int32))
         weights.copy_(sg.gather(-1, idx) * scale)
         return
     s = torch.sigmoid(l) if scoring == "sigmoid" else torch.softmax(l, dim=-1)
     c = s + bias.float() if bias is not None else s
-    idx = torch.argsort(c, dim=-1, descending=True, stable=True)[:, :top_k]
+    idx = torch.argsort(_open_groups(c, groups), dim=-1, descending=True, stable=True)[:, :top_k]
     w = s.gather(-1, idx)
-    w = w / (w.sum(-1, keepdim=True) + 1e-20)
+    w = w if scoring == "softmax_raw" else w / (w.sum(-1, keepdim=True) + 1e-20)
     ids.copy_(idx.to(torch.int32))
     weights.copy_(w * scale)
 
@@ -266,9 +285,9 @@ def moe_route_fits(n_tokens, hidden, n_experts, top_k):
 
 
 def moe_route(x, gate_w, bias, top_k, scoring, scale, logits, ids, weights, expert_counts, expert_offsets,
-              sorted_routes, route_pos, n_extra=0, n_real=None, aux=None):
+              sorted_routes, route_pos, n_extra=0, n_real=None, aux=None, groups=(1, 1)):
     logits.copy_(x.float() @ gate_w.float().T)
-    router_topk(logits, bias, top_k, scoring, scale, ids, weights, n_extra=n_extra, n_real=n_real, aux=aux)
+    router_topk(logits, bias, top_k, scoring, scale, ids, weights, n_extra=n_extra, n_real=n_real, aux=aux, groups=groups)
     moe_permute(ids, gate_w.shape[0] - n_extra if n_real is None else n_real, expert_counts, expert_offsets, sorted_routes,
                 route_pos)
 
@@ -442,18 +461,25 @@ def gated_heads(x, gates, out, dim, act="sigmoid", norm_weight=None, eps=0.0):
 
 def gla_scan(q, k, v, z, z_bias, tau, q_scale, state, state_slots, seg_info, n_segs, chunks, n_chunks, seg_chunks,
              any_single, any_multi, carry, decay_prod, out, k_fac=None, a_head=None, ones_col=False, out_ones=None,
-             qk_div=1):
+             qk_div=1, rope_table=None, neighbours=False):
     """Token by token from each request's slot; the chunk lists only steer how the kernel shares the work."""
     H, D, Dv = state.shape[1:]
     if qk_div > 1:  # queries and keys shared by groups of heads
         q = q.float().view(-1, H // qk_div, D).repeat_interleave(qk_div, dim=1).reshape(-1, H * D)
         k = k.float().view(-1, H // qk_div, D).repeat_interleave(qk_div, dim=1).reshape(-1, H * D)
     if a_head is not None:
-        decay = a_head.float()[:, :, None].expand(-1, H, D)
+        decay = a_head.float().view(-1, H, 1).expand(q.shape[0], H, D)
     else:
         zz = z.float() + (z_bias.float().view(1, -1) if z_bias is not None else 0.0)
         decay = torch.exp(-torch.nn.functional.softplus(-zz) / tau).view(-1, H, D)
     qq, kk = q.float().view(-1, H, D) * q_scale, k.float().view(-1, H, D)
+    if rope_table is not None:
+        qq, kk = qq.clone(), kk.clone()
+        for q_start, q_len, kv_len, _ in seg_info.view(-1, 4)[:n_segs].tolist():
+            for t in range(q_len):
+                p = kv_len - q_len + t
+                for x in (qq, kk):
+                    x[q_start + t] = _turn(x[q_start + t], p, rope_table, rope_table.shape[1], neighbours)
     if k_fac is not None:
         kk = kk * k_fac.float()[:, :, None]
     vv = v.float().view(-1, H, Dv - (1 if ones_col else 0))
@@ -630,7 +656,8 @@ def _group_norm(z, groups, eps):
 
 
 def stream_step(residual, groups=1, vec=None, x=None, routed=None, gate=None, gate_bias=None, post_weight=None, post_eps=0.0,
-                raw_out=None, pre_weight=None, pre_eps=0.0, out=None, norm_f32=None, conv=None, rows=None, dtype=None):
+                raw_out=None, pre_weight=None, pre_eps=0.0, out=None, norm_f32=None, conv=None, rows=None, dtype=None, x2=None,
+                scales=(1.0, 1.0), f32_rounded=False):
     z = residual.float().clone()
     T = z.shape[0]
     if vec is not None:
@@ -640,11 +667,11 @@ def stream_step(residual, groups=1, vec=None, x=None, routed=None, gate=None, ga
             pos, top_k, shared, aux, passed = routed
             y = _sum_of_routes(x, pos, T, top_k, shared, aux, passed)
         else:
-            y = x.float()[:T]
+            y = x.float()[:T] if x2 is None else scales[0] * x.float()[:T] + scales[1] * x2.float()[:T]
         if gate is not None:
             g = gate.float()[:T]
             y = y * torch.sigmoid(g if gate_bias is None else g + gate_bias.float())
-        z = z + _group_norm(y, groups, post_eps) * post_weight.float()
+        z = z + (y if post_weight is None else _group_norm(y, groups, post_eps) * post_weight.float())
     if rows is None:
         residual.copy_(z)
     else:
@@ -655,7 +682,7 @@ def stream_step(residual, groups=1, vec=None, x=None, routed=None, gate=None, ga
         return
     h = _group_norm(z, groups, pre_eps) * pre_weight.float()
     if norm_f32 is not None:
-        norm_f32.copy_(h)
+        norm_f32.copy_((h.to(out.dtype).float() if f32_rounded else h).view(norm_f32.shape))
     if out is not None:
         out.view(h.shape).copy_(h.to(out.dtype))
     if conv is not None:
@@ -722,7 +749,7 @@ def ssm_output(o32, x, d_skip, z, norm_weight, norm_groups, eps, out):
     out.copy_(y.to(out.dtype))
 
 
-def delta_scan(q, k, v, b_raw, a_raw, a_log, dt_bias, q_scale, unit_eps, state, state_slots, seg_info, n_segs, out):
+def delta_scan(q, k, v, b_raw, a_raw, a_log, dt_bias, q_scale, unit_eps, state, state_slots, seg_info, n_segs, out, z=None):
     T, H, Dv = out.shape
     D = state.shape[3]  # the state is kept column by column: [slots, H, Dv, D]
     G = q.shape[1] // D
@@ -732,12 +759,13 @@ def delta_scan(q, k, v, b_raw, a_raw, a_log, dt_bias, q_scale, unit_eps, state, 
     qq, kk = qq.repeat_interleave(H // G, dim=1), kk.repeat_interleave(H // G, dim=1)
     vv = v.float().view(T, H, Dv)
     beta = torch.sigmoid(b_raw.float())
-    g = torch.exp(-torch.exp(a_log.float()) * torch.nn.functional.softplus(a_raw.float() + dt_bias.float(), threshold=1e9))
+    pre = (a_raw if z is None else z).float() + dt_bias.float()  # [T, H], or [T, H * D] with a decay per key channel
+    g = torch.exp(-torch.exp(a_log.float())[:, None] * torch.nn.functional.softplus(pre, threshold=1e9).view(T, H, -1))
     for i, (q_start, q_len, kv_len, _) in enumerate(seg_info.view(-1, 4)[:n_segs].tolist()):
         slot = int(state_slots[i])
         S = torch.zeros(H, D, Dv) if kv_len == q_len else state[slot].transpose(1, 2).clone()
         for t in range(q_start, q_start + q_len):
-            S = g[t][:, None, None] * S
+            S = g[t][:, :, None] * S
             u = beta[t][:, None] * (vv[t] - torch.einsum("hdv,hd->hv", S, kk[t]))
             S = S + kk[t][:, :, None] * u[:, None, :]
             out[t] = torch.einsum("hdv,hd->hv", S, qq[t])
