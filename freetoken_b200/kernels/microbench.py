@@ -18,6 +18,8 @@
     python -m freetoken_b200.kernels.microbench attention --prefill 2048 --dist-bias 2048 --head-sinks
     python -m freetoken_b200.kernels.microbench vodatar --tokens 2048 [--batch 8]
     python -m freetoken_b200.kernels.microbench attention --prefill 2048 --q-heads 96 --softcap 30 --maps 2
+    python -m freetoken_b200.kernels.microbench gizulorn --tokens 2048 [--batch 8]
+    python -m freetoken_b200.kernels.microbench attention --prefill 2048 --window 1024 --head-sinks --keep-first 4
 
 Each case allocates its inputs once (larger than L2 where the real workload is), warms up, then
 times ``--iters`` launches with CUDA events and prints one JSON line: time, the bytes the kernel has
@@ -151,6 +153,7 @@ def bench_attention(a) -> dict:
         sink = torch.randn(Hq, device=dev, generator=g)
     special = window is not None or sink is not None  # of the tcgen05 kernels the one with 128-row tiles takes these
     cap = float(getattr(a, "softcap", 0) or 0) or None  # scores become cap * tanh(score / cap)
+    keep = int(getattr(a, "keep_first", 0) or 0)  # first tokens that the window keeps
     maps = max(1, int(getattr(a, "maps", 1) or 1))  # query rows are zero outside a map's place: a part of Q K^T does no work
     if maps > 1:
         q.view(q0, Hq // maps, maps, maps, D // maps).mul_(torch.eye(maps, device=dev, dtype=q.dtype)[None, None, :, :, None])
@@ -161,15 +164,17 @@ def bench_attention(a) -> dict:
     few_rows = False
     if not a.prefill:
         few_rows = a.few_rows and not no_tc and not special and ops.attention_tc_few_fits(D, P, G)
-        tc = few_rows or (a.tc and not no_tc and not special and ops.attention_tc_fits(D, P, G))
-        fixed = wave_splits(len(segs) * Hkv, 148 if tc else 2 * 148, 16, a.context) if a.splits is None else a.splits
+        tc = few_rows or (a.tc and not no_tc and ops.attention_tc_fits(D, P, G))
+        span = a.context if window is None else min(a.context, window + keep)
+        fixed = wave_splits(len(segs) * Hkv, 148 if tc else 2 * 148, 16 if window is None else max(1, min(16, span // 256)),
+                            span) if a.splits is None else a.splits
         tile = 16 if few_rows else 128 if tc else (16 if G <= 16 else 64)
     tensor_core = few_rows or tile >= 128  # (one CTA per SM: the engine plans these for half as many CTA slots)
     costs = None
     if tile >= 128 and fixed is None:  # as the engine plans these kernels' work lists
         costs = TC_TWO_TILE_COSTS if tile == 256 else TC_ONE_TILE_COSTS
     plan = build_plan(segs, G, tile, window, Hkv, sm_count=74 if tensor_core else 148, fixed_splits=fixed,
-                      key_tile=128 if tensor_core else 0, costs=costs)
+                      key_tile=128 if tensor_core else 0, costs=costs, keep_first=keep)
     items = torch.from_numpy(plan.items).to(dev)
     po = pm = None
     if plan.n_slots:
@@ -177,11 +182,11 @@ def bench_attention(a) -> dict:
         pm = torch.empty(plan.n_slots, Hkv, tile, 2, dtype=torch.float32, device=dev)
     out = torch.empty_like(q)
     us = _time(lambda: ops.paged_attention(q, ks, vs, bt, seg, len(segs), items, plan.n_items, po, pm, out, tile,
-                                           D ** -0.5, window, few_rows=few_rows, dist_bias=bias, sink=sink, softcap=cap), a.iters,
-               a.warmup, a.profile)
-    seen = [(ql, kv if window is None else min(kv, window - 1 + ql)) for ql, kv in segs]  # keys a segment's queries can see
+                                           D ** -0.5, window, few_rows=few_rows, dist_bias=bias, sink=sink, softcap=cap,
+                                           keep_first=keep), a.iters, a.warmup, a.profile)
+    seen = [(ql, kv if window is None else min(kv, window - 1 + ql + keep)) for ql, kv in segs]  # keys a segment's queries can see
     kv_bytes = sum(kv for _, kv in seen) * Hkv * D * 2 * (1 if tied else 2)
-    pairs = lambda ql, kv: sum(min(kv - ql + t + 1, window or (1 << 60)) for t in range(ql))  # noqa: E731  (query, key) pairs
+    pairs = lambda ql, kv: sum(min(kv - ql + t + 1, (window or (1 << 60)) + keep) for t in range(ql))  # noqa: E731  (query, key) pairs
     flops = sum((2 + 2 / maps) * pairs(ql, kv) * Hq * D for ql, kv in segs)
     return {"us": round(us, 2), "tile_rows": tile, "tied": tied, "dist_bias": n_bias, "window": window, "sink": sink is not None, "softcap": cap,
             "items": plan.n_items,
@@ -596,6 +601,135 @@ def bench_vodatar(a) -> dict:
     return results
 
 
+def bench_gizulorn(a) -> dict:
+    """The kernels that the Gizulorn layers add around the library products, each beside the like kernel of another design: two
+    mixers' results or an expert layer's sum into the stream with the norm behind it, the rotation of neighbours on the way
+    to the cache, the delta rule with a decay per key channel, retention (fixed decays, rotation inside the recurrence),
+    routing within groups.  Attention is ``attention --window W --head-sinks --keep-first K``."""
+    from ..parts.gla import chunk_list
+
+    dev = "cuda"
+    T, C, H, G, D, Dv, k, taps = a.tokens, a.hidden, a.heads, a.kv_heads, a.dim, a.vdim, a.top_k, a.taps
+    decode = a.batch > 0
+    segs = [(1, a.context)] * a.batch if decode else [(T, T)]
+    T = sum(q for q, _ in segs)
+    g = torch.Generator(device=dev).manual_seed(0)
+    bf = torch.bfloat16
+    info, q0 = [], 0
+    for ql, kv in segs:
+        info.append([q0, ql, kv, 0])
+        q0 += ql
+    seg = torch.tensor(info, dtype=torch.int32, device=dev)
+    S = len(segs)
+    slots = torch.arange(1, S + 1, dtype=torch.int32, device=dev)
+    results = {}
+    fp32_tflops = 148 * 128 * 2 * 1.965e9 / 1e12
+
+    def add(name, fn, nbytes, flops=0):
+        if a.only and a.only not in name:
+            return
+        us = _time(fn, a.iters, a.warmup, a.profile)
+        results[name] = {"us": round(us, 2), "bytes": nbytes, "gbs": round(nbytes / us / 1e3, 1),
+                         "hbm_frac": round(nbytes / us / 1e3 / HBM_GBS, 3)}
+        if flops:
+            results[name].update(tflops=round(flops / us / 1e6, 2), fp32_frac_nominal=round(flops / us / 1e6 / fp32_tflops, 3))
+
+    rnd = lambda *s: torch.randn(*s, device=dev, generator=g).to(bf)  # noqa: E731
+    res = torch.randn(T, C, device=dev, generator=g)
+    y, y2, shared, h = rnd(T, C), rnd(T, C), rnd(T, C), rnd(T, C)
+    w = torch.ones(C, device=dev)
+    add("stream_step (two scaled results, norm)",
+        lambda: ops.stream_step(res, x=y, x2=y2, scales=(0.8, 1.1), pre_weight=w, pre_eps=1e-6, out=h), T * C * (4 + 4 + 2 + 2 + 2))
+    rows, pos = rnd(T * k, C), torch.randperm(T * k, device=dev, generator=g).to(torch.int32)
+    aux = torch.rand(T, 2, device=dev, generator=g)
+    add("stream_step (expert routes, gated shared row, norm)",
+        lambda: ops.stream_step(res, x=rows, routed=(pos, k, shared, aux, None), pre_weight=w, pre_eps=1e-6, out=h),
+        T * C * (4 + 4 + 2 + 2) + T * k * C * 2)
+    add("like: add_rmsnorm", lambda: ops.add_rmsnorm(y, res, w, 1e-6, False, h), T * C * (4 + 4 + 2 + 2))
+    add("like: add_rmsnorm_routes (shared row)", lambda: ops.add_rmsnorm_routes(rows, pos, k, shared, res, w, 1e-6, False, h),
+        T * C * (4 + 4 + 2 + 2) + T * k * C * 2)
+    # heads to the cache
+    proj = rnd(T, (H + 2 * G) * D)
+    page = 16
+    n_pages = sum(-(-kv // page) for _, kv in segs) + 1
+    ks, vs = (torch.zeros(n_pages, G, page, D, dtype=bf, device=dev) for _ in range(2))
+    positions = torch.cat([torch.arange(kv - ql, kv) for ql, kv in segs]).to(torch.int32).to(dev)
+    smap = (torch.arange(T, device=dev) % (n_pages * page - page) + page).to(torch.int32)
+    table = torch.randn(int(max(kv for _, kv in segs)), D, device=dev, generator=g)
+    qo = torch.empty(T, H, D, dtype=bf, device=dev)
+    for name, nb in (("norm_rope_store (neighbours)", True), ("like: norm_rope_store (halves)", False)):
+        add(name, lambda: ops.norm_rope_store(proj, D, D, positions, table, 1e-6, False, [
+            dict(first_head=0, n_heads=H, norm_weight=None, rotate=True, dense_out=qo),
+            dict(first_head=H, n_heads=G, norm_weight=None, rotate=True, slab=ks, slot_map=smap),
+            dict(first_head=H + G, n_heads=G, norm_weight=None, rotate=False, slab=vs, slot_map=smap)], neighbours=nb),
+            T * (H + 2 * G) * D * 4)
+    # the delta rule
+    conv_dim = 2 * G * D + H * Dv
+    dproj = (torch.randn(T, conv_dim + 2 * H + H * Dv, device=dev, generator=g) * 0.5).to(bf)
+    cw = torch.randn(conv_dim, taps, device=dev, generator=g) * 0.3
+    cst = torch.zeros(S + 1, taps - 1, conv_dim, device=dev)
+    qkv = torch.empty(T, conv_dim, dtype=bf, device=dev)
+    add("conv_act (silu: q, k, v of the delta rule)",
+        lambda: ops.conv_act(dproj[:, :conv_dim], cw, None, "silu", cst, slots, seg, S, qkv),
+        T * conv_dim * 4 + (2 * S * (taps - 1) * conv_dim * 4 if decode else 0))
+    qkv = rnd(T, conv_dim)
+    z, z0 = torch.empty(T, H * D, device=dev), torch.randn(T, H * D, device=dev, generator=g)
+    st = torch.zeros(S + 1, H, Dv, D, device=dev)
+    o32 = torch.empty(T, H, Dv, device=dev)
+    al, db, dbc = torch.zeros(H, device=dev), torch.zeros(H, device=dev), torch.zeros(H * D, device=dev)
+    b_raw, a_raw = dproj[:, conv_dim:conv_dim + H], dproj[:, conv_dim + H:conv_dim + 2 * H]
+    args = (qkv[:, :G * D], qkv[:, G * D:2 * G * D], qkv[:, 2 * G * D:], b_raw)
+    z.copy_(z0)
+    nbytes = T * H * ((2 * D + Dv) * 2 + Dv * 4) + 2 * S * H * D * Dv * 4
+    # (logits to decays in place: with every launch they lie nearer to 1, at the same cost)
+    add("delta_scan (a decay per key channel)",
+        lambda: ops.delta_scan(*args, None, al, dbc, D ** -0.5, 1e-6, st, slots, seg, S, o32, z=z),
+        nbytes + T * H * D * 4 * (1 if decode else 3), T * H * D * Dv * 7)
+    add("like: delta_scan (a decay per head)",
+        lambda: ops.delta_scan(*args, a_raw, al, db, D ** -0.5, 1e-6, st, slots, seg, S, o32), nbytes, T * H * D * Dv * 7)
+    o, hw = torch.empty(T, H, Dv, dtype=bf, device=dev), torch.ones(Dv, device=dev)
+    gates = dproj[:, conv_dim + 2 * H:]
+    add("gated_heads (head norm, sigmoid gate)", lambda: ops.gated_heads(o32, gates, o, Dv, "sigmoid", hw, 1e-6), T * H * Dv * 8)
+    # retention
+    chunks, per_seg, single, multi = chunk_list(segs, a.chunk)
+    n = chunks.shape[0]
+    rproj = (torch.randn(T, 2 * H * D + H * Dv, device=dev, generator=g) * 0.5).to(bf)
+    rst = torch.zeros(S + 1, H, D, Dv, device=dev)
+    carry = torch.empty(n, H, D, Dv, device=dev) if multi else None
+    prod = torch.empty(n, H, D, device=dev) if multi else None
+    cd, pd = torch.from_numpy(chunks).to(dev), torch.from_numpy(per_seg).to(dev)
+    dec = torch.full((H,), 0.99, device=dev)
+    decs = torch.full((T, H), 0.99, device=dev)
+    passes = 2 if multi else 1
+    rargs = (rproj[:, :H * D], rproj[:, H * D:2 * H * D], rproj[:, 2 * H * D:])
+    rest = (1.0, D ** -0.5, rst, slots, seg, S, cd, n, pd, single, multi, carry, prod, o32)
+    rbytes = T * H * (2 * D + Dv) * 2 * passes + T * H * Dv * 4 + (2 * S + (4 * n if multi else 0)) * H * D * Dv * 4
+    rflops = T * H * D * Dv * (8 if multi else 5)
+    add("gla_scan (retention: rotation inside)", lambda: ops.gla_scan(*rargs, None, None, *rest, a_head=dec, rope_table=table),
+        rbytes + T * D * 4, rflops)
+    add("like: gla_scan (a decay per head and token, no rotation)",
+        lambda: ops.gla_scan(*rargs, None, None, *rest, a_head=decs), rbytes + T * H * 4, rflops)
+    add("like: gla_scan (a decay per key channel, no rotation)", lambda: ops.gla_scan(*rargs, z, None, *rest),
+        rbytes + T * H * D * 4 * (passes + (2 if multi else 0)), rflops)
+    # routing
+    E = a.experts
+    ids, wts = torch.empty(T, k, dtype=torch.int32, device=dev), torch.empty(T, k, device=dev)
+    auxo, logits = torch.empty(T, 2, device=dev), torch.randn(T, E + 1, device=dev, generator=g)
+    gw = torch.randn(E + 1, C, device=dev, generator=g) * C ** -0.5
+    x32 = torch.randn(T, C, device=dev, generator=g)
+    for name, groups in (("(groups, shared gate)", (a.groups, a.keep)), ("like: {} (one group)", (1, 1))):
+        op = "moe_route" if ops.moe_route_fits(T, C, E, k) else "router_topk"
+        label = name.format(op) if "{}" in name else f"{op} {name}"
+        if op == "moe_route":
+            add(label, lambda: ops.moe_route(x32, gw, None, k, "softmax_raw", 1.0, logits, ids, wts, n_extra=1, aux=auxo, groups=groups),
+                (E + 1 + T) * C * 4)
+        else:
+            add(label, lambda: ops.router_topk(logits, None, k, "softmax_raw", 1.0, ids, wts, n_extra=1, aux=auxo, groups=groups),
+                T * (E + 1) * 4)
+    results["status"] = ops.read_status()
+    return results
+
+
 def bench_few(a) -> dict:
     """The few-token kernels (``csrc/gemv.cu``) at the headline sizes: the qkv and output projections of
     ``--tokens`` tokens, and the routed gate/up and down products of their routes.  Six copies of the dense
@@ -711,7 +845,7 @@ def bench_sample(a) -> dict:
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="microbench")
     sub = ap.add_subparsers(dest="case", required=True)
-    for name in ("moe", "attention", "sample", "sparse", "few", "rows", "gla", "kekopel", "nusudra", "vodatar"):
+    for name in ("moe", "attention", "sample", "sparse", "few", "rows", "gla", "kekopel", "nusudra", "vodatar", "gizulorn"):
         p = sub.add_parser(name)
         p.add_argument("--iters", type=int, default=20)
         p.add_argument("--warmup", type=int, default=5)
@@ -743,6 +877,7 @@ def main(argv=None) -> int:
             p.add_argument("--tied", action="store_true", help="the values are the keys (one slab)")
             p.add_argument("--dist-bias", type=int, default=0, help="entries per head of a bias by distance (0 = none)")
             p.add_argument("--window", type=int, default=0, help="a sliding window of this many tokens (0 = none)")
+            p.add_argument("--keep-first", type=int, default=0, help="with --window: first tokens that stay visible")
             p.add_argument("--softcap", type=float, default=0.0, help="scores become cap * tanh(score / cap) (0 = as they are)")
             p.add_argument("--maps", type=int, default=1, help="softmax maps a head: query rows that are zero outside their map")
             p.add_argument("--sink", action="store_true", help="a sink of logit 0 in the softmax's denominator")
@@ -798,6 +933,22 @@ def main(argv=None) -> int:
             p.add_argument("--experts", type=int, default=64)
             p.add_argument("--identity", type=int, default=8)
             p.add_argument("--top-k", type=int, default=8)
+        elif name == "gizulorn":
+            p.add_argument("--tokens", type=int, default=2048)
+            p.add_argument("--batch", type=int, default=0, help="requests with one token each instead of one portion")
+            p.add_argument("--context", type=int, default=2048)
+            p.add_argument("--hidden", type=int, default=3072)
+            p.add_argument("--taps", type=int, default=4)
+            p.add_argument("--heads", type=int, default=48)
+            p.add_argument("--kv-heads", type=int, default=8)
+            p.add_argument("--dim", type=int, default=128)
+            p.add_argument("--vdim", type=int, default=128)
+            p.add_argument("--experts", type=int, default=64)
+            p.add_argument("--groups", type=int, default=4)
+            p.add_argument("--keep", type=int, default=2, help="open groups of experts")
+            p.add_argument("--top-k", type=int, default=8)
+            p.add_argument("--chunk", type=int, default=64)
+            p.add_argument("--only", default=None, help="cases whose name holds this text")
         elif name == "few":
             p.add_argument("--tokens", type=int, default=1)
             p.add_argument("--hidden", type=int, default=3072)
@@ -835,7 +986,8 @@ def main(argv=None) -> int:
             p.add_argument("--temperature", type=float, default=0.0)
     a = ap.parse_args(argv)
     res = {"moe": bench_moe, "attention": bench_attention, "sample": bench_sample, "sparse": bench_sparse, "few": bench_few,
-           "rows": bench_rows, "gla": bench_gla, "kekopel": bench_kekopel, "nusudra": bench_nusudra, "vodatar": bench_vodatar}[a.case](a)
+           "rows": bench_rows, "gla": bench_gla, "kekopel": bench_kekopel, "nusudra": bench_nusudra, "vodatar": bench_vodatar,
+           "gizulorn": bench_gizulorn}[a.case](a)
     print(json.dumps({"case": a.case, **{k: v for k, v in vars(a).items() if k != "case"}, "result": res}))
     return 0
 

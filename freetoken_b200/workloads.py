@@ -20,7 +20,8 @@ attention with a learned sink per head and matrix memory in turns; dense and inp
 and Nusudra (several residual streams, latent attention, attention beside Mamba-2, the gated delta rule) and Vodatar
 (norms over groups on both sides of every sub-layer, a short convolution in front and a gate behind, differential
 attention with a soft cap and latent attention in turns, identity experts and a gated shared expert, a looped range)
-beside MiniMax-M3 at equal layer sizes, all with random weights: a
+and Gizulorn (windowed attention that keeps its first tokens beside the delta rule with a decay per key channel, and
+retention, in turns; dense feed-forwards and experts in groups) beside MiniMax-M3 at equal layer sizes, all with random weights: a
 2 048-token prompt in one step and decode steps of eight requests at 2 048 tokens of context, at a few
 sizes that resemble real models' layers.
 
@@ -208,7 +209,20 @@ def _design_configs(width, heads, kv, dim, experts, top, ff, vocab, layers):
             "residual_mult": 0.5, "canon": {"taps": 4}, "loop": {"start": 1, "stop": layers, "times": 1},
             "layers": [{"type": "latent_attention" if i % 2 else "attention", "mixer": vlat if i % 2 else vatt, "mlp": vmlp}
                        for i in range(layers)]}
-    return {"rumalorn": ruma, "pabavik": paba, "kekopel": keko, "nusudra": nusu, "vodatar": voda, "minimax_m3": m3}
+    # Gizulorn: attention with the same window, four kept tokens and a sink per head beside the delta rule (heads as Nusudra's),
+    # and retention, in turns; dense feed-forwards as wide as a token's experts, and the same experts in four groups of
+    # which two are open, with a shared expert of an expert's width
+    gleft = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window, "keep_first": 4},
+             "rot": {"dims": dim, "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    gpair = {"left": gleft, "right": dict(delta, decay_rank=dim, gate_rank=dim), "left_scale": 0.8, "right_scale": 1.1}
+    gret = {"heads": heads, "dim": dim, "vdim": dim, "decay": [1.0 - 2.0 ** -(5 + 5 * i / heads) for i in range(heads)],
+            "rot": {"dims": dim, "base": 10000.0}}
+    gmoe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "groups": {"count": 4, "keep": 2}},
+            "shared": {"ff": ff}}
+    gizu = {"architecture": "Gizulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": [{"type": "retention", "mixer": gret, "mlp": gmoe} if i % 2 else
+                       {"type": "parallel", "mixer": gpair, "mlp": {"kind": "dense", "ff": top * ff}} for i in range(layers)]}
+    return {"rumalorn": ruma, "pabavik": paba, "kekopel": keko, "nusudra": nusu, "vodatar": voda, "gizulorn": gizu, "minimax_m3": m3}
 
 
 def _time_design(raw: Dict[str, Any], prompt: int, batch: int, steps: int, warmup: int) -> Dict[str, Any]:

@@ -177,13 +177,13 @@ def attention_problem(dtype, Hq, Hkv, D, P, segs, seed=0, scale_k=1.0):
 
 
 def run_attention(dtype, Hq, Hkv, D, P, segs, tile, window, sink, fixed_splits=None, force_split=False, problem=None,
-                  kv_split=1, scale=None):
+                  kv_split=1, scale=None, keep_first=0):
     q, ks, vs, bt, seg = problem or attention_problem(dtype, Hq, Hkv, D, P, segs)
     kw = dict(sm_count=4096, min_split_keys=32) if force_split else dict(sm_count=148)
     if tile == 128:
         kw["key_tile"] = 128  # as the engine plans the tcgen05 kernel's work
     Hv = Hkv * kv_split
-    plan = build_plan(segs, Hq // Hv, tile, window, Hv, fixed_splits=fixed_splits, **kw)
+    plan = build_plan(segs, Hq // Hv, tile, window, Hv, fixed_splits=fixed_splits, keep_first=keep_first, **kw)
     items = torch.from_numpy(plan.items).to(DEV)
     part_o = part_ml = None
     if plan.n_slots:
@@ -193,8 +193,9 @@ def run_attention(dtype, Hq, Hkv, D, P, segs, tile, window, sink, fixed_splits=N
     want = torch.empty_like(out)
     scale = scale or 0.8 * D ** -0.5
     ops.paged_attention(q, ks, vs, bt, seg, len(segs), items, plan.n_items, part_o, part_ml, out, tile, scale, window,
-                        kv_split=kv_split, sink=sink)
-    ref.paged_attention(q, ks, vs, bt, seg, len(segs), items, plan.n_items, None, None, want, tile, scale, window, sink=sink)
+                        kv_split=kv_split, sink=sink, keep_first=keep_first)
+    ref.paged_attention(q, ks, vs, bt, seg, len(segs), items, plan.n_items, None, None, want, tile, scale, window, sink=sink,
+                        keep_first=keep_first)
     return out, want, plan
 
 
