@@ -73,15 +73,23 @@ __host__ __device__ constexpr size_t delta_smem_bytes() {
 }
 
 // the decays of all of a step's tokens, in place
-__global__ void delta_decay_kernel(float* z, const float* __restrict__ a_log, const float* __restrict__ dt_bias, long long n, int D, int hd) {
+// (a thread keeps its channel; blocks of a grid column take the tokens in turns)
+constexpr int kDecayTokens = 8;  // tokens a thread has in flight
+__global__ void __launch_bounds__(128) delta_decay_kernel(float* z, const float* __restrict__ a_log, const float* __restrict__ dt_bias,
+                                                          int n_tokens, int D, int hd) {
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  const bool live = c < hd;
+  const float rate = live ? -expf(a_log[c / D]) : 0.f, bias = live ? dt_bias[c] : 0.f;
   pdl_wait();
   pdl_trigger();
-  long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-  const long long stride = (long long)gridDim.x * blockDim.x;
-  for (; i < n; i += stride) {
-    const int c = (int)(i % hd);
-    z[i] = expf(-expf(a_log[c / D]) * delta_softplus(z[i] + dt_bias[c]));
-  }
+  if (!live) return;
+  const int t0 = blockIdx.y * kDecayTokens;
+  float v[kDecayTokens];
+#pragma unroll
+  for (int u = 0; u < kDecayTokens; ++u) v[u] = t0 + u < n_tokens ? z[(size_t)(t0 + u) * hd + c] : 0.f;
+#pragma unroll
+  for (int u = 0; u < kDecayTokens; ++u)
+    if (t0 + u < n_tokens) z[(size_t)(t0 + u) * hd + c] = expf(rate * delta_softplus(v[u] + bias));
 }
 
 template <typename T, int DPT, int LPC, bool CH>
@@ -433,7 +441,11 @@ template <typename T, int DPT, int LPC, bool CH>
 static int launch_delta_as(const DeltaArgs& a, cudaStream_t s) {
   constexpr int kDeltaCols = delta_cols<LPC>();
   dim3 grid(a.n_segs, a.H, (a.Dv + kDeltaCols - 1) / kDeltaCols);
-  constexpr size_t smem = delta_smem_bytes<T, DPT, LPC, CH>();
+  // A long request's blocks all run to the request's end.  They start while the kernel before still fills the SMs, and would
+  // gather on the first SMs with room: each takes as much shared memory as spreads the grid over all of them.
+  const long long per_sm = ((long long)grid.x * grid.y * grid.z + 147) / 148;
+  size_t smem = delta_smem_bytes<T, DPT, LPC, CH>();
+  if (a.n_tokens > a.n_segs && per_sm <= 4) smem = max(smem, (size_t)(200 * 1024) / (size_t)per_sm - 8 * 1024);
   auto kern = delta_scan_kernel<T, DPT, LPC, CH>;
   if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   FTK_LAUNCH(kern, grid, kDeltaThreads, smem, s, a);
@@ -452,10 +464,12 @@ static int launch_delta(DeltaArgs a, cudaStream_t s) {
   a.wide = a.D % e == 0 && a.Dv % e == 0 && a.q_stride % e == 0 && a.k_stride % e == 0 && a.v_stride % e == 0 &&
            (((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.z) & 15) == 0;
   if (a.z && a.n_tokens > a.n_segs) {  // some request brings several tokens
-    const long long n = (long long)a.n_tokens * a.H * a.D;
-    const unsigned blocks = (unsigned)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
-    FTK_LAUNCH(delta_decay_kernel, blocks, 256, 0, s, a.z, a.a_log, a.dt_bias, n, a.D, a.H * a.D);
-    FTK_LAUNCH_CHECK("delta_scan (decays)");
+    for (int t0 = 0; t0 < a.n_tokens; t0 += 65535 * kDecayTokens) {
+      const int nt = min(a.n_tokens - t0, 65535 * kDecayTokens);
+      const dim3 dgrid((a.H * a.D + 127) / 128, (nt + kDecayTokens - 1) / kDecayTokens);
+      FTK_LAUNCH(delta_decay_kernel, dgrid, 128, 0, s, a.z + (size_t)t0 * a.H * a.D, a.a_log, a.dt_bias, nt, a.D, a.H * a.D);
+      FTK_LAUNCH_CHECK("delta_scan (decays)");
+    }
     a.z_is_decay = 1;
   }
   if (a.D <= 16) return launch_delta_sized<T, 4, 4>(a, s);

@@ -181,7 +181,7 @@ __device__ __forceinline__ bool step_state(const FtkStreamStep& p, int row, floa
 // and the request's earlier inputs, which a kernel of an earlier step wrote) before the wait on the kernel before.
 // ROUTED: the result is a sum over expert routes.  TAPS: the tap count where it is four, else 0.
 template <typename T, int PER, bool ROUTED, bool CONV, int TAPS, int MAX_THREADS>
-__global__ void __launch_bounds__(MAX_THREADS) stream_step_regs_kernel(const __grid_constant__ StepArgs a) {
+__global__ void __launch_bounds__(MAX_THREADS, MAX_THREADS <= 256 && PER <= 3 ? 2 : 1) stream_step_regs_kernel(const __grid_constant__ StepArgs a) {
   const FtkStreamStep& p = a.p;
   __shared__ float red[2][32];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
