@@ -47,7 +47,8 @@ TC_MIN_DECODE_SPAN = 0   # decode steps go there from this length of the longest
 
 def attention_kernel_form(dtype: torch.dtype, decode_only: bool = False, group: int = 1, n_tokens: int = 0,
                           head_dim: int = 0, page_size: int = 0, window: Optional[int] = None,
-                          longest_span: int = 0, one_tile_only: bool = False, no_few: bool = False) -> Tuple[int, bool]:
+                          longest_span: int = 0, one_tile_only: bool = False, no_few: bool = False,
+                          window_on_tc: bool = False) -> Tuple[int, bool]:
     """``(query rows one attention CTA handles, the tcgen05 kernel's form for few rows)``.
 
     16 rows in the 32-bit kernel.  bfloat16 steps whose sizes the tcgen05 kernels take: 128 rows for
@@ -58,7 +59,9 @@ def attention_kernel_form(dtype: torch.dtype, decode_only: bool = False, group: 
     decode steps go to the same kernel in its form for tiles of at
     most 16 rows, where one warp takes the softmax (groups of up to 16 heads; ``longest_span`` is the longest
     request's length rounded up to a power of two, from which on they go there:
-    ``TC_MIN_DECODE_SPAN``), larger groups to the 128-row kernel.  Otherwise 16 rows for decode steps
+    ``TC_MIN_DECODE_SPAN``), larger groups and, with ``window_on_tc``, windows to the 128-row kernel (measured on B200, 48 heads on 8 of 128, a window of
+    1,024, with and without kept first tokens: 8.5 to 13 microseconds against 16 to 22 for one request, 14 to 18 against 23 to
+    25 for eight, 74 to 93 against 105 to 111 for 64).  Otherwise 16 rows for decode steps
     of small groups and 64 in the bfloat16 mma.sync kernels.  ``one_tile_only``: of the tcgen05 kernels only
     the ones with a single query tile a piece may be chosen (they are the ones that take a bias by distance);
     ``no_few``: nor the form for tiles of at most 16 rows (a window or a sink: the 128-row form alone takes them)."""
@@ -68,8 +71,8 @@ def attention_kernel_form(dtype: torch.dtype, decode_only: bool = False, group: 
     if window is not None:  # (of the tcgen05 kernels the one with a single 128-row tile a piece takes a window)
         one_tile_only = no_few = True
     if decode_only:
-        if sized and not no_few and longest_span >= TC_MIN_DECODE_SPAN:
-            if ops.attention_tc_few_fits(head_dim, page_size, group):
+        if sized and (not no_few or (window is not None and window_on_tc)) and longest_span >= TC_MIN_DECODE_SPAN:
+            if not no_few and ops.attention_tc_few_fits(head_dim, page_size, group):
                 return 16, True
             if ops.attention_tc_fits(head_dim, page_size, group):
                 return 128, False
@@ -235,7 +238,7 @@ class GQAttention(Mixer):
         special = has_sink or self.window is not None
         return attention_kernel_form(self.env.dtype, decode_only, self.plan_group, n_tokens,
                                      self.pad_dim if sized else 0, page_size, self.window, longest_span,
-                                     one_tile_only=special or self.log_dist_bias, no_few=special)
+                                     one_tile_only=special or self.log_dist_bias, no_few=special, window_on_tc=True)
 
     def tile_rows(self, decode_only: bool, n_tokens: int = 0, page_size: int = 0, longest_span: int = 0) -> int:
         return self.kernel_form(decode_only, n_tokens, page_size, longest_span)[0]

@@ -254,6 +254,7 @@ def test_which_attention_kernel_a_step_gets():
     assert form(bf, False, 6, 4096, 128, 16) == (256, False)
     assert rows(bf, True, 6, 8, 64, 16, None, 4096) == 16            # head size it does not take
     assert rows(bf, True, 6, 8, 128, 16, 512, 4096) == 16            # a window
+    assert form(bf, True, 6, 8, 128, 16, 512, 4096, no_few=True, window_on_tc=True) == (128, False)
     assert rows(bf, True, 6, 8, 128, 8, None, 4096) == 16            # pages of 8 tokens
     assert rows(bf, False, 6, TC_MIN_TOKENS - 1, 128, 16) == 64
     assert rows(bf, False, 6, TC_MIN_TOKENS, 128, 16) == 128

@@ -475,7 +475,9 @@ def test_heads_of_128_run_the_tensor_core_attention(tmp_path_factory):
     check_rows(replay_whole(eng, "w", toks), plain, toks, "bfloat16", "whole", want=want)
     forms = ops.variant_counts()
     assert forms.get("attention: tcgen05, 128-row query tiles, window or sink", 0) == 1, forms
+    ops.variant_counts(reset=True)
     check_rows(replay_cuts(eng, "c", toks, [250, 130, 2]), plain, toks, "bfloat16", "portions, the rest one by one", want=want)
+    assert eng.graphs and not any("mma.sync, 16-row" in k for k in ops.variant_counts())  # single tokens too
     others = {f"o{i}": tokens_for(plain.vocab, 20 + i, 20 + i) for i in range(3)}
     for r, t in others.items():  # three requests that decode beside a long portion
         eng.step([StepEntry(r, t[:-1], [])])
