@@ -292,7 +292,7 @@ def designs(raw: Dict[str, Any], layers: int = 4, prompt: int = 2048, batch: int
             row[design] = _time_design(cfg, prompt, batch, steps, warmup)
             gc.collect()
             torch.cuda.empty_cache()
-        for design in ("rumalorn", "pabavik", "kekopel", "nusudra", "vodatar"):
+        for design in ("rumalorn", "pabavik", "kekopel", "nusudra", "vodatar", "gizulorn"):
             if design not in row:
                 continue
             row[f"{design}_over_minimax_m3"] = {
